@@ -56,6 +56,15 @@ delta rule:
                  "mixer": {"left": {"heads", "kv_heads", "dim", "vdim", "scale", "mask": {"size", "pool"},
                                     "rot": {"base", "dims", "scaling": {"factor", "original", "fast", "slow"}}},
                            "right": {"heads", "dim"}}, "mlp": ...}, ...]}
+
+``BokenexRingModel``: learned positions, one scalar RMS norm a layer whose output feeds the mixer and the feed-forward side
+by side, windowed attention whose weights are sigmoids of distance-biased scores:
+
+    {"architecture": "Bokenex", "vocab": V, "width": W, "norm": {"eps": e}, "residual_mult": m, "max_positions": P,
+     "layers": [{"type": "attention",
+                 "mixer": {"heads", "kv_heads", "dim", "vdim", "conv", "scale", "mask": {"size"}},
+                 "mlp": {"kind": "dense", "ff": F}
+                      | {"kind": "moe", "router": {"experts", "top", "scale"}, "expert": {"ff"}} | null}, ...]}
 """
 from __future__ import annotations
 
@@ -116,6 +125,10 @@ def _attention_cfg(lc: _seqabi.LayerCfg, mx: dict, qk_norm, mask: str = "block",
     lc.conv = int(mx.get("conv", 0) or 0)
 
 
+_NORM_KIND = {"rms": _seqabi.DN_NORM_RMS, "dyt": _seqabi.DN_NORM_DYT, "layer": _seqabi.DN_NORM_LAYER, "rms_scalar": _seqabi.DN_NORM_RMS_SCALAR}
+_EXPERT_ACT = {"cglu": _seqabi.DN_EXPERT_CGLU, "swiglu": _seqabi.DN_EXPERT_SWIGLU, "relu2": _seqabi.DN_EXPERT_RELU2}
+
+
 def parse_layer_list(cfg: dict, family: Optional[dict] = None,
                      shapes: Optional[Dict[str, Tuple[int, ...]]] = None) -> Tuple[_seqabi.SeqCfg, List[_seqabi.LayerCfg]]:
     """config.json of a layer-list family -> the C structs.  Every size and constant comes from the config, or (what
@@ -124,6 +137,7 @@ def parse_layer_list(cfg: dict, family: Optional[dict] = None,
     fam = {"norm": "rms", "post_norm": False, "pre_norm": True, "embed_norm": False, "qk_norm": True, "sink": False, "head_gate": False,
            "mask": "block", "ff_act": "geglu", "router": "topk", "expert_act": "cglu", "shared_gate": False}
     fam.update({"v_is_k": False, "rot_layout": "interleaved", "right": "gla", "branch_norm": False})
+    fam.update({"attn_weight": "softmax", "dist_bias": False, "parallel_ff": False, "router_score": "softmax"})
     fam.update(family or {})
     shapes = shapes or {}
 
@@ -149,6 +163,8 @@ def parse_layer_list(cfg: dict, family: Optional[dict] = None,
             lc.mixer = _seqabi.DN_MIX_ATTENTION
             _attention_cfg(lc, mx, per("qk_norm", kind), fam["mask"], fam["rot_layout"])
             lc.sink, lc.out_gate, lc.v_is_k = int(per("sink", kind)), int(per("head_gate", kind)), int(per("v_is_k", kind))
+            lc.attn_weight = _seqabi.DN_ATTN_SIGMOID if fam["attn_weight"] == "sigmoid" else _seqabi.DN_ATTN_SOFTMAX
+            lc.dist_bias = int(per("dist_bias", kind))
         elif kind in ("latent_attention", "latent_attention_2"):
             # the second type sends its queries through a normed latent too, pairs rotary dims half apart and gates its heads
             second = kind == "latent_attention_2"
@@ -200,10 +216,10 @@ def parse_layer_list(cfg: dict, family: Optional[dict] = None,
                 lc.ff_act = _seqabi.DN_FF_RELU2 if fam["ff_act"] == "relu2" else _seqabi.DN_FF_GEGLU
             elif mk == "moe":
                 lc.mlp_kind = _seqabi.DN_MLP_MOE
-                swiglu = fam["expert_act"] == "swiglu"
-                lc.expert_act = _seqabi.DN_EXPERT_SWIGLU if swiglu else _seqabi.DN_EXPERT_CGLU
+                lc.expert_act = _EXPERT_ACT[fam["expert_act"]]
+                clamped = lc.expert_act == _seqabi.DN_EXPERT_CGLU      # its limits are required
                 lc.ff = int(mlp["expert"]["ff"])
-                lc.limit = float(mlp["expert"].get("limit", 0.0)) if swiglu else float(mlp["expert"]["limit"])
+                lc.limit = float(mlp["expert"]["limit"]) if clamped else 0.0
                 r = mlp["router"]
                 lc.experts, lc.top = int(r["experts"]), int(r["top"])
                 if fam["router"] == "scored":
@@ -212,10 +228,11 @@ def parse_layer_list(cfg: dict, family: Optional[dict] = None,
                     g = r.get("groups") or {}
                     lc.groups, lc.groups_keep = int(g.get("count", 0) or 0), int(g.get("keep", g.get("count", 0)) or 0)
                     lc.router_scale = float(r.get("scale", 1.0))
+                    lc.score_kind = _seqabi.DN_SCORE_SIGMOID if fam["router_score"] == "sigmoid" else _seqabi.DN_SCORE_SOFTMAX
                 sh = mlp.get("shared")
                 if sh:
                     lc.shared_ff = int(sh["ff"])
-                    lc.shared_limit = float(sh.get("limit", 0.0)) if swiglu else float(sh["limit"])
+                    lc.shared_limit = float(sh["limit"]) if clamped else 0.0
                     lc.shared_gate = int(fam["shared_gate"])
             else:
                 raise ValueError(f"layer {i}: feed-forward kind {mk!r} unsupported")
@@ -223,7 +240,9 @@ def parse_layer_list(cfg: dict, family: Optional[dict] = None,
     sc = _seqabi.SeqCfg(width=int(cfg["width"]), vocab=int(cfg["vocab"]), n_layers=len(layers), streams=int(cfg.get("streams", 0) or 0),
                         eps=float((cfg.get("norm") or {}).get("eps", 1e-6)),
                         embed_scale=float((cfg.get("embedding") or {}).get("scale", 1.0)))
-    sc.norm_kind = {"dyt": _seqabi.DN_NORM_DYT, "layer": _seqabi.DN_NORM_LAYER}.get(fam["norm"], _seqabi.DN_NORM_RMS)
+    sc.norm_kind = _NORM_KIND[fam["norm"]]
+    sc.parallel_ff, sc.residual_mult = int(fam["parallel_ff"]), float(cfg.get("residual_mult", 1.0))
+    sc.max_positions = int(cfg.get("max_positions", 0) or 0)
     sc.canon_taps = int((cfg.get("canon") or {}).get("taps", 0) or 0)
     bg = (cfg.get("embedding") or {}).get("bigram")
     if bg:
@@ -282,6 +301,7 @@ class SeqMixRingModel(BaseRingModel):
         self.abs_to_local = {i: i for i in self.layers}
         self.hidden_size, self.vocab_size = int(sc.width), int(sc.vocab)
         self.max_seqs, self.max_batch_tokens, self.pool_pages = int(sc.max_seqs), int(sc.max_batch_tokens), int(sc.pool_pages)
+        self.max_positions = int(sc.max_positions)      # longest sequence (0: no limit but the pool)
         self._bound: Dict[str, torch.Tensor] = {}
 
     # -- weights -----------------------------------------------------------------------------
@@ -291,14 +311,18 @@ class SeqMixRingModel(BaseRingModel):
         sc = self._cfg_struct
         dyt = sc.norm_kind == _seqabi.DN_NORM_DYT
         lnorm = sc.norm_kind == _seqabi.DN_NORM_LAYER
-        out: Dict[str, Tuple[int, ...]] = {"embed": (V, W), "final.norm": (W,)}
+        scalar = sc.norm_kind == _seqabi.DN_NORM_RMS_SCALAR
+        relu2_bias = self.family.get("ff_bias", True)
+        out: Dict[str, Tuple[int, ...]] = {"embed": (V, W)}
+        if sc.max_positions > 0:
+            out["pos"] = (sc.max_positions, W)
         if sc.bigram_buckets > 0:
             out["bigram"] = (sc.bigram_buckets + 1, W)
         if not self.family.get("tied_head"):
             out["head"] = (V, W)
 
         def norm(name: str) -> None:
-            out[name] = (W,)
+            out[name] = () if scalar else (W,)
             if dyt:
                 out[name + ".b"], out[name + ".alpha"] = (W,), ()
             if lnorm:
@@ -354,6 +378,10 @@ class SeqMixRingModel(BaseRingModel):
                     out[p + "sink"] = (lc.heads,)
                 if lc.out_gate:
                     out[p + "head_gate"] = (lc.heads, W)
+                if lc.dist_bias:
+                    out[p + "mix.r1"] = out[p + "mix.r2"] = (lc.heads,)
+                if lc.attn_weight == _seqabi.DN_ATTN_SIGMOID:
+                    out[p + "mix.pb"] = (lc.heads,)
             if lc.mixer == _seqabi.DN_MIX_PARALLEL and lc.r_kind == _seqabi.DN_RIGHT_GDELTA:
                 rc = lc.r_heads * lc.r_dim
                 for q in "qkvga":
@@ -380,26 +408,32 @@ class SeqMixRingModel(BaseRingModel):
                 out[p + "mix.A_log"] = out[p + "mix.dt_bias"] = (lc.heads,)
                 out[p + "mix.norm"] = (lc.vdim,)
             if lc.ff > 0:
-                if not sc.no_pre_norm:
+                if not sc.no_pre_norm and not sc.parallel_ff:
                     norm(p + "norm2")
                 if sc.post_norm:
                     norm(p + "post2")
                 if lc.mlp_kind == _seqabi.DN_MLP_MOE:
                     if lc.router_kind == _seqabi.DN_ROUTER_SCORED:
-                        out[p + "router"], out[p + "router.corr"] = (lc.experts + lc.identity, W), (lc.experts + lc.identity,)
+                        out[p + "router"] = (lc.experts + lc.identity, W)
+                        if self.family.get("router_corr", True):
+                            out[p + "router.corr"] = (lc.experts + lc.identity,)
                     else:
                         out[p + "router"], out[p + "router.b"] = (lc.experts, W), (lc.experts,)
                     if lc.shared_ff > 0 and lc.shared_gate:
                         out[p + "shared.sg"] = (1, W)
+                    gated = lc.expert_act != _seqabi.DN_EXPERT_RELU2
                     for e in range(lc.experts):
-                        out[f"{p}mlp.e{e}.gate"] = out[f"{p}mlp.e{e}.up"] = (lc.ff, W)
-                        out[f"{p}mlp.e{e}.down"] = (W, lc.ff)
+                        if gated:
+                            out[f"{p}mlp.e{e}.gate"] = (lc.ff, W)
+                        out[f"{p}mlp.e{e}.up"], out[f"{p}mlp.e{e}.down"] = (lc.ff, W), (W, lc.ff)
                     if lc.shared_ff > 0:
-                        out[p + "shared.gate"] = out[p + "shared.up"] = (lc.shared_ff, W)
-                        out[p + "shared.down"] = (W, lc.shared_ff)
+                        if gated:
+                            out[p + "shared.gate"] = (lc.shared_ff, W)
+                        out[p + "shared.up"], out[p + "shared.down"] = (lc.shared_ff, W), (W, lc.shared_ff)
                 elif lc.ff_act == _seqabi.DN_FF_RELU2:
-                    out[p + "mlp.up"], out[p + "mlp.up.b"] = (lc.ff, W), (lc.ff,)
-                    out[p + "mlp.down"], out[p + "mlp.down.b"] = (W, lc.ff), (W,)
+                    out[p + "mlp.up"], out[p + "mlp.down"] = (lc.ff, W), (W, lc.ff)
+                    if relu2_bias:
+                        out[p + "mlp.up.b"], out[p + "mlp.down.b"] = (lc.ff,), (W,)
                 else:
                     out[p + "mlp.gate"] = out[p + "mlp.up"] = (lc.ff, W)
                     out[p + "mlp.down"] = (W, lc.ff)
@@ -613,3 +647,16 @@ class VulanexRingModel(SeqMixRingModel):
                      "mix.right.a.b": "r.ab", "mix.right.w1": "decay1", "mix.right.w2": "decay2", "mix.right.w0": "decay.b",
                      "mix.right.norm": "r.norm", "mix.right.o": "r.o"},
     }
+
+
+class BokenexRingModel(SeqMixRingModel):
+    """Bokenex: a learned position row on the embedding; layers of one scalar RMS norm whose output the mixer and the
+    feed-forward read side by side, both joining the residual together times a factor; GQA attention with short convolutions
+    and per-head q / k norms, no rotation, a sliding window, a score that falls with the logarithm of the distance and
+    weights that are sigmoids of the scores (nothing is normalized over the keys); a dense relu-squared feed-forward or
+    experts chosen and weighed by sigmoid scores."""
+
+    model_type = "bokenex"
+    family = {"norm": "rms_scalar", "parallel_ff": True, "qk_norm": "head", "mask": "window", "attn_weight": "sigmoid", "dist_bias": True,
+              "ff_act": "relu2", "ff_bias": False, "router": "scored", "router_score": "sigmoid", "router_corr": False, "expert_act": "relu2"}
+    tensor_alias = {"*": _MOE_ALIAS}

@@ -242,9 +242,14 @@ extern "C" int dn_seq_model_create(const dn_seq_cfg* cfg, const dn_seq_layer_cfg
   const bool looped = cfg->loop_times > 0;
   if (looped && (cfg->loop_start < 0 || cfg->loop_stop > cfg->n_layers || cfg->loop_start >= cfg->loop_stop))
     rc = fail(DN_EINVAL, "loop [%d, %d) x %d does not fit %d layers", cfg->loop_start, cfg->loop_stop, cfg->loop_times, cfg->n_layers);
-  if (rc == DN_OK && cfg->norm_kind != DN_NORM_RMS && cfg->norm_kind != DN_NORM_DYT && cfg->norm_kind != DN_NORM_LAYER) rc = fail(DN_EINVAL, "norm kind %d unknown", cfg->norm_kind);
+  if (rc == DN_OK && cfg->norm_kind != DN_NORM_RMS && cfg->norm_kind != DN_NORM_DYT && cfg->norm_kind != DN_NORM_LAYER && cfg->norm_kind != DN_NORM_RMS_SCALAR) rc = fail(DN_EINVAL, "norm kind %d unknown", cfg->norm_kind);
   if (rc == DN_OK && cfg->norm_kind != DN_NORM_DYT && cfg->embed_norm) rc = fail(DN_EINVAL, "a norm on the embedding exists as dynamic tanh only");
-  if (rc == DN_OK && cfg->norm_kind == DN_NORM_LAYER && (cfg->post_norm || cfg->no_pre_norm)) rc = fail(DN_EINVAL, "layer norms stand before the sublayers only");
+  if (rc == DN_OK && (cfg->norm_kind == DN_NORM_LAYER || cfg->norm_kind == DN_NORM_RMS_SCALAR) && (cfg->post_norm || cfg->no_pre_norm))
+    rc = fail(DN_EINVAL, "layer norms and RMS norms with one number stand before the sublayers only");
+  if (rc == DN_OK && cfg->parallel_ff && (cfg->post_norm || cfg->no_pre_norm || cfg->streams > 0 || cfg->canon_taps > 0 || cfg->norm_kind == DN_NORM_DYT))
+    rc = fail(DN_EINVAL, "mixer and feed-forward side by side need an RMS or layer norm before them, the plain residual and no input convolutions");
+  if (rc == DN_OK && cfg->residual_mult != 0.f && cfg->residual_mult != 1.f && cfg->post_norm) rc = fail(DN_EINVAL, "a residual factor behind a norm after the sublayer is unsupported");
+  if (rc == DN_OK && cfg->max_positions < 0) rc = fail(DN_EINVAL, "max_positions %d is negative", cfg->max_positions);
   if (rc == DN_OK && (cfg->canon_taps < 0 || cfg->canon_taps > 9 || (cfg->canon_taps > 0 && (cfg->no_pre_norm || cfg->norm_kind == DN_NORM_DYT || cfg->loop_times > 0))))
     rc = fail(DN_EINVAL, "input convolutions of %d taps unsupported (0..9, behind an RMS or layer norm before the sublayer, no loop)", cfg->canon_taps);
   if (rc == DN_OK && (cfg->bigram_buckets < 0 || (cfg->bigram_buckets > 0 && (cfg->bigram_mul_prev < 0 || cfg->bigram_mul_cur < 0))))
@@ -292,6 +297,11 @@ extern "C" int dn_seq_model_create(const dn_seq_cfg* cfg, const dn_seq_layer_cfg
         rc = fail(DN_EINVAL, "layer %d: pooled blocks of %d tokens stand behind a sliding window of the layer's own keys", i, c.pool);
         break;
       }
+      if ((c.attn_weight != DN_ATTN_SOFTMAX && c.attn_weight != DN_ATTN_SIGMOID) || (c.attn_weight == DN_ATTN_SIGMOID && c.sink) || (c.dist_bias && c.pool > 0)) {
+        rc = fail(DN_EINVAL, "layer %d: attention weights %d (sink %d, distance bias %d, pooled blocks of %d) unsupported", i, c.attn_weight, c.sink, c.dist_bias, c.pool);
+        break;
+      }
+      if (cfg->parallel_ff && c.mixer == DN_MIX_PARALLEL) { rc = fail(DN_EINVAL, "layer %d: a parallel mixer beside the feed-forward is unsupported", i); break; }
       if (c.qtemp_every < 0 || (c.rot_layout == DN_ROT_HALF && c.dim < c.rot_dims)) { rc = fail(DN_EINVAL, "layer %d: query scale / rotary layout unsupported", i); break; }
       if (c.rot_dims > 0) {
         // frequencies base^(-2j/dims); scaled: dims that turn fast within the original context keep theirs, slow ones are
@@ -386,14 +396,15 @@ extern "C" int dn_seq_model_create(const dn_seq_cfg* cfg, const dn_seq_layer_cfg
         break;
       }
       if (c.router_kind != DN_ROUTER_TOPK && c.router_kind != DN_ROUTER_SCORED) { rc = fail(DN_EINVAL, "layer %d: router kind %d unknown", i, c.router_kind); break; }
-      if (c.expert_act != DN_EXPERT_CGLU && c.expert_act != DN_EXPERT_SWIGLU) { rc = fail(DN_EINVAL, "layer %d: expert activation %d unknown", i, c.expert_act); break; }
+      if (c.score_kind != DN_SCORE_SOFTMAX && c.score_kind != DN_SCORE_SIGMOID) { rc = fail(DN_EINVAL, "layer %d: router score %d unknown", i, c.score_kind); break; }
+      if (c.expert_act != DN_EXPERT_CGLU && c.expert_act != DN_EXPERT_SWIGLU && c.expert_act != DN_EXPERT_RELU2) { rc = fail(DN_EINVAL, "layer %d: expert activation %d unknown", i, c.expert_act); break; }
       if (c.router_kind == DN_ROUTER_SCORED && (c.identity < 0 || c.groups < 0 || c.groups > 256 ||
                                                 (c.groups > 0 && (Et % c.groups || c.groups_keep < 1 || c.groups_keep > c.groups)))) {
         rc = fail(DN_EINVAL, "layer %d: %d + %d experts in %d groups of which %d are kept unsupported", i, c.experts, c.identity, c.groups, c.groups_keep);
         break;
       }
-      if ((c.shared_gate || (c.router_kind == DN_ROUTER_SCORED && c.identity > 0)) && !(cfg->post_norm && cfg->streams <= 0)) {
-        rc = fail(DN_EINVAL, "layer %d: a gated shared expert and identity experts are joined by the kernels of a norm after the sublayer on the plain residual", i);
+      if ((c.shared_gate || (c.router_kind == DN_ROUTER_SCORED && c.identity > 0)) && !((cfg->post_norm || cfg->parallel_ff) && cfg->streams <= 0)) {
+        rc = fail(DN_EINVAL, "layer %d: a gated shared expert and identity experts are joined on the plain residual, by a norm after the sublayer or beside the mixer", i);
         break;
       }
       l.etab_h.assign((size_t)3 * c.experts, nullptr);
@@ -535,7 +546,7 @@ extern "C" int dn_seq_bind(dn_seq_model* m, int layer, int which, const void* p)
     else if (which == DN_SQ_HEAD) {
       m->head = p;
       m->tm_head_ok = b16 && make_tmap(&m->tm_head, p, m->cfg.vocab, m->cfg.width, dn::TC_BM);
-    } else if (which > DN_SQ_HEAD && which <= DN_SQ_BIGRAM) {
+    } else if (which > DN_SQ_HEAD && which <= DN_SQ_POS) {
       m->mw[which - DN_SQ_EMBED] = p;
       if (which == DN_SQ_LOOP_IN) m->tm_loop_ok = b16 && make_tmap(&m->tm_loop_in, p, m->cfg.width, 2 * m->cfg.width, dn::TC_BM);
     } else return fail(DN_EINVAL, "tensor %d is not a model tensor", which);
@@ -718,24 +729,24 @@ template <class T>
 static bool attn_tiles_ok(const dn_seq_layer_cfg& lc, const Batch& b) {
   return std::is_same<T, bf16>::value && b.max_len >= 16 && lc.dim % 8 == 0 && lc.vdim % 8 == 0 && lc.dim <= 128 && lc.vdim <= 128;
 }
-template <int DKP, int DVP>
+template <int DKP, int DVP, bool SIG>
 static cudaError_t attn_tiles_launch(cudaStream_t s, const Batch& b, const bf16* q, const bf16* kp, const bf16* vp, const dn_seq_layer_cfg& lc,
                                      const AttnExtra& ex, bf16* out) {
   constexpr size_t smem = ((size_t)2 * AT_ROWS * (DKP + 8) + (size_t)AT_ROWS * (DVP + 8)) * 2;
   static bool attr = false;
   if (!attr) {
-    cudaError_t e = cudaFuncSetAttribute(k_attn_tiles<DKP, DVP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(k_attn_tiles<DKP, DVP, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return e;
     attr = true;
   }
   g_launches++;
-  k_attn_tiles<DKP, DVP><<<dim3(b.row_tiles, lc.heads), 128, smem, s>>>(b, q, kp, vp, lc.heads, lc.kv_heads, lc.dim, lc.vdim, lc.chunk, lc.scale, ex, out);
+  k_attn_tiles<DKP, DVP, SIG><<<dim3(b.row_tiles, lc.heads), 128, smem, s>>>(b, q, kp, vp, lc.heads, lc.kv_heads, lc.dim, lc.vdim, lc.chunk, lc.scale, ex, out);
   return cudaGetLastError();
 }
 static cudaError_t attn_tiles(cudaStream_t s, const Batch& b, const bf16* q, const bf16* kp, const bf16* vp, const dn_seq_layer_cfg& lc,
                               const AttnExtra& ex, bf16* out) {
   const int kq = lc.dim <= 32 ? 0 : lc.dim <= 64 ? 1 : 2, vq = lc.vdim <= 32 ? 0 : lc.vdim <= 64 ? 1 : 2;
-#define AT(a, c, A, Cc) if (kq == a && vq == c) return attn_tiles_launch<A, Cc>(s, b, q, kp, vp, lc, ex, out);
+#define AT(a, c, A, Cc) if (kq == a && vq == c) return ex.off ? attn_tiles_launch<A, Cc, true>(s, b, q, kp, vp, lc, ex, out) : attn_tiles_launch<A, Cc, false>(s, b, q, kp, vp, lc, ex, out);
   AT(0, 0, 32, 32) AT(0, 1, 32, 64) AT(0, 2, 32, 128) AT(1, 0, 64, 32) AT(1, 1, 64, 64) AT(1, 2, 64, 128)
   AT(2, 0, 128, 32) AT(2, 1, 128, 64) AT(2, 2, 128, 128)
 #undef AT
@@ -820,13 +831,14 @@ static int moe_ff(dn_seq_model* m, SeqLayer& l, int N, bool fused, NextNorm<T> n
   const dn_seq_layer_cfg& lc = l.c;
   const bool scored = lc.router_kind == DN_ROUTER_SCORED;
   const int W = m->cfg.width, E = lc.experts, Et = E + (scored ? lc.identity : 0), top = lc.top, P = N * top;
-  const int eact = lc.expert_act == DN_EXPERT_SWIGLU ? ACT_SWIGLU : ACT_CGLU;
+  const int eact = lc.expert_act == DN_EXPERT_SWIGLU ? ACT_SWIGLU : lc.expert_act == DN_EXPERT_RELU2 ? ACT_RELU2 : ACT_CGLU;
+  const bool gated = act_two(eact);      // experts without a gate have an up and a down matrix
   auto w = [&](int i) { return (const T*)l.w[i]; };
   auto wm = [&](int i) { return l.tm_ok[i] ? &l.tm[i] : (const CUtensorMap*)nullptr; };
   CK(mark(m, DN_SEQ_PH_ROUTER, s));
   if (scored)
     CK(launch(k_router_scored<T>, dim3(N), dim3(32 * std::min(32, std::max(4, Et + 1))), (size_t)2 * Et * 4, s, (const T*)m->h, w(DN_SQ_ROUTER), w(DN_SQ_ROUTER_CORR),
-              W, Et, top, lc.groups, lc.groups_keep, lc.router_scale, lc.shared_gate ? w(DN_SQ_SH_SG) : (const T*)nullptr, m->ridx, m->rwt, m->rpos, m->sgate));
+              W, Et, top, lc.groups, lc.groups_keep, lc.router_scale, lc.shared_gate ? w(DN_SQ_SH_SG) : (const T*)nullptr, m->ridx, m->rwt, m->rpos, m->sgate, lc.score_kind == DN_SCORE_SIGMOID ? 1 : 0));
   else
     CK(launch(k_router<T>, dim3(N), dim3(32 * std::min(32, std::max(4, E))), (size_t)E * 4, s, (const T*)m->h, w(DN_SQ_ROUTER), w(DN_SQ_ROUTER_B), W, E, top, m->ridx, m->rwt, m->rpos));
   const bool few = N <= 8;
@@ -843,7 +855,7 @@ static int moe_ff(dn_seq_model* m, SeqLayer& l, int N, bool fused, NextNorm<T> n
     MoePlan pl{m->rpos, m->rtok, m->tiles, m->tiles + m->max_tiles, m->tiles + 2 * m->max_tiles, m->tiles + 3 * m->max_tiles};
     const int mt = std::min(m->max_tiles, P / MOE_ROWS + E + 1);
     bool tc = std::is_same<T, bf16>::value && m->x_xg_ok && l.x_eact_ok && l.emaps_d && lc.ff >= 32 && W >= 32;
-    for (char ok : l.emap_ok) tc = tc && ok;
+    for (size_t i = gated ? 0 : E; i < l.emap_ok.size(); i++) tc = tc && l.emap_ok[i];
     // rows of a token tile: 128 (the tensor cores read the weight tile once for twice the tokens) when an expert gets
     // two such tiles on average, else 64 (less padding); the CUDA-core tiles are 64 rows
     const int tile_rows = tc && P / E >= 256 ? 128 : MOE_ROWS;
@@ -856,7 +868,11 @@ static int moe_ff(dn_seq_model* m, SeqLayer& l, int N, bool fused, NextNorm<T> n
       p.g_tile_e = pl.tile_e; p.g_tile_r0 = pl.tile_r0; p.g_tile_rows = pl.tile_rows; p.g_ntiles = pl.n_tiles;
       CK(mark(m, DN_SEQ_PH_MOE_UP, s));
       p.T = P; p.N = lc.ff; p.K = W; p.ldy = lc.ff; p.Y = (dn::bf16*)m->eact; p.g_mapW = l.emaps_d; p.g_mapW2 = l.emaps_d + E;
-      if (eact == ACT_SWIGLU) {
+      if (eact == ACT_RELU2) {
+        p.g_mapW = p.g_mapW2;      // the up matrices
+        if (tile_rows == 128) CK(gemm_tc_grouped<dn::EPI_RELU2, 128>(m->x_xg[1], p, s));
+        else CK(gemm_tc_grouped<dn::EPI_RELU2, 64>(m->x_xg[0], p, s));
+      } else if (eact == ACT_SWIGLU) {
         if (tile_rows == 128) CK(gemm_tc_grouped<dn::EPI_SGLU, 128>(m->x_xg[1], p, s));
         else CK(gemm_tc_grouped<dn::EPI_SGLU, 64>(m->x_xg[0], p, s));
       } else if (tile_rows == 128) CK(gemm_tc_grouped<dn::EPI_CGLU, 128>(m->x_xg[1], p, s));
@@ -874,8 +890,9 @@ static int moe_ff(dn_seq_model* m, SeqLayer& l, int N, bool fused, NextNorm<T> n
   }
   if (lc.shared_ff > 0 && !few) {
     CK(mark(m, DN_SEQ_PH_FF_UP, s));
-    CK(linear<T>(m, s, (const T*)m->h, l.w[DN_SQ_SH_GATE], l.w[DN_SQ_SH_UP], m->act, N, lc.shared_ff, W, false, eact,
-                 LinMaps{wm(DN_SQ_SH_GATE), wm(DN_SQ_SH_UP), &m->x_h}, lc.shared_limit));
+    const int first = gated ? DN_SQ_SH_GATE : DN_SQ_SH_UP;
+    CK(linear<T>(m, s, (const T*)m->h, l.w[first], l.w[DN_SQ_SH_UP], m->act, N, lc.shared_ff, W, false, eact,
+                 LinMaps{wm(first), wm(DN_SQ_SH_UP), &m->x_h}, lc.shared_limit));
     CK(mark(m, DN_SEQ_PH_FF_DOWN, s));
     CK(linear<T>(m, s, (const T*)m->act, l.w[DN_SQ_SH_DOWN], nullptr, m->y2, N, W, lc.shared_ff, true, 0, LinMaps{wm(DN_SQ_SH_DOWN), nullptr, &l.x_act}));
   }
@@ -923,6 +940,8 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
   const bool dyt = c.norm_kind == DN_NORM_DYT;
   const int lnorm = c.norm_kind == DN_NORM_LAYER ? 1 : 0;
   const int taps = c.canon_taps;
+  const int wmode = c.norm_kind == DN_NORM_RMS_SCALAR ? NW_SCALAR : dyt ? NW_PLAIN : NW_ONE_PLUS;      // weights of the width-spanning RMS norms
+  const float rmul = c.residual_mult != 0.f ? c.residual_mult : 1.f;
   const bool pre = !c.no_pre_norm;      // false: the sublayers read the residual itself, h = T(x)
   auto mwp = [&](int which) { return (const T*)m->mw[which - DN_SQ_EMBED]; };
   auto write_back = [&](const T* mix, const T* out) {
@@ -957,7 +976,7 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
   PH(DN_SEQ_PH_EMBED);
   CK(launch(k_embed<T>, dim3(N), dim3(128), 0, s, (const T*)m->embed, b, c.embed_scale, W, S1, m->xs, mwp(DN_SQ_EMBED_NORM), mwp(DN_SQ_EMBED_NORM_B),
             c.embed_norm ? mwp(DN_SQ_EMBED_NORM_ALPHA) : (const T*)nullptr, m->x0, pre ? (T*)nullptr : (T*)m->h,
-            c.bigram_buckets > 0 ? mwp(DN_SQ_BIGRAM) : (const T*)nullptr));
+            c.bigram_buckets > 0 ? mwp(DN_SQ_BIGRAM) : (const T*)nullptr, c.max_positions > 0 ? mwp(DN_SQ_POS) : (const T*)nullptr));
   // the norm before a sublayer and, where the model has them, the sublayer's input convolution with its carried rows
   auto norm_in = [&](SeqLayer& l, const Run& run, int q) -> int {
     auto w = [&](int i) { return (const T*)l.w[i]; };
@@ -966,7 +985,7 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
     T* dst = taps > 0 && !fused ? (T*)m->hn : (T*)m->h;
     T* cst = taps > 0 ? (T*)m->conv_state + run.canon_off[q] : (T*)nullptr;
     const T* cwq = taps > 0 ? w(q == 0 ? DN_SQ_CANON1 : DN_SQ_CANON2) : (const T*)nullptr;
-    CK(launch(k_read_norm<T>, dim3(N), nthr, nsm, s, m->xs, N, W, S, w(q == 0 ? DN_SQ_HC1_IN : DN_SQ_HC2_IN), w(nrm), dyt ? 0 : 1, 0, c.eps, (const int32_t*)nullptr, dst,
+    CK(launch(k_read_norm<T>, dim3(N), nthr, nsm, s, m->xs, N, W, S, w(q == 0 ? DN_SQ_HC1_IN : DN_SQ_HC2_IN), w(nrm), wmode, 0, c.eps, (const int32_t*)nullptr, dst,
               w(nb), dyt ? w(na) : (const T*)nullptr, lnorm, fused ? cwq : (const T*)nullptr, taps, b.slot, cst, m->conv_stride));
     if (taps > 0 && !fused) {
       CK(mark(m, DN_SEQ_PH_CANON, s));
@@ -977,6 +996,20 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
         CK(launch(k_conv_carry<T>, dim3((W + 127) / 128, b.E, 1), dim3(128), 0, s, cs, taps, b, cst, m->conv_stride));
       }
     }
+    return DN_OK;
+  };
+  // a dense feed-forward: h [N, W] -> y [N, W] fp32
+  auto dense_ff = [&](SeqLayer& l, int N, float* y) -> int {
+    const dn_seq_layer_cfg& lc = l.c;
+    auto wm = [&](int i) { return l.tm_ok[i] ? &l.tm[i] : (const CUtensorMap*)nullptr; };
+    PH(DN_SEQ_PH_FF_UP);
+    if (lc.ff_act == DN_FF_RELU2)      // no gate: relu(W_up h + b)^2
+      CK(linear<T>(m, s, (const T*)m->h, l.w[DN_SQ_UP], nullptr, m->act, N, lc.ff, W, false, ACT_RELU2, LinMaps{wm(DN_SQ_UP), nullptr, &m->x_h}, 0.f, l.w[DN_SQ_UP_B]));
+    else
+      CK(linear<T>(m, s, (const T*)m->h, l.w[DN_SQ_GATE], l.w[DN_SQ_UP], m->act, N, lc.ff, W, false, ACT_GEGLU, LinMaps{wm(DN_SQ_GATE), wm(DN_SQ_UP), &m->x_h}));
+    PH(DN_SEQ_PH_FF_DOWN);
+    CK(linear<T>(m, s, (const T*)m->act, l.w[DN_SQ_DOWN], nullptr, y, N, W, lc.ff, true, 0, LinMaps{wm(DN_SQ_DOWN), nullptr, &l.x_act}, 0.f,
+                 lc.ff_act == DN_FF_RELU2 ? l.w[DN_SQ_DOWN_B] : nullptr));
     return DN_OK;
   };
   bool h_ready = !pre;
@@ -1007,14 +1040,18 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
     T* cst = (T*)m->conv_state + run.conv_off;
     float* st = m->delta_state + run.state_off;
     const bool few = N <= 8;      // a decode step: all projections of the mixer in one launch of the row kernel
-    float ja = 1.f, jb = 0.f;
+    float ja = rmul, jb = 0.f;
     const float* jy2 = nullptr;
     LinSegs sg;
     memset(&sg, 0, sizeof(sg));
-    auto add = [&](const void* x, int which, void* y, int rows, int o32) {
+    auto add = [&](const void* x, int which, void* y, int rows, int o32, int act = ACT_NONE, int K = 0) {
       if (rows <= 0) return;
-      sg.X[sg.n] = x; sg.W[sg.n] = l.w[which]; sg.Y[sg.n] = y; sg.O[sg.n] = rows; sg.out32[sg.n] = o32; sg.act[sg.n] = ACT_NONE; sg.n++;
+      sg.X[sg.n] = x; sg.W[sg.n] = l.w[which]; sg.Y[sg.n] = y; sg.O[sg.n] = rows; sg.out32[sg.n] = o32; sg.act[sg.n] = act; sg.K[sg.n] = K; sg.n++;
     };
+    // a decode step whose dense feed-forward reads the mixer's input: its up product rides with the projections, its down product
+    // with the output product
+    const bool ride = few && c.parallel_ff && lc.ff > 0 && lc.mlp_kind == DN_MLP_DENSE && lc.ff_act == DN_FF_RELU2 && lc.mixer == DN_MIX_ATTENTION &&
+                      !l.w[DN_SQ_UP_B] && !l.w[DN_SQ_DOWN_B];
     auto run_segs = [&]() {
       int blocks = 0;
       for (int i = 0; i < sg.n; i++) blocks += (sg.O[i] + 7) / 8;
@@ -1026,6 +1063,7 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
         add(nullptr, DN_SQ_Q, m->uq, l.Cq, 0); add(nullptr, DN_SQ_K, m->uk, l.Ck, 0); add(nullptr, DN_SQ_V, m->uv, l.Cv, 0);
         if (lc.mixer == DN_MIX_DELTA) { add(nullptr, DN_SQ_A, m->pa, lc.heads, 1); add(nullptr, DN_SQ_B, m->pb, lc.heads, 1); add(nullptr, DN_SQ_G, m->gt, l.Co, 0); }
         if (lc.mixer != DN_MIX_DELTA && lc.out_gate) add(nullptr, DN_SQ_HEAD_GATE, m->pa, lc.heads, 1);
+        if (ride) add(nullptr, DN_SQ_UP, m->act, lc.ff, 0, ACT_RELU2);
         CK(run_segs());
       } else {
         CK(linear<T>(m, s, (const T*)m->h, l.w[DN_SQ_Q], nullptr, m->uq, N, l.Cq, W, false, 0, LinMaps{wm(DN_SQ_Q), nullptr, &m->x_h}));
@@ -1038,18 +1076,19 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
     if (lc.mixer == DN_MIX_ATTENTION || lc.mixer == DN_MIX_PARALLEL) {
       AttnPrep a{lc.heads, lc.kv_heads, lc.dim, lc.vdim, lc.conv, lc.rot_dims, l.Ck ? 1 : 0, lc.qk_norm, c.eps, l.inv_freq,
                  lc.v_is_k ? 0 : 1, lc.rot_layout == DN_ROT_HALF ? 1 : 0, lc.yarn_factor > 0.f ? 0.1f * logf(lc.yarn_factor) + 1.f : 1.f,
-                 lc.qtemp_coef, lc.qtemp_every};
+                 lc.qtemp_coef, lc.qtemp_every, lc.conv > 0 && b.max_len == 1 ? 1 : 0};
       // values that are the keys: the value pool is the key pool (row stride G dk); the pooled rows likewise
       const void* vpl = lc.v_is_k ? m->kpool[run.kv_index] : m->vpool[run.kv_index];
       void* pkp = m->pkpool[run.kv_index];
       void* pvp = lc.v_is_k ? pkp : m->pvpool[run.kv_index];
       const int Ckk = lc.kv_heads * lc.dim;
       AttnExtra ex{lc.softcap, lc.sink ? l.w[DN_SQ_SINK] : nullptr, lc.out_gate ? (const float*)m->pa : nullptr, lc.mask_kind == DN_MASK_WINDOW ? 1 : 0,
-                   lc.v_is_k ? Ckk : 0, lc.pool, pkp, pvp};
+                   lc.v_is_k ? Ckk : 0, lc.pool, pkp, pvp, lc.dist_bias ? l.w[DN_SQ_DIST1] : nullptr, lc.dist_bias ? l.w[DN_SQ_DIST2] : nullptr,
+                   lc.attn_weight == DN_ATTN_SIGMOID ? l.w[DN_SQ_ATTN_OFF] : nullptr};
       const size_t sm = ((size_t)l.Cq + l.Ck + 40 + lc.heads + lc.kv_heads + lc.rot_dims) * 4;
       PH(DN_SEQ_PH_ATTN_PREP);
       CK(launch(k_attn_prep<T>, dim3(N), dim3(256), sm, s, a, b, (const T*)m->uq, (const T*)m->uk, (const T*)m->uv, w(DN_SQ_Q_CONV),
-                w(DN_SQ_K_CONV), w(DN_SQ_V_CONV), w(DN_SQ_Q_NORM), w(DN_SQ_K_NORM), (const T*)cst, m->conv_stride, (T*)m->qb,
+                w(DN_SQ_K_CONV), w(DN_SQ_V_CONV), w(DN_SQ_Q_NORM), w(DN_SQ_K_NORM), cst, m->conv_stride, (T*)m->qb,
                 (T*)m->kpool[run.kv_index], (T*)m->vpool[run.kv_index]));
       if (lc.pool > 0)      // blocks that this step's tokens complete get their mean key and value
         CK(launch(k_pool_rows<T>, dim3(N), dim3(128), 0, s, b, lc.pool, Ckk, lc.v_is_k ? 0 : lc.kv_heads * lc.vdim, (const T*)m->kpool[run.kv_index], (const T*)vpl,
@@ -1059,8 +1098,10 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
         CK(attn_tiles(s, b, (const bf16*)m->qb, (const bf16*)m->kpool[run.kv_index], (const bf16*)vpl, lc, ex, (bf16*)m->mo));
       else {
         // a small step (decode): long rows are split over up to AT_MAX_SPLITS blocks, joined by k_attn_merge
-        const int Z = N <= AT_SPLIT_ROWS ? AT_MAX_SPLITS : 1;
-        CK(launch(k_attn<T, 8>, dim3(N, lc.heads, Z), dim3(AT_WARPS * 32), (size_t)(((lc.dim + 3) & ~3) + AT_WARPS * (2 + (lc.vdim + 31) / 32 * 32)) * 4, s, b,
+        // (a mask of `chunk` positions bounds the keys of a row, and with them its splits)
+        const int zcap = lc.chunk > 0 && lc.pool == 0 ? std::min((int)AT_MAX_SPLITS, (lc.chunk + AT_SPLIT_KEYS - 1) / AT_SPLIT_KEYS) : AT_MAX_SPLITS;
+        const int Z = N <= AT_SPLIT_ROWS ? zcap : 1;
+        CK(launch(ex.off ? k_attn<T, 8, true> : k_attn<T, 8, false>, dim3(N, lc.heads, Z), dim3(AT_WARPS * 32), (size_t)(((lc.dim + 3) & ~3) + AT_WARPS * (2 + (lc.vdim + 31) / 32 * 32)) * 4, s, b,
                   (const T*)m->qb, (const T*)m->kpool[run.kv_index],
                   (const T*)vpl, lc.heads, lc.kv_heads, lc.dim, lc.vdim, lc.chunk, lc.scale, ex, (T*)m->mo, m->attn_part));
         if (Z > 1) CK(launch(k_attn_merge<T>, dim3(N, lc.heads), dim3(128), 0, s, b, lc.heads, lc.vdim, lc.chunk, Z, ex, (const float*)m->attn_part, (T*)m->mo));
@@ -1184,13 +1225,41 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
       CK(launch(k_delta_out<T>, dim3(N, lc.heads), dim3(32), 0, s, (const float*)m->od, (const T*)m->gt, w(DN_SQ_OUT_NORM), lc.heads, lc.vdim,
                 c.eps, (T*)m->mo, lc.vdim, 0));
     }
-    if (lc.conv > 1) {
+    if (lc.conv > 1 && !(b.max_len == 1 && (lc.mixer == DN_MIX_ATTENTION || lc.mixer == DN_MIX_PARALLEL))) {      // (those carry in k_attn_prep)
       PH(DN_SEQ_PH_CARRY);
       CarrySrc<T> cs{{(const T*)m->uq, (const T*)m->uk, (const T*)m->uv}, {l.Cq, l.Ck, l.Cv}};
       CK(launch(k_conv_carry<T>, dim3((std::max(l.Cq, std::max(l.Ck, l.Cv)) + 127) / 128, b.E, 3), dim3(128), 0, s, cs, lc.conv, b, cst, m->conv_stride));
     }
     PH(DN_SEQ_PH_OUT_PROJ);
-    CK(linear<T>(m, s, (const T*)m->mo, l.w[DN_SQ_O], nullptr, m->y, N, W, l.Co, true, 0, LinMaps{wm(DN_SQ_O), nullptr, &l.x_mo}));
+    if (ride) {
+      memset(&sg, 0, sizeof(sg));
+      add(m->mo, DN_SQ_O, m->y, W, 1, ACT_NONE, l.Co); add(m->act, DN_SQ_DOWN, m->y2, W, 1, ACT_NONE, lc.ff);
+      CK(run_segs());
+    } else
+      CK(linear<T>(m, s, (const T*)m->mo, l.w[DN_SQ_O], nullptr, m->y, N, W, l.Co, true, 0, LinMaps{wm(DN_SQ_O), nullptr, &l.x_mo}));
+    if (c.parallel_ff) {      // the feed-forward on the same normed input; both outputs join together, and the next run's norm with them
+      const float* ffy = nullptr;
+      MoeSrc<T> ms = no_moe;
+      if (lc.ff > 0 && lc.mlp_kind == DN_MLP_MOE) {
+        const int rc = moe_ff<T>(m, l, N, false, no_next, s, false);
+        if (rc != DN_OK) return rc;
+        ms = MoeSrc<T>{m->eo, m->rwt, m->rpos, m->ridx, lc.top, lc.router_kind == DN_ROUTER_SCORED ? lc.experts : INT32_MAX, (const T*)m->h,
+                       lc.shared_ff > 0 ? (const float*)m->y2 : (const float*)nullptr, lc.shared_gate ? (const float*)m->sgate : (const float*)nullptr};
+      } else if (lc.ff > 0) {
+        if (!ride) { const int rc = dense_ff(l, N, m->y2); if (rc != DN_OK) return rc; }
+        ffy = m->y2;
+      }
+      PH(DN_SEQ_PH_WRITE_BACK);
+      const bool fuse = !lnorm && ri + 1 < (int)m->runs.size() && !m->runs[ri + 1].inject;
+      const T* nw = fuse ? (const T*)m->L[m->runs[ri + 1].layer].w[DN_SQ_NORM1] : (const T*)nullptr;
+      T* hout = fuse ? (T*)m->h : (T*)nullptr;
+      if (W % 4 == 0) CK(launch(k_parallel_join<T, 4>, dim3(N), nthr, nsm, s, m->xs, W, rmul, (const float*)m->y, ffy, ms, nw, wmode, c.eps, hout));
+      else CK(launch(k_parallel_join<T, 1>, dim3(N), nthr, nsm, s, m->xs, W, rmul, (const float*)m->y, ffy, ms, nw, wmode, c.eps, hout));
+      h_ready = fuse;
+      PH(DN_SEQ_PH_OTHER);
+      if (trace) CK(launch(k_stream_sum, dim3(ew), dim3(256), 0, s, (const float*)m->xs, N, W, S1, trace + (size_t)ri * N * W));
+      continue;
+    }
     if (lc.mixer == DN_MIX_PARALLEL && lc.r_kind == DN_RIGHT_GDELTA) {     // the generalized delta rule, on the same input
       PH(DN_SEQ_PH_PROJ);
       if (few) {
@@ -1247,7 +1316,7 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
                 c.eps, (T*)m->mo, lc.r_dim, 1));
       PH(DN_SEQ_PH_OUT_PROJ);
       CK(linear<T>(m, s, (const T*)m->mo, l.w[DN_SQ_R_O], nullptr, m->y2, N, W, l.Rv, true, 0, LinMaps{wm(DN_SQ_R_O), nullptr, &l.x_mo_r}));
-      ja = lc.left_scale; jb = lc.right_scale; jy2 = m->y2;
+      ja = rmul * lc.left_scale; jb = rmul * lc.right_scale; jy2 = m->y2;
     } else if (lc.mixer == DN_MIX_PARALLEL) {     // the linear-attention half, on the same input; its scratch is free again
       PH(DN_SEQ_PH_PROJ);
       if (few) {
@@ -1273,7 +1342,7 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
                 c.eps, (T*)m->mo, 0, 0));
       PH(DN_SEQ_PH_OUT_PROJ);
       CK(linear<T>(m, s, (const T*)m->mo, l.w[DN_SQ_R_O], nullptr, m->y2, N, W, l.Rv, true, 0, LinMaps{wm(DN_SQ_R_O), nullptr, &l.x_mo_r}));
-      ja = lc.left_scale; jb = lc.right_scale; jy2 = m->y2;
+      ja = rmul * lc.left_scale; jb = rmul * lc.right_scale; jy2 = m->y2;
     }
     PH(DN_SEQ_PH_WRITE_BACK);
     const NextNorm<T> nx_mix = lc.ff > 0 ? (can_fuse_next ? next_norm(l, DN_SQ_NORM2) : no_next) : nx_run;
@@ -1299,19 +1368,13 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
           const MoeSrc<T> ms{m->eo, m->rwt, m->rpos, m->ridx, lc.top, scored ? lc.experts : INT32_MAX, (const T*)m->h,
                              lc.shared_ff > 0 ? (const float*)m->y2 : (const float*)nullptr, lc.shared_gate ? (const float*)m->sgate : (const float*)nullptr};
           CK(join(l, DN_SQ_POST2, DN_SQ_HC2_MIX, DN_SQ_HC2_OUT, 1.f, nullptr, 0.f, no_next, &ms));
-        } else if (!fused) CK(join(l, DN_SQ_POST2, DN_SQ_HC2_MIX, DN_SQ_HC2_OUT, 1.f, lc.shared_ff > 0 ? (const float*)m->y2 : nullptr, 1.f, nx_run));
+        } else if (!fused) CK(join(l, DN_SQ_POST2, DN_SQ_HC2_MIX, DN_SQ_HC2_OUT, rmul, lc.shared_ff > 0 ? (const float*)m->y2 : nullptr, rmul, nx_run));
         h_ready = nx_run.alpha != nullptr || !pre;
       } else {
-        PH(DN_SEQ_PH_FF_UP);
-        if (lc.ff_act == DN_FF_RELU2)      // no gate: relu(W_up h + b)^2
-          CK(linear<T>(m, s, (const T*)m->h, l.w[DN_SQ_UP], nullptr, m->act, N, lc.ff, W, false, ACT_RELU2, LinMaps{wm(DN_SQ_UP), nullptr, &m->x_h}, 0.f, l.w[DN_SQ_UP_B]));
-        else
-          CK(linear<T>(m, s, (const T*)m->h, l.w[DN_SQ_GATE], l.w[DN_SQ_UP], m->act, N, lc.ff, W, false, ACT_GEGLU, LinMaps{wm(DN_SQ_GATE), wm(DN_SQ_UP), &m->x_h}));
-        PH(DN_SEQ_PH_FF_DOWN);
-        CK(linear<T>(m, s, (const T*)m->act, l.w[DN_SQ_DOWN], nullptr, m->y, N, W, lc.ff, true, 0, LinMaps{wm(DN_SQ_DOWN), nullptr, &l.x_act}, 0.f,
-                     lc.ff_act == DN_FF_RELU2 ? l.w[DN_SQ_DOWN_B] : nullptr));
+        const int rc = dense_ff(l, N, m->y);
+        if (rc != DN_OK) return rc;
         PH(DN_SEQ_PH_WRITE_BACK);
-        CK(join(l, DN_SQ_POST2, DN_SQ_HC2_MIX, DN_SQ_HC2_OUT, 1.f, nullptr, 0.f, nx_run));
+        CK(join(l, DN_SQ_POST2, DN_SQ_HC2_MIX, DN_SQ_HC2_OUT, rmul, nullptr, 0.f, nx_run));
         h_ready = (nx_run.alpha != nullptr && c.post_norm && S <= 0) || !pre;
       }
     }
@@ -1320,7 +1383,7 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
   }
   if (n_want > 0) {
     PH(DN_SEQ_PH_NORM);
-    CK(launch(k_read_norm<T>, dim3(n_want), nthr, nsm, s, m->xs, N, W, S, (const T*)nullptr, (const T*)m->final_norm, dyt ? 0 : 1, 1, c.eps, want_dev, (T*)m->h,
+    CK(launch(k_read_norm<T>, dim3(n_want), nthr, nsm, s, m->xs, N, W, S, (const T*)nullptr, (const T*)m->final_norm, wmode, 1, c.eps, want_dev, (T*)m->h,
               mwp(DN_SQ_FINAL_NORM_B), dyt ? mwp(DN_SQ_FINAL_NORM_ALPHA) : (const T*)nullptr, lnorm, (const T*)nullptr, 0, (const int32_t*)nullptr, (T*)nullptr,
               (size_t)0));
     PH(DN_SEQ_PH_HEAD);
@@ -1349,6 +1412,8 @@ extern "C" int dn_seq_step(dn_seq_model* m, int E, const int32_t* slots, const i
     if (counts[e] <= 0) return fail(DN_EINVAL, "entry %d brings no tokens", e);
     N += counts[e];
     const size_t pages = ((size_t)m->length[sl] + counts[e] + PAGE - 1) / PAGE;
+    if (m->cfg.max_positions > 0 && (int64_t)m->length[sl] + counts[e] > m->cfg.max_positions)
+      return fail(DN_EINVAL, "entry %d: the sequence would hold %lld tokens, the model has %d positions", e, (long long)m->length[sl] + counts[e], m->cfg.max_positions);
     if (pages > (size_t)m->max_pages) return fail(DN_ENOSPC, "sequence too long for the block table");
     if (pages > m->pages[sl].size()) need += pages - m->pages[sl].size();
   }
@@ -1364,6 +1429,7 @@ extern "C" int dn_seq_step(dn_seq_model* m, int E, const int32_t* slots, const i
   if (m->cfg.embed_norm && (!mhas(DN_SQ_EMBED_NORM) || !mhas(DN_SQ_EMBED_NORM_B) || !mhas(DN_SQ_EMBED_NORM_ALPHA))) return fail(DN_ENOENT, "the embedding's norm is not bound");
   if (m->cfg.loop_times > 0 && !mhas(DN_SQ_LOOP_IN)) return fail(DN_ENOENT, "the loop's input matrix is not bound");
   if (m->cfg.norm_kind == DN_NORM_LAYER && !mhas(DN_SQ_FINAL_NORM_B)) return fail(DN_ENOENT, "the final norm's bias is not bound");
+  if (m->cfg.max_positions > 0 && !mhas(DN_SQ_POS)) return fail(DN_ENOENT, "the position table is not bound");
   if (m->cfg.bigram_buckets > 0 && !mhas(DN_SQ_BIGRAM)) return fail(DN_ENOENT, "the bigram table is not bound");
   for (int i = 0; i < m->cfg.n_layers; i++) {
     const SeqLayer& l = m->L[i];
@@ -1371,12 +1437,13 @@ extern "C" int dn_seq_step(dn_seq_model* m, int E, const int32_t* slots, const i
     const int mx = l.c.mixer;
     const bool moe = l.c.mlp_kind == DN_MLP_MOE;
     bool ok = has(DN_SQ_Q) && has(DN_SQ_O);
-    if (!m->cfg.no_pre_norm) ok = ok && has(DN_SQ_NORM1) && (l.c.ff == 0 || has(DN_SQ_NORM2));
+    if (!m->cfg.no_pre_norm) ok = ok && has(DN_SQ_NORM1) && (l.c.ff == 0 || m->cfg.parallel_ff || has(DN_SQ_NORM2));
     if (l.c.ff > 0 && !moe) ok = ok && (l.c.ff_act == DN_FF_RELU2 || has(DN_SQ_GATE)) && has(DN_SQ_UP) && has(DN_SQ_DOWN);
     if (l.c.ff > 0 && moe) {
-      ok = ok && has(DN_SQ_ROUTER) && (l.c.shared_ff == 0 || (has(DN_SQ_SH_GATE) && has(DN_SQ_SH_UP) && has(DN_SQ_SH_DOWN)));
+      const bool gated = l.c.expert_act != DN_EXPERT_RELU2;
+      ok = ok && has(DN_SQ_ROUTER) && (l.c.shared_ff == 0 || ((!gated || has(DN_SQ_SH_GATE)) && has(DN_SQ_SH_UP) && has(DN_SQ_SH_DOWN)));
       if (l.c.shared_gate) ok = ok && has(DN_SQ_SH_SG);
-      for (const void* p : l.etab_h) ok = ok && p != nullptr;
+      for (size_t k = gated ? 0 : l.c.experts; k < l.etab_h.size(); k++) ok = ok && l.etab_h[k] != nullptr;
     }
     if (dyt) ok = ok && has(DN_SQ_NORM1_B) && has(DN_SQ_NORM1_ALPHA) && (l.c.ff == 0 || (has(DN_SQ_NORM2_B) && has(DN_SQ_NORM2_ALPHA)));
     if (m->cfg.post_norm) ok = ok && has(DN_SQ_POST1) && (l.c.ff == 0 || has(DN_SQ_POST2));
@@ -1384,12 +1451,14 @@ extern "C" int dn_seq_step(dn_seq_model* m, int E, const int32_t* slots, const i
     if (mx == DN_MIX_LATENT) ok = ok && has(DN_SQ_DKV) && has(DN_SQ_DKV_NORM) && has(DN_SQ_UK) && has(DN_SQ_UV) && (!l.c.out_gate || has(DN_SQ_HEAD_GATE)) &&
                                   (l.c.q_rank == 0 || (has(DN_SQ_DQ) && has(DN_SQ_DQ_NORM)));
     else if (l.Ck) ok = ok && has(DN_SQ_K) && (l.c.v_is_k || has(DN_SQ_V));
-    if (m->cfg.norm_kind == DN_NORM_LAYER) ok = ok && has(DN_SQ_NORM1_B) && (l.c.ff == 0 || has(DN_SQ_NORM2_B));
+    if (m->cfg.norm_kind == DN_NORM_LAYER) ok = ok && has(DN_SQ_NORM1_B) && (l.c.ff == 0 || m->cfg.parallel_ff || has(DN_SQ_NORM2_B));
     if (m->cfg.canon_taps > 0) ok = ok && has(DN_SQ_CANON1) && (l.c.ff == 0 || has(DN_SQ_CANON2));
     if (l.c.conv > 0) ok = ok && has(DN_SQ_Q_CONV) && (!l.Ck || (has(DN_SQ_K_CONV) && has(DN_SQ_V_CONV)));
     if (mx == DN_MIX_ATTENTION || mx == DN_MIX_PARALLEL) {
       if (l.c.qk_norm) ok = ok && has(DN_SQ_Q_NORM) && (!l.Ck || has(DN_SQ_K_NORM));
       if (l.c.sink) ok = ok && has(DN_SQ_SINK);
+      if (l.c.dist_bias) ok = ok && has(DN_SQ_DIST1) && has(DN_SQ_DIST2);
+      if (l.c.attn_weight == DN_ATTN_SIGMOID) ok = ok && has(DN_SQ_ATTN_OFF);
       if (l.c.out_gate) ok = ok && has(DN_SQ_HEAD_GATE);
     }
     if (mx == DN_MIX_DELTA) ok = ok && has(DN_SQ_A) && has(DN_SQ_B) && has(DN_SQ_G) && has(DN_SQ_A_LOG) && has(DN_SQ_DT_BIAS) && has(DN_SQ_OUT_NORM);

@@ -26,6 +26,9 @@
 //     interpolation; a query scale that grows with the logarithm of the position; values that are the keys
 //   * a sliding window followed by mean-pooled blocks of the tokens that have left it (one softmax over both)
 //   * (dn_seq_gdelta.cuh) generalized delta rule with a decay and a removal rate per key channel
+//   * a learned position row added to the embedding; RMS norm with one number for all coordinates; mixer and feed-forward
+//     side by side on one normed input, joined with a factor and the next layer's norm in one pass
+//   * attention without a softmax: sigmoid weights with an offset per head; scores that fall with the logarithm of the distance
 // T is the storage type of weights and activations (bf16 or float); sums, norms, scores, positions, gates and
 // states are fp32 in both.
 #pragma once
@@ -125,6 +128,12 @@ __device__ __forceinline__ void kahan_add(float& sum, float& c, float v) {
   c = __fsub_rn(__fsub_rn(t, sum), y);
   sum = t;
 }
+// weight of column c in an RMS norm: w[c], 1 + w[c] or, one number for all columns, w[0]
+constexpr int NW_PLAIN = 0, NW_ONE_PLUS = 1, NW_SCALAR = 2;
+template <class T>
+__device__ __forceinline__ float norm_weight(const T* __restrict__ w, int c, int mode) {
+  return mode == NW_SCALAR ? ldf(w) : ldf(w + c) + (mode == NW_ONE_PLUS ? 1.f : 0.f);
+}
 // dynamic tanh: tanh(alpha x) w + b
 template <class T>
 __device__ __forceinline__ float dyt_f(float x, float alpha, const T* __restrict__ w, const T* __restrict__ b, int c) {
@@ -153,14 +162,16 @@ struct Batch {
 template <class T>
 __global__ void k_embed(const T* __restrict__ embed, Batch b, float scale, int W, int S1, float* __restrict__ xs, const T* __restrict__ nw,
                         const T* __restrict__ nb, const T* __restrict__ nalpha, float* __restrict__ x0, T* __restrict__ hout,
-                        const T* __restrict__ bigram) {
+                        const T* __restrict__ bigram, const T* __restrict__ ptab) {
   const int n = blockIdx.x;
   const size_t row = (size_t)b.tok[n] * W;
   const float alpha = nalpha ? ldf(nalpha) : 0.f;
   const T* brow = bigram ? bigram + (size_t)b.brow[n] * W : nullptr;
+  const T* prow = ptab ? ptab + (size_t)b.pos[n] * W : nullptr;      // learned position row
   for (int c = threadIdx.x; c < W; c += blockDim.x) {
     float v = ldf(embed + row + c) * scale;
     if (brow) v += ldf(brow + c);      // the hashed (previous token, token) row, summed in fp32
+    if (prow) v += ldf(prow + c);
     if (nalpha) v = dyt_f(v, alpha, nw, nb, c);
     for (int s = 0; s < S1; s++) xs[((size_t)s * b.N + n) * W + c] = v;
     if (x0) x0[(size_t)n * W + c] = v;
@@ -204,12 +215,12 @@ __device__ __forceinline__ void canon_tail(const float* __restrict__ u, const T*
   }
 }
 
-// stream read-out (u = sum_s in[s] x_s, or x_0) + RMS norm with weight (1 + w) or w; rows[] optionally gathers.
+// stream read-out (u = sum_s in[s] x_s, or x_0) + RMS norm with weight (1 + w), w or a scalar (NW_*); rows[] optionally gathers.
 // 16-byte loads of the streams when the width allows; a thread's partial sum of squares runs over its own columns in
 // ascending order and the block adds the partials by index, so the result depends on W and the block size only.
 template <class T>
 __global__ void k_read_norm(const float* __restrict__ xs, int N, int W, int S, const T* __restrict__ hc_in, const T* __restrict__ nw,
-                            int one_plus, int sum_all, float eps, const int32_t* __restrict__ rows, T* __restrict__ h,
+                            int wmode, int sum_all, float eps, const int32_t* __restrict__ rows, T* __restrict__ h,
                             const T* __restrict__ nb, const T* __restrict__ nalpha, int layer_norm,
                             const T* __restrict__ cw = nullptr, int taps = 0, const int32_t* __restrict__ slot_of = nullptr,
                             T* __restrict__ cstate = nullptr, size_t slot_stride = 0) {
@@ -263,7 +274,7 @@ __global__ void k_read_norm(const float* __restrict__ xs, int N, int W, int S, c
     ss = block_sum(ss, red);
     const float rinv = 1.f / sqrtf(ss / (float)W + eps);
     for (int c = threadIdx.x; c < W; c += blockDim.x) {
-      const float g = ldf(nw + c) + (one_plus ? 1.f : 0.f);
+      const float g = norm_weight(nw, c, wmode);
       if (cw) u[c] = round_to<T>(u[c] * rinv * g);
       else stf(h + (size_t)r * W + c, u[c] * rinv * g);
     }
@@ -447,6 +458,65 @@ __global__ void k_rms_join(float* __restrict__ x, int W, const float* __restrict
     x[base + c] = xn;
     if (hout) stf(hout + base + c, xn);
   }
+}
+
+// Mixer and feed-forward of one layer, both fed by the same normed input, join the plain residual together, and the next
+// layer's norm is formed in the same pass:
+//   u = y + y2 + sum_j wt[j] (expert output j | the input, for an identity expert) + gate sh        (all but y optional)
+//   x <- x + m u;   h <- RMS norm of x with the next layer's weight (hout null: no norm follows)
+// One block per token, VEC columns a thread; partial sums of squares in the fixed order of k_read_norm.
+template <class T, int VEC>
+__global__ void k_parallel_join(float* __restrict__ x, int W, float m, const float* __restrict__ y, const float* __restrict__ y2, MoeSrc<T> ms,
+                                const T* __restrict__ nw, int wmode, float eps, T* __restrict__ hout) {
+  extern __shared__ __align__(16) float sm[];
+  float* v = sm;            // [W]
+  float* red = sm + W;      // [33]
+  const size_t n = blockIdx.x, base = n * W;
+  auto ld = [](const float* p, float (&o)[VEC]) {
+    if (VEC == 4) *reinterpret_cast<float4*>(o) = *reinterpret_cast<const float4*>(p);
+    else o[0] = p[0];
+  };
+  float ss = 0.f;
+  for (int c = threadIdx.x * VEC; c < W; c += blockDim.x * VEC) {
+    float u[VEC], t[VEC], xv[VEC];
+    ld(y + base + c, u);
+    ld(x + base + c, xv);
+    if (y2) {
+      ld(y2 + base + c, t);
+#pragma unroll
+      for (int i = 0; i < VEC; i++) u[i] += t[i];
+    }
+    if (ms.eo) {
+      for (int j = 0; j < ms.top; j++) {
+        const float wj = ms.wt[n * ms.top + j];
+        if (ms.idx[n * ms.top + j] < ms.E) ld(ms.eo + (size_t)ms.pos[n * ms.top + j] * W + c, t);
+        else {
+#pragma unroll
+          for (int i = 0; i < VEC; i++) t[i] = ldf(ms.hid + base + c + i);
+        }
+#pragma unroll
+        for (int i = 0; i < VEC; i++) u[i] = fmaf(wj, t[i], u[i]);
+      }
+    }
+    if (ms.sh) {
+      const float gs = ms.sgate ? ms.sgate[n] : 1.f;
+      ld(ms.sh + base + c, t);
+#pragma unroll
+      for (int i = 0; i < VEC; i++) u[i] = fmaf(gs, t[i], u[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < VEC; i++) {
+      xv[i] += m * u[i];
+      v[c + i] = xv[i];
+      ss += xv[i] * xv[i];
+    }
+    if (VEC == 4) *reinterpret_cast<float4*>(x + base + c) = *reinterpret_cast<float4*>(xv);
+    else x[base + c] = xv[0];
+  }
+  if (!hout) return;
+  ss = block_sum(ss, red);
+  const float rinv = 1.f / sqrtf(ss / (float)W + eps);
+  for (int c = threadIdx.x; c < W; c += blockDim.x) stf(hout + base + c, v[c] * rinv * norm_weight(nw, c, wmode));
 }
 
 // The two halves of a parallel mixer join the plain residual, each through an RMS norm of its own over the width:
@@ -648,7 +718,8 @@ struct LinSegs {
   void* Y[MAX_SEGS];
   int O[MAX_SEGS];
   int out32[MAX_SEGS];
-  int act[MAX_SEGS];         // ACT_NONE or ACT_TANH
+  int act[MAX_SEGS];         // ACT_NONE or a one-operand activation
+  int K[MAX_SEGS];           // 0: the launch's common K
   int n;
 };
 template <class T>
@@ -662,7 +733,8 @@ __global__ void __launch_bounds__(256) k_linear_rows_multi(const T* __restrict__
   if (i >= sg.n) return;
   const int o = blk * 8 + (threadIdx.x >> 5);
   if (o >= sg.O[i]) return;
-  linear_row<T>(sg.X[i] ? (const T*)sg.X[i] : X, (const T*)sg.W[i], (const T*)nullptr, sg.Y[i], sg.out32[i] != 0, N, sg.O[i], K, sg.act[i], o);
+  linear_row<T>(sg.X[i] ? (const T*)sg.X[i] : X, (const T*)sg.W[i], (const T*)nullptr, sg.Y[i], sg.out32[i] != 0, N, sg.O[i], sg.K[i] > 0 ? sg.K[i] : K,
+                sg.act[i], o);
 }
 
 // ---------------------------------------------------------------------------------------------------------------
@@ -680,6 +752,20 @@ __device__ __forceinline__ float conv_at(const T* __restrict__ U, int ldu, const
   float a = 0.f;
   for (int j = 0; j < taps; j++) a += ldf(cw + (size_t)c * taps + j) * conv_in(U, ldu, c, n, local, taps - 1 - j, st, ldst, taps);
   return a;
+}
+
+// the same for the only token of its entry (every older input is a carried one), which then takes its place among them
+template <class T>
+__device__ __forceinline__ float conv_carry_at(const T* __restrict__ U, int ldu, const T* __restrict__ cw, int c, int n, T* __restrict__ st, int ldst, int taps) {
+  float a = 0.f;
+  for (int j = 0; j + 1 < taps; j++) {
+    const float x = ldf(st + (size_t)j * ldst + c);
+    a += ldf(cw + (size_t)c * taps + j) * x;
+    if (j > 0) stf(st + (size_t)(j - 1) * ldst + c, x);
+  }
+  const float x = ldf(U + (size_t)n * ldu + c);
+  if (taps > 1) stf(st + (size_t)(taps - 2) * ldst + c, x);
+  return a + ldf(cw + (size_t)c * taps + taps - 1) * x;
 }
 
 // after a step: the last taps-1 inputs of every entry become its slot's carried inputs; blockIdx.z picks the
@@ -768,6 +854,7 @@ struct AttnPrep {
   int half;                          // 1: rotary pairs (i, i + rot / 2), else (2i, 2i + 1)
   float mscale;                      // cos and sin are multiplied by this
   float qt_coef; int qt_every;       // q times 1 + qt_coef ln(floor((p + 1) / qt_every) + 1) (qt_every 0: no)
+  int carry;                         // 1: every entry brings one token, and the kernel carries its inputs itself (no k_conv_carry)
 };
 
 // attention mixer, between the projections and the scores: conv -> RMS norm (over the whole q / k projection or per
@@ -776,7 +863,7 @@ struct AttnPrep {
 template <class T>
 __global__ void k_attn_prep(AttnPrep a, Batch b, const T* __restrict__ Uq, const T* __restrict__ Uk, const T* __restrict__ Uv,
                             const T* __restrict__ cwq, const T* __restrict__ cwk, const T* __restrict__ cwv, const T* __restrict__ nq,
-                            const T* __restrict__ nk, const T* __restrict__ cstate, size_t slot_stride, T* __restrict__ qout,
+                            const T* __restrict__ nk, T* __restrict__ cstate, size_t slot_stride, T* __restrict__ qout,
                             T* __restrict__ kpool, T* __restrict__ vpool) {
   extern __shared__ float sm[];
   // a layer that borrows its keys and values projects and carries q only
@@ -790,17 +877,20 @@ __global__ void k_attn_prep(AttnPrep a, Batch b, const T* __restrict__ Uq, const
   float* snt = cst + a.rot / 2;
   const int n = blockIdx.x, slot = b.slot[n], p = b.pos[n];
   const int local = n - b.first[n];   // rows of this step that precede the token in its sequence
-  const T* st = cstate + (size_t)slot * slot_stride;
+  T* st = cstate + (size_t)slot * slot_stride;
+  auto conv = [&](const T* U, int ldu, const T* cw, int c, int off) {
+    return a.carry ? conv_carry_at(U, ldu, cw, c, n, st + off, ldst, a.taps) : conv_at(U, ldu, cw, c, n, local, st + off, ldst, a.taps);
+  };
   float sq = 0.f, sk = 0.f;
   for (int c = threadIdx.x; c < Cq; c += blockDim.x) {
-    const float v = conv_at(Uq, Cq, cwq, c, n, local, st, ldst, a.taps);
+    const float v = conv(Uq, Cq, cwq, c, 0);
     qs[c] = v;
     sq += v * v;
   }
   sq = block_sum(sq, red);
   if (a.own_kv) {
     for (int c = threadIdx.x; c < Ck; c += blockDim.x) {
-      const float v = conv_at(Uk, Ck, cwk, c, n, local, st + Cq, ldst, a.taps);
+      const float v = conv(Uk, Ck, cwk, c, Cq);
       ks[c] = v;
       sk += v * v;
     }
@@ -868,7 +958,7 @@ __global__ void k_attn_prep(AttnPrep a, Batch b, const T* __restrict__ Uq, const
   if (Cv > 0) {
     T* vr = vpool + ((size_t)page * PAGE + prow) * Cv;
     for (int c = threadIdx.x; c < Cv; c += blockDim.x)
-      stf(vr + c, conv_at(Uv, Cv, cwv, c, n, local, st + Cq + Ck, ldst, a.taps));
+      stf(vr + c, conv(Uv, Cv, cwv, c, Cq + Ck));
   }
 }
 
@@ -920,6 +1010,9 @@ struct AttnExtra {
   int pool;        // > 0 (with window): blocks of this many tokens wholly before the window are seen as one mean key / value each
   const void* pk;  // their pools [pages][pool_rows(pool)][row], strides as the token pools'
   const void* pv;
+  const void* r1;  // [H] with r2: r1_h ln(1 + r2_h (p - j)) is taken off the score (after scale and cap) of the key at j (null: no)
+  const void* r2;
+  const void* off; // [H] sigmoid weights: added to the score inside the sigmoid
 };
 // keys a query at p sees: the pooled blocks first (virtual indices 0 .. nb - 1), then the tokens lo .. p
 __device__ __forceinline__ int attn_pooled(int p, int chunk, const AttnExtra& ex) { return ex.pool > 0 ? pooled_seen(p, chunk, ex.pool) : 0; }
@@ -958,7 +1051,8 @@ __device__ __forceinline__ void ld_vals(float (&v)[8], const T* p, int cnt, bool
 #pragma unroll
   for (int i = 0; i < 8; i++) if (i < cnt) v[i] = ldf(p + i);
 }
-template <class T, int MAXV>      // MAXV: value dims a lane owns at most (8: dv <= 256, 16: dv <= 512)
+// SIG: a key's weight is sigmoid(score + off_h) and nothing is divided by a sum; running maximum and sum do not exist, partials add
+template <class T, int MAXV, bool SIG = false>      // MAXV: value dims a lane owns at most (8: dv <= 256, 16: dv <= 512)
 __global__ void __launch_bounds__(AT_WARPS * 32) k_attn(Batch b, const T* __restrict__ q, const T* __restrict__ kpool,
                                                         const T* __restrict__ vpool, int H, int G, int dk, int dv, int chunk, float scale,
                                                         AttnExtra ex, T* __restrict__ out, float* __restrict__ part_g) {
@@ -996,6 +1090,8 @@ __global__ void __launch_bounds__(AT_WARPS * 32) k_attn(Batch b, const T* __rest
   };
   const T* kpl = (const T*)ex.pk;
   const T* vpl = (const T*)ex.pv;
+  const float r1 = ex.r1 ? ldf((const T*)ex.r1 + h) : 0.f, r2 = ex.r1 ? ldf((const T*)ex.r2 + h) : 0.f;
+  const float soff = SIG ? ldf((const T*)ex.off + h) : 0.f;
   for (int j0 = (z * AT_WARPS + warp) * 32; j0 < nkeys; j0 += nz * AT_WARPS * 32) {
     const int j = j0 + lane;
     float s = -INFINITY;
@@ -1022,13 +1118,18 @@ __global__ void __launch_bounds__(AT_WARPS * 32) k_attn(Batch b, const T* __rest
       }
       s = d0 * scale;
       if (ex.softcap > 0.f) s = ex.softcap * tanhf(s / ex.softcap);
+      if (ex.r1) s -= r1 * log1pf(r2 * (float)(nkeys - 1 - j));      // (no pooled blocks here: the last key is the query's own)
     }
-    const float mn = fmaxf(m, warp_max(s));
-    const float corr = expf(m - mn);      // exp(-inf) = 0 on the warp's first tile
-    const float pj = j < nkeys ? expf(s - mn) : 0.f;
-    l = l * corr + warp_sum(pj);
+    float mn = 0.f, pj;
+    if (SIG) pj = j < nkeys ? sigmoid_f(s + soff) : 0.f;
+    else {
+      mn = fmaxf(m, warp_max(s));
+      const float corr = expf(m - mn);      // exp(-inf) = 0 on the warp's first tile
+      pj = j < nkeys ? expf(s - mn) : 0.f;
+      l = l * corr + warp_sum(pj);
 #pragma unroll
-    for (int i = 0; i < MAXV; i++) acc[i] *= corr;
+      for (int i = 0; i < MAXV; i++) acc[i] *= corr;
+    }
     const int cnt = min(32, nkeys - j0);
     if (vraw) {
       // a lane's run of values is one 4-, 8- or 16-byte load a row: the loads of eight rows are issued together, then
@@ -1086,6 +1187,13 @@ __global__ void __launch_bounds__(AT_WARPS * 32) k_attn(Batch b, const T* __rest
   const float og = ex.gate ? sigmoid_f(ex.gate[(size_t)n * H + h]) : 1.f;
   float* pg = split ? part_g + (((size_t)n * H + h) * gridDim.z + z) * (2 + dvp) : nullptr;
   for (int d = threadIdx.x; d < dv; d += blockDim.x) {
+    if (SIG) {
+      float a = 0.f;
+      for (int w = 0; w < AT_WARPS; w++) a += part[(size_t)w * (2 + dvp) + 2 + d];
+      if (split) pg[2 + d] = a;
+      else stf(out + ((size_t)n * H + h) * dv + d, a * og);
+      continue;
+    }
     float M = snk;
     for (int w = 0; w < AT_WARPS; w++) M = fmaxf(M, part[(size_t)w * (2 + dvp)]);
     float L = (ex.sink && !split) ? expf(snk - M) : 0.f, a = 0.f;
@@ -1105,6 +1213,7 @@ __global__ void __launch_bounds__(AT_WARPS * 32) k_attn(Batch b, const T* __rest
 template <class T>
 __global__ void k_attn_merge(Batch b, int H, int dv, int chunk, int zmax, AttnExtra ex, const float* __restrict__ part_g, T* __restrict__ out) {
   const int n = blockIdx.x, h = blockIdx.y, p = b.pos[n];
+  const bool sig = ex.off != nullptr;      // sigmoid weights: the partials add
   const int lo = attn_lo(p, chunk, ex.window);
   const int nz = attn_splits(attn_pooled(p, chunk, ex) + p - lo + 1, zmax);
   if (nz <= 1) return;
@@ -1113,8 +1222,15 @@ __global__ void k_attn_merge(Batch b, int H, int dv, int chunk, int zmax, AttnEx
   const float snk = ex.sink ? ldf((const T*)ex.sink + h) : -INFINITY;
   const float og = ex.gate ? sigmoid_f(ex.gate[(size_t)n * H + h]) : 1.f;
   float M = snk;
-  for (int z = 0; z < nz; z++) M = fmaxf(M, pg[(size_t)z * (2 + dvp)]);
+  if (!sig)
+    for (int z = 0; z < nz; z++) M = fmaxf(M, pg[(size_t)z * (2 + dvp)]);
   for (int d = threadIdx.x; d < dv; d += blockDim.x) {
+    if (sig) {
+      float a = 0.f;
+      for (int z = 0; z < nz; z++) a += pg[(size_t)z * (2 + dvp) + 2 + d];
+      stf(out + ((size_t)n * H + h) * dv + d, a * og);
+      continue;
+    }
     float L = ex.sink ? expf(snk - M) : 0.f, a = 0.f;
     for (int z = 0; z < nz; z++) {
       const float* pz = pg + (size_t)z * (2 + dvp);
@@ -1135,6 +1251,8 @@ __global__ void k_attn_merge(Batch b, int H, int dv, int chunk, int zmax, AttnEx
 // visited in ascending absolute position and a tile that the row does not see changes nothing, so a row's result
 // does not depend on how the prompt was cut or what else is in the batch.
 // DKP / DVP: head sizes rounded up to the template's; the padding is zero in shared memory.
+// A distance bias depends on p - key alone, of which a tile has 127 values: they are tabled in shared memory once a tile.
+// SIG: sigmoid weights (see k_attn): no running maximum, no sum; the head's offset rides in the table.
 __device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], const void* p) {
   const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
@@ -1178,7 +1296,7 @@ __device__ __forceinline__ void load_tile64_rows(bf16* __restrict__ dst, const b
 }
 
 constexpr int AT_ROWS = 64;      // query rows of a block, and keys of a tile (= PAGE)
-template <int DKP, int DVP>
+template <int DKP, int DVP, bool SIG = false>
 __global__ void __launch_bounds__(128) k_attn_tiles(Batch b, const bf16* __restrict__ q, const bf16* __restrict__ kpool,
                                                     const bf16* __restrict__ vpool, int H, int G, int dk, int dv, int chunk, float scale,
                                                     AttnExtra ex, bf16* __restrict__ out) {
@@ -1207,10 +1325,13 @@ __global__ void __launch_bounds__(128) k_attn_tiles(Batch b, const bf16* __restr
   load_tile64<LQ>(Qs, q + ((size_t)s0 * H + h) * dk, (size_t)H * dk, dk, rows);
   __syncthreads();
   // this thread's two rows of its warp's 16
-  const int r0 = warp * 16 + (lane >> 2), r1 = r0 + 8;
-  const int p0 = r0 < rows ? p_first + r0 : -1, p1 = r1 < rows ? p_first + r1 : -1;
+  const int r0 = warp * 16 + (lane >> 2), r1w = r0 + 8;
+  const int p0 = r0 < rows ? p_first + r0 : -1, p1 = r1w < rows ? p_first + r1w : -1;
   const int lo0 = p0 >= 0 ? attn_lo(p0, chunk, ex.window) : 0, lo1 = p1 >= 0 ? attn_lo(p1, chunk, ex.window) : 0;
   const bool warp_live = warp * 16 < rows;
+  __shared__ float tb[2 * AT_ROWS];      // tb[p - key - (p_first - j0 - 63)]: the bias (SIG: minus the offset) of the tile's distances
+  const float r1 = ex.r1 ? __bfloat162float(((const bf16*)ex.r1)[h]) : 0.f, r2 = ex.r1 ? __bfloat162float(((const bf16*)ex.r2)[h]) : 0.f;
+  const float soff = SIG ? __bfloat162float(((const bf16*)ex.off)[h]) : 0.f;
   uint32_t qf[DKP / 16][4];
 #pragma unroll
   for (int kk = 0; kk < DKP / 16; kk++) ldsm_x4(qf[kk], Qs + (warp * 16 + (lane & 15)) * LQ + kk * 16 + (lane >> 4) * 8);
@@ -1236,6 +1357,7 @@ __global__ void __launch_bounds__(128) k_attn_tiles(Batch b, const bf16* __restr
       const int kvalid = min(PAGE, p_last - j0 + 1);      // rows of the page beyond the last query's position are not read
       load_tile64<LQ>(Ks, kpool + prow * Ck + (size_t)g * dk, (size_t)Ck, dk, kvalid);
       if (!vk) load_tile64<LV>(Vs, vpool + prow * Cv + (size_t)g * dv, (size_t)Cv, dv, kvalid);
+      if (SIG || ex.r1) tb[threadIdx.x] = r1 * log1pf(r2 * (float)max(0, p_first - j0 - (AT_ROWS - 1) + (int)threadIdx.x)) - soff;
     }
     __syncthreads();
     if (!warp_live) continue;
@@ -1252,6 +1374,24 @@ __global__ void __launch_bounds__(128) k_attn_tiles(Batch b, const bf16* __restr
         mma_bf16(sc[2 * jj + 1], qf[kk], kf[2], kf[3]);
       }
     }
+    const bool biased = ex.r1 != nullptr && !pooled;
+    if (SIG) {
+      // weight 1 / (1 + 2^z), z = (bias - offset - score) log2(e); masked keys weigh 0.  ex2 and rcp of the special-function unit: a few
+      // units in the last place of fp32, far inside what the bf16 operands carry
+      constexpr float LOG2E_ = 1.4426950408889634f;
+#pragma unroll
+      for (int j = 0; j < 8; j++) {
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+          const int kc = j * 8 + (lane & 3) * 2 + (i & 1), key = j0 + kc;
+          float a = sc[j][i] * scale;
+          if (ex.softcap > 0.f) a = ex.softcap * tanhf(a / ex.softcap);
+          const float z = (tb[(i < 2 ? r0 : r1w) + (AT_ROWS - 1) - kc] - a) * LOG2E_;
+          const bool see = i < 2 ? (key <= p0 && key >= lo0) : (key <= p1 && key >= lo1);
+          sc[j][i] = see ? __fdividef(1.f, 1.f + exp2f(z)) : 0.f;
+        }
+      }
+    } else {
     // scale, mask, running maximum
     float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
@@ -1261,6 +1401,7 @@ __global__ void __launch_bounds__(128) k_attn_tiles(Batch b, const bf16* __restr
         const int key = j0 + j * 8 + (lane & 3) * 2 + i;
         float a0 = sc[j][i] * scale, a1 = sc[j][2 + i] * scale;
         if (ex.softcap > 0.f) { a0 = ex.softcap * tanhf(a0 / ex.softcap); a1 = ex.softcap * tanhf(a1 / ex.softcap); }
+        if (biased) { a0 -= tb[r0 + (AT_ROWS - 1) - (key - j0)]; a1 -= tb[r1w + (AT_ROWS - 1) - (key - j0)]; }
         sc[j][i] = (pooled ? key < nb0 : (key <= p0 && key >= lo0)) ? a0 : -INFINITY;
         sc[j][2 + i] = (pooled ? key < nb1 : (key <= p1 && key >= lo1)) ? a1 : -INFINITY;
         mx0 = fmaxf(mx0, sc[j][i]);
@@ -1289,6 +1430,7 @@ __global__ void __launch_bounds__(128) k_attn_tiles(Batch b, const bf16* __restr
     m0 = n0; m1 = n1;
 #pragma unroll
     for (int j = 0; j < DVP / 8; j++) { o[j][0] *= c0; o[j][1] *= c0; o[j][2] *= c1; o[j][3] *= c1; }
+    }
     // O += P V with P = hi + lo
 #pragma unroll
     for (int kk = 0; kk < 4; kk++) {       // 16 keys per step
@@ -1320,17 +1462,17 @@ __global__ void __launch_bounds__(128) k_attn_tiles(Batch b, const bf16* __restr
 #pragma unroll
     for (int j = 0; j < DVP / 8; j++) { o[j][0] *= c0; o[j][1] *= c0; o[j][2] *= c1; o[j][3] *= c1; }
   }
-  float i0 = p0 >= 0 ? 1.f / l0 : 0.f, i1 = p1 >= 0 ? 1.f / l1 : 0.f;
+  float i0 = p0 >= 0 ? (SIG ? 1.f : 1.f / l0) : 0.f, i1 = p1 >= 0 ? (SIG ? 1.f : 1.f / l1) : 0.f;
   if (ex.gate) {
     if (p0 >= 0) i0 *= sigmoid_f(ex.gate[(size_t)(s0 + r0) * H + h]);
-    if (p1 >= 0) i1 *= sigmoid_f(ex.gate[(size_t)(s0 + r1) * H + h]);
+    if (p1 >= 0) i1 *= sigmoid_f(ex.gate[(size_t)(s0 + r1w) * H + h]);
   }
 #pragma unroll
   for (int j = 0; j < DVP / 8; j++) {
     const int d = j * 8 + (lane & 3) * 2;
     if (d < dv) {
       if (p0 >= 0) *reinterpret_cast<uint32_t*>(out + ((size_t)(s0 + r0) * H + h) * dv + d) = pack_bf16(o[j][0] * i0, o[j][1] * i0);
-      if (p1 >= 0) *reinterpret_cast<uint32_t*>(out + ((size_t)(s0 + r1) * H + h) * dv + d) = pack_bf16(o[j][2] * i1, o[j][3] * i1);
+      if (p1 >= 0) *reinterpret_cast<uint32_t*>(out + ((size_t)(s0 + r1w) * H + h) * dv + d) = pack_bf16(o[j][2] * i1, o[j][3] * i1);
     }
   }
 }
@@ -1351,7 +1493,7 @@ __global__ void k_delta_prep(DeltaPrep a, Batch b, const T* __restrict__ Uq, con
   const int Cq = a.G * a.dk, Cv = a.H * a.dv, ldst = 2 * Cq + Cv;
   float* qs = sm;
   float* ks = sm + Cq;
-  const int n = blockIdx.x, slot = b.slot[n], p = b.pos[n];
+  const int n = blockIdx.x, slot = b.slot[n];
   const int local = n - b.first[n];
   const T* st = cstate + (size_t)slot * slot_stride;
   for (int c = threadIdx.x; c < Cq; c += blockDim.x) {

@@ -12,7 +12,8 @@
 // only, keeps the best groups of neighbouring experts, and weighs the chosen with their uncorrected scores divided by
 // their sum; its last outputs may stand for identity experts, which return the token's input and have no matrices:
 // the plan gives them no tiles, the row kernels skip them, and the combining kernels add the input itself.  Experts
-// are a clamped GLU or silu(gate) * up (`act`); a shared expert may be scaled by a sigmoid gate, one number a token.
+// are a clamped GLU, silu(gate) * up or, without a gate matrix, relu(up)^2 (`act`); a shared expert may be scaled by a sigmoid
+// gate, one number a token.  The scores may be a sigmoid of each logit instead of the softmax.
 #pragma once
 #include "dn_seq_kernels.cuh"
 
@@ -88,7 +89,7 @@ __device__ __forceinline__ float warp_dot(const T* __restrict__ x, const T* __re
   return warp_sum(a);
 }
 
-// Scored router, one block per token.  Et = real + identity experts.  Logits fp32; s = softmax over all Et; choice score
+// Scored router, one block per token.  Et = real + identity experts.  Logits fp32; s = softmax over all Et, or sigmoid of each; choice score
 // c = s + corr; with groups > 0 the Et experts form `groups` equal runs, a run's score is its largest c, and only experts
 // of the `keep` best runs can be chosen (ties: the lower index, for runs and experts alike); the `top` largest c choose;
 // weights = s[chosen] / (their sum + 1e-20) * scale.  sg (optional): one more row, sgate[n] = sigmoid(sg . h).
@@ -96,7 +97,7 @@ template <class T>
 __global__ void __launch_bounds__(1024) k_router_scored(const T* __restrict__ h, const T* __restrict__ Wr, const T* __restrict__ corr, int W, int Et,
                                                        int top, int groups, int keep, float scale, const T* __restrict__ sg,
                                                        int32_t* __restrict__ idx, float* __restrict__ wt, int32_t* __restrict__ pos,
-                                                       float* __restrict__ sgate) {
+                                                       float* __restrict__ sgate, int score_sigmoid) {
   extern __shared__ float zl[];      // [Et] scores, [Et] choice scores
   float* ch = zl + Et;
   const int n = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
@@ -110,45 +111,65 @@ __global__ void __launch_bounds__(1024) k_router_scored(const T* __restrict__ h,
     }
   }
   __syncthreads();
-  if (threadIdx.x == 0) {
+  if (warp != 0) return;
+  // one warp scores and chooses: lane l holds the experts l, l + 32, ...
+  if (score_sigmoid) {
+    for (int e = lane; e < Et; e += 32) zl[e] = sigmoid_f(zl[e]);
+  } else {
     float zmax = -INFINITY, sum = 0.f;
-    for (int e = 0; e < Et; e++) zmax = fmaxf(zmax, zl[e]);
-    for (int e = 0; e < Et; e++) { zl[e] = expf(zl[e] - zmax); sum += zl[e]; }
-    for (int e = 0; e < Et; e++) { zl[e] /= sum; ch[e] = zl[e] + (corr ? ldf(corr + e) : 0.f); }
-    if (groups > 0 && keep < groups) {
-      const int per = Et / groups;
-      // drop the groups - keep worst runs: repeatedly the run with the smallest best score (ties: the higher index goes)
-      unsigned long long alive[4] = {~0ull, ~0ull, ~0ull, ~0ull};      // groups <= 256
-      for (int d = 0; d < groups - keep; d++) {
-        int worst = -1;
-        float wv = INFINITY;
-        for (int g = 0; g < groups; g++) {
-          if (!((alive[g >> 6] >> (g & 63)) & 1ull)) continue;
-          float best = -INFINITY;
-          for (int e = g * per; e < (g + 1) * per; e++) best = fmaxf(best, ch[e]);
-          if (worst < 0 || best <= wv) { wv = best; worst = g; }
-        }
-        alive[worst >> 6] &= ~(1ull << (worst & 63));
-        for (int e = worst * per; e < (worst + 1) * per; e++) ch[e] = -INFINITY;
+    for (int e = lane; e < Et; e += 32) zmax = fmaxf(zmax, zl[e]);
+    zmax = warp_max(zmax);
+    for (int e = lane; e < Et; e += 32) { zl[e] = expf(zl[e] - zmax); sum += zl[e]; }
+    sum = warp_sum(sum);
+    for (int e = lane; e < Et; e += 32) zl[e] /= sum;
+  }
+  for (int e = lane; e < Et; e += 32) ch[e] = zl[e] + (corr ? ldf(corr + e) : 0.f);
+  __syncwarp();
+  if (groups > 0 && keep < groups && lane == 0) {
+    const int per = Et / groups;
+    // drop the groups - keep worst runs: repeatedly the run with the smallest best score (ties: the higher index goes)
+    unsigned long long alive[4] = {~0ull, ~0ull, ~0ull, ~0ull};      // groups <= 256
+    for (int d = 0; d < groups - keep; d++) {
+      int worst = -1;
+      float wv = INFINITY;
+      for (int g = 0; g < groups; g++) {
+        if (!((alive[g >> 6] >> (g & 63)) & 1ull)) continue;
+        float best = -INFINITY;
+        for (int e = g * per; e < (g + 1) * per; e++) best = fmaxf(best, ch[e]);
+        if (worst < 0 || best <= wv) { wv = best; worst = g; }
       }
+      alive[worst >> 6] &= ~(1ull << (worst & 63));
+      for (int e = worst * per; e < (worst + 1) * per; e++) ch[e] = -INFINITY;
     }
-    int32_t* id = idx + (size_t)n * top;
-    float ssum = 0.f;
-    for (int j = 0; j < top; j++) {
-      int arg = -1;
-      float m = -INFINITY;
-      for (int e = 0; e < Et; e++) {
-        bool taken = false;
-        for (int i = 0; i < j; i++) taken = taken || id[i] == e;
-        if (!taken && (arg < 0 || ch[e] > m)) { m = ch[e]; arg = e; }
-      }
-      id[j] = arg;
-      ssum += zl[arg];
+  }
+  __syncwarp();
+  // the `top` largest in descending order, the lower index first among equals; a taken expert's choice score becomes NaN.  Lane j
+  // keeps choice j (top <= 16).
+  int mine = 0;
+  float ssum = 0.f;
+  for (int j = 0; j < top; j++) {
+    int arg = -1;
+    float m = -INFINITY;
+    for (int e = lane; e < Et; e += 32) {
+      const float c = ch[e];
+      if (c == c && (arg < 0 || c > m)) { m = c; arg = e; }
     }
-    for (int j = 0; j < top; j++) {
-      wt[(size_t)n * top + j] = zl[id[j]] / (ssum + 1e-20f) * scale;
-      pos[(size_t)n * top + j] = n * top + j;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const int a2 = __shfl_xor_sync(0xffffffffu, arg, o);
+      const float m2 = __shfl_xor_sync(0xffffffffu, m, o);
+      if (a2 >= 0 && (arg < 0 || m2 > m || (m2 == m && a2 < arg))) { m = m2; arg = a2; }
     }
+    arg = max(arg, 0);      // (scores that are not numbers choose nothing; any index in range will do)
+    ssum += zl[arg];
+    if (lane == j) mine = arg;
+    if (lane == 0) ch[arg] = __int_as_float(0x7fffffff);
+    __syncwarp();
+  }
+  if (lane < top) {
+    idx[(size_t)n * top + lane] = mine;
+    wt[(size_t)n * top + lane] = zl[mine] / (ssum + 1e-20f) * scale;
+    pos[(size_t)n * top + lane] = n * top + lane;
   }
 }
 
@@ -203,8 +224,9 @@ __global__ void __launch_bounds__(256) k_moe_tiles(const T* __restrict__ X, cons
   __shared__ float Xs[BK][BM + 4], Ws[BK][BN + 4], Vs[BK][BN + 4];
   __shared__ int32_t src[BM];
   const int e = pl.tile_e[t], r0 = pl.tile_r0[t], rows = pl.tile_rows[t];
-  const T* Wa = (const T*)etab[UP ? e : 2 * E + e];
-  const T* Wb = UP ? (const T*)etab[E + e] : nullptr;
+  const bool two = UP && act_two(act);      // an expert without a gate has its up matrix alone
+  const T* Wa = (const T*)etab[UP ? (two ? e : E + e) : 2 * E + e];
+  const T* Wb = two ? (const T*)etab[E + e] : nullptr;
   for (int r = threadIdx.x; r < BM; r += 256) src[r] = r < rows ? (UP ? pl.row_tok[r0 + r] : r0 + r) : -1;
   __syncthreads();
   const int o0 = blockIdx.x * BN;
@@ -219,7 +241,7 @@ __global__ void __launch_bounds__(256) k_moe_tiles(const T* __restrict__ X, cons
       const int r = el / BK, c = el % BK;
       Xs[c][r] = (src[r] >= 0 && k0 + c < K) ? ldf(X + (size_t)src[r] * K + k0 + c) : 0.f;
       Ws[c][r] = (o0 + r < O && k0 + c < K) ? ldf(Wa + (size_t)(o0 + r) * K + k0 + c) : 0.f;
-      if (UP) Vs[c][r] = (o0 + r < O && k0 + c < K) ? ldf(Wb + (size_t)(o0 + r) * K + k0 + c) : 0.f;
+      if (two) Vs[c][r] = (o0 + r < O && k0 + c < K) ? ldf(Wb + (size_t)(o0 + r) * K + k0 + c) : 0.f;
     }
     __syncthreads();
     float part[4][4], part2[4][4];
@@ -238,7 +260,7 @@ __global__ void __launch_bounds__(256) k_moe_tiles(const T* __restrict__ X, cons
       for (int i = 0; i < 4; i++)
 #pragma unroll
         for (int j = 0; j < 4; j++) part[i][j] = fmaf(a[i], w[j], part[i][j]);
-      if (UP) {
+      if (two) {
 #pragma unroll
         for (int j = 0; j < 4; j++) w[j] = Vs[k][tx * 4 + j];
 #pragma unroll
@@ -252,7 +274,7 @@ __global__ void __launch_bounds__(256) k_moe_tiles(const T* __restrict__ X, cons
 #pragma unroll
       for (int j = 0; j < 4; j++) {
         kahan_add(acc[i][j], cmp[i][j], part[i][j]);
-        if (UP) kahan_add(acc2[i][j], cmp2[i][j], part2[i][j]);
+        if (two) kahan_add(acc2[i][j], cmp2[i][j], part2[i][j]);
       }
     __syncthreads();
   }
@@ -288,7 +310,7 @@ __global__ void __launch_bounds__(256) k_moe_rows(const T* __restrict__ X, const
   if (p >= P) {
     const int n = p - P;
     if (UP) {
-      if (o < sh.ff) linear_row<T>(h + (size_t)n * K, (const T*)sh.gate, (const T*)sh.up, (T*)sh.act + (size_t)n * sh.ff, false, 1, sh.ff, K, act, o, sh.limit);
+      if (o < sh.ff) linear_row<T>(h + (size_t)n * K, (const T*)(act_two(act) ? sh.gate : sh.up), (const T*)sh.up, (T*)sh.act + (size_t)n * sh.ff, false, 1, sh.ff, K, act, o, sh.limit);
     } else {
       if (o < O) linear_row<T>((const T*)sh.act + (size_t)n * sh.ff, (const T*)sh.down, (const T*)nullptr, sh.out + (size_t)n * O, true, 1, O, sh.ff, ACT_NONE, o, 0.f);
     }
@@ -297,7 +319,7 @@ __global__ void __launch_bounds__(256) k_moe_rows(const T* __restrict__ X, const
   const int e = idx[p];
   if (o >= O || e >= E) return;      // an identity expert has no matrices: the combining kernel adds the token's input
   if (UP)
-    linear_row<T>(X + (size_t)(p / top) * K, (const T*)etab[e], (const T*)etab[E + e], (T*)Y + (size_t)p * O, false, 1, O, K, act, o, limit);
+    linear_row<T>(X + (size_t)(p / top) * K, (const T*)etab[act_two(act) ? e : E + e], (const T*)etab[E + e], (T*)Y + (size_t)p * O, false, 1, O, K, act, o, limit);
   else
     linear_row<T>(X + (size_t)p * K, (const T*)etab[2 * E + e], (const T*)nullptr, (float*)Y + (size_t)p * O, true, 1, O, K, ACT_NONE, o, 0.f);
 }

@@ -153,6 +153,12 @@ class SequenceBatcher:
     # -- the token loop -------------------------------------------------------------------------------
     def generate(self, requests: Iterable[GenRequest], generator=None) -> Dict[str, List[int]]:
         waiting = list(requests)
+        cap = getattr(self.model, "max_positions", 0)
+        for r in waiting:
+            if len(r.prompt) == 0:
+                raise ValueError(f"request {r.id!r} has an empty prompt")
+            if cap and len(r.prompt) + r.max_new_tokens - 1 > cap:      # the last sampled token is never fed
+                raise ValueError(f"request {r.id!r} would reach position {len(r.prompt) + r.max_new_tokens - 2}, the model has {cap} positions")
         done: Dict[str, List[int]] = {}
         state: Dict[str, dict] = {}
         while waiting or state:
@@ -166,8 +172,6 @@ class SequenceBatcher:
                         raise RuntimeError(f"request {r.id!r} needs {need} pages, the pool has {self.model.pool_pages}")
                     break
                 waiting.pop(0)
-                if len(r.prompt) == 0:
-                    raise ValueError(f"request {r.id!r} has an empty prompt")
                 h = self.admit(r.id)
                 state[r.id] = {"req": r, "fed": 0, "out": [], "next": None,
                                "pages": (lambda hh=h: (hh.offset + PAGE - 1) // PAGE)}

@@ -5,7 +5,8 @@
  * compressed row per token, a gated delta-rule recurrence, a generalized delta rule with a decay and a removal rate per
  * key channel, decayed outer-product recurrences, or attention beside one of those) plus an optional dense, gated or
  * routed feed-forward, tied together by S residual streams; a span of layers may run several times on the same weights;
- * every sublayer's input may pass a short causal convolution first, and the embedding may add a hashed bigram row.
+ * every sublayer's input may pass a short causal convolution first, and the embedding may add a hashed bigram row or a
+ * learned position row; a layer's mixer and feed-forward run one after the other or side by side on one normed input.
  *
  * Same conventions as dnet_b200.h: plain C, opaque handles, 0 or a negative DN_E* code, dn_seq_last_error() for
  * the text, caller-owned streams and buffers, weights BORROWED by pointer.  One handle serves one compute thread.
@@ -41,10 +42,14 @@ extern "C" {
 #define DN_NORM_RMS 0       /* x / sqrt(mean(x^2) + eps) * w  (or 1 + w) */
 #define DN_NORM_DYT 1       /* tanh(alpha x) * w + b, elementwise */
 #define DN_NORM_LAYER 2     /* (x - mean) / sqrt(variance + eps) * w + b */
+#define DN_NORM_RMS_SCALAR 3   /* x / sqrt(mean(x^2) + eps) * g, one number g for all coordinates */
 
 #define DN_QKNORM_NONE 0
 #define DN_QKNORM_WHOLE 1   /* RMS norm over the whole q (k) projection, weight [heads dim] */
 #define DN_QKNORM_HEAD 2    /* RMS norm over each head's dim, one weight [dim] for all heads */
+
+#define DN_ATTN_SOFTMAX 0   /* a visible key's weight is its share of the softmax */
+#define DN_ATTN_SIGMOID 1   /* a visible key's weight is sigmoid(score + offset_h); weights are not normalized over the keys */
 
 #define DN_RIGHT_GLA 0      /* right half of DN_MIX_PARALLEL: gated linear attention, M <- diag(d) M + k v^T */
 #define DN_RIGHT_GDELTA 1   /* generalized delta rule: S <- diag(w) S - (a u)(u^T S) + k v^T with u = k / |k|, read after the update */
@@ -53,14 +58,17 @@ extern "C" {
 #define DN_MLP_MOE 1        /* routed GLU experts (+ an optional shared one) */
 
 #define DN_FF_GEGLU 0       /* dense feed-forward: gelu_tanh(W_gate h) * (W_up h) */
-#define DN_FF_RELU2 1       /* dense feed-forward: relu(W_up h + b)^2, no gate; up and down may carry biases */
+#define DN_FF_RELU2 1       /* dense feed-forward: relu(W_up h + b)^2, no gate; up and down may carry biases (unbound: none) */
 
 #define DN_ROUTER_TOPK 0    /* the `top` largest logits choose; softmax over the chosen logits weighs */
-#define DN_ROUTER_SCORED 1  /* softmax over all experts scores; a correction is added for the choice only; experts form groups of
-                               which the best are kept; weights = chosen scores / their sum * router_scale */
+#define DN_ROUTER_SCORED 1  /* every expert gets a score (DN_SCORE_*); a correction, if bound, is added for the choice only; experts form
+                               groups of which the best are kept; weights = chosen scores / their sum * router_scale */
+#define DN_SCORE_SOFTMAX 0  /* DN_ROUTER_SCORED: softmax over all experts */
+#define DN_SCORE_SIGMOID 1  /* DN_ROUTER_SCORED: sigmoid of each logit */
 
 #define DN_EXPERT_CGLU 0    /* clamped GLU: g = min(gate, limit), u = clamp(up, +-limit), g sigmoid(1.702 g) (u + 1) */
 #define DN_EXPERT_SWIGLU 1  /* silu(gate) * up */
+#define DN_EXPERT_RELU2 2   /* relu(up)^2, no gate matrix */
 
 typedef struct dn_seq_model dn_seq_model;
 typedef void* dn_seq_stream;   /* cudaStream_t */
@@ -120,6 +128,10 @@ typedef struct dn_seq_layer_cfg {
   /* DN_MIX_PARALLEL */
   int32_t r_kind;      /* DN_RIGHT_* */
   int32_t branch_norm; /* 1: each half's output is RMS-normed over the width (weights DN_SQ_L_OUT / DN_SQ_R_OUT) before the scaled sum */
+  /* attention */
+  int32_t attn_weight; /* DN_ATTN_*: what turns a score into a key's weight */
+  int32_t dist_bias;   /* 1: r1_h ln(1 + r2_h (i - j)) is taken off the score of the key at j for the query at i */
+  int32_t score_kind;  /* DN_SCORE_*: DN_ROUTER_SCORED */
 } dn_seq_layer_cfg;
 
 typedef struct dn_seq_cfg {
@@ -146,6 +158,10 @@ typedef struct dn_seq_cfg {
    * sequence's first token; the previous token is carried per sequence (buckets 0: none) */
   int32_t bigram_buckets, bigram_mul_prev, bigram_mul_cur;
   float logit_scale;         /* logits are multiplied by this (0: by 1) */
+  /* 1: a layer has one norm, whose output both its mixer and its feed-forward read; both outputs join the residual together */
+  int32_t parallel_ff;
+  float residual_mult;       /* sublayer outputs are multiplied by this as they join the residual (0: by 1) */
+  int32_t max_positions;     /* rows of DN_SQ_POS: row p is added to the embedding of the token at position p (0: none); no sequence grows longer */
 } dn_seq_cfg;
 
 /* tensors of a layer (dn_seq_bind: layer >= 0) and of the model (layer = -1) */
@@ -177,9 +193,11 @@ enum {
    * DN_RIGHT_GDELTA: the removal rate's projection [C, W] and bias [C] (DN_SQ_R_Q is the read vector's projection,
    * DN_SQ_DECAY1 / 2 / _B the decay's, DN_SQ_R_NORM [C] one weight per channel) */
   DN_SQ_CANON1, DN_SQ_CANON2, DN_SQ_L_OUT, DN_SQ_R_OUT, DN_SQ_R_A, DN_SQ_R_AB,
+  /* dist_bias: r1, r2 [H]; DN_ATTN_SIGMOID: the offset of the scores [H] */
+  DN_SQ_DIST1, DN_SQ_DIST2, DN_SQ_ATTN_OFF,
   DN_SQ_COUNT,
   DN_SQ_EMBED = 100, DN_SQ_FINAL_NORM, DN_SQ_HEAD, DN_SQ_FINAL_NORM_B, DN_SQ_FINAL_NORM_ALPHA,
-  DN_SQ_EMBED_NORM, DN_SQ_EMBED_NORM_B, DN_SQ_EMBED_NORM_ALPHA, DN_SQ_LOOP_IN, DN_SQ_BIGRAM
+  DN_SQ_EMBED_NORM, DN_SQ_EMBED_NORM_B, DN_SQ_EMBED_NORM_ALPHA, DN_SQ_LOOP_IN, DN_SQ_BIGRAM, DN_SQ_POS
 };
 /* matrices of a routed expert (dn_seq_bind_expert) */
 enum { DN_SQ_E_GATE = 0, DN_SQ_E_UP, DN_SQ_E_DOWN };

@@ -65,7 +65,7 @@ def test_header_and_binding_agree():
              "HEAD_GATE": "head_gate", "SINK": "sink", "BONUS": "bonus", "DECAY1": "decay1", "DECAY2": "decay2", "DECAY_B": "decay.b",
              "ROUTER": "router", "ROUTER_B": "router.b", "SH_GATE": "shared.gate", "SH_UP": "shared.up", "SH_DOWN": "shared.down",
              "UP_B": "mlp.up.b", "DOWN_B": "mlp.down.b", "ROUTER_CORR": "router.corr", "SH_SG": "shared.sg",
-             "CANON1": "canon1", "CANON2": "canon2", "L_OUT": "l.out"}
+             "CANON1": "canon1", "CANON2": "canon2", "L_OUT": "l.out", "DIST1": "mix.r1", "DIST2": "mix.r2", "ATTN_OFF": "mix.pb"}
     for i, name in enumerate(order):
         n = name[len("DN_SQ_"):]
         if n in spell:
@@ -77,7 +77,7 @@ def test_header_and_binding_agree():
         assert _seqabi.LAYER_SLOT[want] == i, (name, want)
     model = [n.strip().split("=")[0].strip() for n in txt.split("DN_SQ_COUNT,", 1)[1].split("}", 1)[0].replace("\n", " ").split(",") if n.strip()]
     assert [_seqabi.MODEL_SLOT[k] for k in ("embed", "final.norm", "head", "final.norm.b", "final.norm.alpha", "embed.norm", "embed.norm.b",
-                                           "embed.norm.alpha", "loop.in", "bigram")] == list(range(100, 100 + len(model)))
+                                           "embed.norm.alpha", "loop.in", "bigram", "pos")] == list(range(100, 100 + len(model)))
 
 
 def _filinex_cfg():
@@ -442,3 +442,123 @@ def test_vulanex_oracle_by_hand():
     # layer norm with the variance of the deviations
     x = torch.tensor([[1.0, 3.0]], dtype=D)
     assert torch.allclose(vo.layer_norm(x, torch.tensor([2.0, 2.0]), torch.tensor([0.5, 0.5]), 0.0), torch.tensor([[-1.5, 2.5]], dtype=D))
+
+
+def _bokenex_cfg():
+    mx = {"heads": 6, "kv_heads": 2, "dim": 10, "vdim": 7, "conv": 3, "scale": 0.35, "mask": {"size": 19}}
+    moe = {"kind": "moe", "router": {"experts": 5, "top": 2, "scale": 1.75}, "expert": {"ff": 12}}
+    return {"architecture": "Bokenex", "vocab": 50, "width": 36, "norm": {"eps": 1e-5}, "residual_mult": 0.45, "max_positions": 77,
+            "layers": [{"type": "attention", "mixer": mx, "mlp": moe},
+                       {"type": "attention", "mixer": {**mx, "heads": 1, "kv_heads": 1, "vdim": 10, "conv": 1, "mask": {"size": 4}}, "mlp": None},
+                       {"type": "attention", "mixer": {k: v for k, v in mx.items() if k not in ("conv", "mask")}, "mlp": {"kind": "dense", "ff": 24}}]}
+
+
+def test_bokenex_config_and_checkpoint_names():
+    """every constant of the config lands in the structs, what the design fixes comes from the family, and every tensor the
+    oracle writes finds its place through the aliases with its shape (scalars of the norms, no gates, no biases)"""
+    from dnet_b200 import _seqabi
+    from dnet_b200.core.models import ring_model_class
+    from dnet_b200.core.models.seqmix import _LAYER_KEY, parse_layer_list
+    from oracle import bokenex_oracle as bo
+
+    cfg = _bokenex_cfg()
+    cls = ring_model_class("bokenex")
+    sc, layers = parse_layer_list(cfg, cls.family, bo.tensor_shapes(cfg))
+    assert (sc.norm_kind, sc.parallel_ff, sc.post_norm, sc.no_pre_norm, sc.embed_norm, sc.streams) == (_seqabi.DN_NORM_RMS_SCALAR, 1, 0, 0, 0, 0)
+    assert abs(sc.residual_mult - 0.45) < 1e-7 and sc.max_positions == 77 and abs(sc.eps - 1e-5) < 1e-9 and abs(sc.embed_scale - 1.0) < 1e-7
+    assert sc.logit_scale == 1.0 and sc.logit_softcap == 0.0 and sc.bigram_buckets == 0 and sc.canon_taps == 0
+    a, b, c = layers
+    for l in layers:
+        assert (l.mixer, l.attn_weight, l.dist_bias, l.qk_norm, l.mask_kind) == (_seqabi.DN_MIX_ATTENTION, _seqabi.DN_ATTN_SIGMOID, 1, _seqabi.DN_QKNORM_HEAD,
+                                                                                  _seqabi.DN_MASK_WINDOW)
+        assert (l.sink, l.out_gate, l.v_is_k, l.rot_dims, l.pool, l.kv_from, l.qtemp_every) == (0, 0, 0, 0, 0, -1, 0) and abs(l.scale - 0.35) < 1e-7
+    assert (a.heads, a.kv_heads, a.dim, a.vdim, a.conv, a.chunk) == (6, 2, 10, 7, 3, 19)
+    assert (b.heads, b.kv_heads, b.dim, b.vdim, b.conv, b.chunk, b.ff) == (1, 1, 10, 10, 1, 4, 0)
+    assert (c.conv, c.chunk, c.ff, c.mlp_kind, c.ff_act) == (0, 0, 24, _seqabi.DN_MLP_DENSE, _seqabi.DN_FF_RELU2)
+    assert (a.mlp_kind, a.experts, a.top, a.ff, a.expert_act) == (_seqabi.DN_MLP_MOE, 5, 2, 12, _seqabi.DN_EXPERT_RELU2)
+    assert (a.router_kind, a.score_kind, a.groups, a.identity, a.shared_ff) == (_seqabi.DN_ROUTER_SCORED, _seqabi.DN_SCORE_SIGMOID, 0, 0, 0) and a.router_scale == 1.75
+    m = cls.__new__(cls)
+    m.config, m._cfg_struct, m._layer_structs, m.hidden_size, m.vocab_size = cfg, sc, layers, sc.width, sc.vocab
+    want = m.expected_tensors()
+    got = {}
+    for key, sh in bo.tensor_shapes(cfg).items():
+        if _LAYER_KEY.match(key):
+            lname, suffix = key.split(".", 1)
+            key = f"{lname}.{cls.tensor_alias['*'].get(suffix, suffix)}"
+        got[key] = tuple(sh)
+    assert got == {k: tuple(v) for k, v in want.items()}
+    assert want["l0.norm1"] == () and want["final.norm"] == () and want["pos"] == (77, 36)
+    for k in want:
+        if _LAYER_KEY.match(k):
+            suffix = k.split(".", 1)[1]
+            assert suffix in _seqabi.LAYER_SLOT or suffix.split(".")[1].startswith("e"), k
+
+
+def test_other_families_keep_their_defaults():
+    """what the new keys of a family switch on is off where a family does not name them"""
+    from dnet_b200 import _seqabi
+    from dnet_b200.core.models import ring_model_class
+    from dnet_b200.core.models.seqmix import parse_layer_list
+    from oracle import vulanex_oracle as vo
+
+    cfg = _vulanex_cfg()
+    sc, layers = parse_layer_list(cfg, ring_model_class("vulanex").family, vo.tensor_shapes(cfg, rank=5))
+    assert (sc.parallel_ff, sc.residual_mult, sc.max_positions) == (0, 1.0, 0)
+    assert all((l.attn_weight, l.dist_bias, l.score_kind) == (_seqabi.DN_ATTN_SOFTMAX, 0, _seqabi.DN_SCORE_SOFTMAX) for l in layers)
+
+
+def test_bokenex_oracle_by_hand():
+    """the oracle's pieces on numbers small enough to follow"""
+    from oracle import bokenex_oracle as bo
+
+    D = torch.float64
+    # one number weighs all coordinates of a norm; the head norm has one per dimension
+    x = torch.tensor([[3.0, -4.0]], dtype=D)
+    r = math.sqrt(12.5)
+    assert torch.allclose(bo.scalar_rms_norm(x, torch.tensor(2.0, dtype=D), 0.0), x * 2.0 / r)
+    assert torch.allclose(bo.scalar_rms_norm(x, torch.tensor([2.0], dtype=D), 12.5), x * 2.0 / 5.0)        # eps under the root
+    assert torch.allclose(bo.head_rms_norm(x[None], torch.tensor([1.0, 10.0], dtype=D), 0.0), torch.tensor([[[3.0 / r, -40.0 / r]]], dtype=D))
+    # embedding row + position row
+    e = bo.embed([2, 0, 2], torch.tensor([[1.0], [2.0], [4.0]]), torch.tensor([[10.0], [20.0], [30.0], [99.0]]))
+    assert e[:, 0].tolist() == [14.0, 21.0, 34.0]
+    # convolution: the last tap meets the token itself, zeros before the start
+    u = torch.tensor([[1.0], [10.0], [100.0]], dtype=D)
+    y = bo.short_convolution(u, torch.tensor([[0.5, 2.0, 3.0]], dtype=D))
+    assert y[:, 0].tolist() == [3.0, 32.0, 0.5 + 20.0 + 300.0]
+    # a window of 3: position 5 sees 3, 4, 5
+    assert bo.visible(5, 3) == [3, 4, 5] and bo.visible(1, 3) == [0, 1] and bo.visible(3, 0) == [0, 1, 2, 3] and bo.visible(7, 1) == [7]
+    # distance bias: nothing at distance 0, r1 ln(1 + r2 d) beyond
+    d = bo.distance_bias(torch.tensor([0.0, 3.0], dtype=D), torch.tensor([2.0], dtype=D), torch.tensor([0.5], dtype=D))
+    assert d[0, 0] == 0.0 and abs(float(d[0, 1]) - 2.0 * math.log(2.5)) < 1e-12
+    # weights do not sum to one: two keys of score 0 with offset 0 weigh one half each, with offset ln 3 three quarters each
+    z = torch.zeros(2, 1, 1, dtype=D)
+    v = torch.tensor([[[2.0]], [[6.0]]], dtype=D)
+    zero = torch.zeros(1, dtype=D)
+    o = bo.sigmoid_attention(z, z, v, 1.0, 0, zero, zero, zero)
+    assert o[:, 0, 0].tolist() == [1.0, 4.0]
+    o = bo.sigmoid_attention(z, z, v, 1.0, 1, zero, zero, torch.tensor([math.log(3.0)], dtype=D))       # a window of one token
+    assert torch.allclose(o[:, 0, 0], torch.tensor([1.5, 4.5], dtype=D))
+    # query head h reads key / value head h // (H / G)
+    v2 = torch.tensor([[[2.0], [20.0]]], dtype=D)
+    o = bo.sigmoid_attention(torch.zeros(1, 4, 1, dtype=D), torch.zeros(1, 2, 1, dtype=D), v2, 1.0, 0, *[torch.zeros(4, dtype=D)] * 3)
+    assert o[0, :, 0].tolist() == [1.0, 1.0, 10.0, 10.0]
+    # router: sigmoid scores, the two largest divided by their sum, times the scale
+    c, a = bo.route(torch.tensor([1.0], dtype=D), torch.tensor([[0.0], [math.log(3.0)], [-9.0]], dtype=D), 2, 5.0)
+    assert c == [1, 0] and abs(a[0] - 5 * 0.75 / 1.25) < 1e-12 and abs(a[1] - 5 * 0.5 / 1.25) < 1e-12
+    # squared relu
+    assert bo.two_layer(torch.tensor([[2.0]], dtype=D), torch.tensor([[1.0], [-1.0]], dtype=D), torch.tensor([[1.0, 7.0]], dtype=D)).tolist() == [[4.0]]
+
+
+def test_generate_refuses_requests_beyond_the_position_table():
+    from dnet_b200.shard.batching import GenRequest, SequenceBatcher
+
+    class Model:
+        max_positions, max_batch_tokens, free_slots, free_pages = 10, 64, 2, 4
+
+    eng = SequenceBatcher.__new__(SequenceBatcher)
+    eng.model, eng.step_tokens, eng.live = Model(), 64, {}
+    with pytest.raises(ValueError, match="10 positions"):
+        eng.generate([GenRequest("fits", [1] * 3, max_new_tokens=2), GenRequest("long", [1] * 8, max_new_tokens=4)])
+    assert not eng.live
+    with pytest.raises(ValueError, match="empty"):
+        eng.generate([GenRequest("none", [])])
