@@ -695,6 +695,7 @@ static cudaError_t gemm_tc(const CUtensorMap& w, const CUtensorMap& w2, const XM
 // One product Y[N, O] = X[N, K] W[O, K]^T (act: an ACT_* epilogue, the two-operand ones on X W^T and X W2^T).  bf16 batches of 16 tokens and more run on
 // the tcgen05 GEMM when the operands have TMA descriptors; a few rows (decode) on the weight-streaming row kernel;
 // everything else, and all of fp32, on the CUDA-core tiles.
+constexpr int ROWS_PAIR = 2048;      // output features from which a warp of the row kernels takes two (fewer leave too few warps)
 struct LinMaps { const CUtensorMap* w; const CUtensorMap* w2; const XMaps* x; };
 template <class T>
 static cudaError_t linear(dn_seq_model* m, cudaStream_t s, const T* X, const void* W, const void* W2, void* Y, int N, int O, int K, bool out32,
@@ -714,9 +715,13 @@ static cudaError_t linear(dn_seq_model* m, cudaStream_t s, const T* X, const voi
     return gemm_tc<dn::EPI_STORE>(*tm.w, *tm.w, *tm.x, p, s);
   }
   if (N <= 8) {
-    dim3 grid((O + 7) / 8);
-    if (out32) return launch(k_linear_rows<T, true>, grid, dim3(256), 0, s, X, (const T*)W, (const T*)W2, Y, N, O, K, act, alim, (const T*)bias);
-    return launch(k_linear_rows<T, false>, grid, dim3(256), 0, s, X, (const T*)W, (const T*)W2, Y, N, O, K, act, alim, (const T*)bias);
+    const bool two = act_two(act), pair = !two && O >= ROWS_PAIR;
+    const int per = pair ? 2 : 1;
+    dim3 grid((O + 8 * per - 1) / (8 * per));
+#define LR(NT) (two || pair ? launch(k_linear_rows<T, NT, true>, grid, dim3(256), 0, s, X, (const T*)W, (const T*)W2, Y, out32 ? 1 : 0, N, O, K, act, per, alim, (const T*)bias) \
+                            : launch(k_linear_rows<T, NT, false>, grid, dim3(256), 0, s, X, (const T*)W, (const T*)W2, Y, out32 ? 1 : 0, N, O, K, act, per, alim, (const T*)bias))
+    return N == 1 ? LR(1) : N == 2 ? LR(2) : N <= 4 ? LR(4) : LR(8);
+#undef LR
   }
   dim3 grid((O + 63) / 64, (N + 63) / 64);
   if (out32) return launch(k_linear<T, true>, grid, dim3(256), 0, s, X, (const T*)W, (const T*)W2, Y, N, O, K, act, alim, (const T*)bias);
@@ -1053,9 +1058,14 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
     const bool ride = few && c.parallel_ff && lc.ff > 0 && lc.mlp_kind == DN_MLP_DENSE && lc.ff_act == DN_FF_RELU2 && lc.mixer == DN_MIX_ATTENTION &&
                       !l.w[DN_SQ_UP_B] && !l.w[DN_SQ_DOWN_B];
     auto run_segs = [&]() {
-      int blocks = 0;
-      for (int i = 0; i < sg.n; i++) blocks += (sg.O[i] + 7) / 8;
-      return launch(k_linear_rows_multi<T>, dim3(blocks), dim3(256), 0, s, (const T*)m->h, sg, N, W);
+      int blocks = 0, rows = 0;
+      for (int i = 0; i < sg.n; i++) rows += sg.O[i];
+      const bool pair = rows >= ROWS_PAIR;
+      for (int i = 0; i < sg.n; i++) blocks += pair ? (sg.O[i] + 15) / 16 : (sg.O[i] + 7) / 8;
+#define LR(NT) (pair ? launch(k_linear_rows_multi<T, NT, true>, dim3(blocks), dim3(256), 0, s, (const T*)m->h, sg, N, W) \
+                     : launch(k_linear_rows_multi<T, NT, false>, dim3(blocks), dim3(256), 0, s, (const T*)m->h, sg, N, W))
+      return N == 1 ? LR(1) : N == 2 ? LR(2) : N <= 4 ? LR(4) : LR(8);
+#undef LR
     };
     if (lc.mixer == DN_MIX_ATTENTION || lc.mixer == DN_MIX_DELTA || lc.mixer == DN_MIX_PARALLEL) {
       PH(DN_SEQ_PH_PROJ);
@@ -1087,9 +1097,22 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
                    lc.attn_weight == DN_ATTN_SIGMOID ? l.w[DN_SQ_ATTN_OFF] : nullptr};
       const size_t sm = ((size_t)l.Cq + l.Ck + 40 + lc.heads + lc.kv_heads + lc.rot_dims) * 4;
       PH(DN_SEQ_PH_ATTN_PREP);
-      CK(launch(k_attn_prep<T>, dim3(N), dim3(256), sm, s, a, b, (const T*)m->uq, (const T*)m->uk, (const T*)m->uv, w(DN_SQ_Q_CONV),
-                w(DN_SQ_K_CONV), w(DN_SQ_V_CONV), w(DN_SQ_Q_NORM), w(DN_SQ_K_NORM), cst, m->conv_stride, (T*)m->qb,
-                (T*)m->kpool[run.kv_index], (T*)m->vpool[run.kv_index]));
+      // heads that do not rotate and are normed alone (or not at all): a warp a head (a function of the model, not of the batch)
+      uintptr_t al = (uintptr_t)cst | (m->conv_stride * sizeof(T));
+      for (int q : {DN_SQ_Q_CONV, DN_SQ_K_CONV, DN_SQ_V_CONV, DN_SQ_Q_NORM, DN_SQ_K_NORM}) al |= (uintptr_t)l.w[q];
+      const bool by_head = lc.rot_dims == 0 && lc.qk_norm != DN_QKNORM_WHOLE && lc.dim % 4 == 0 && lc.vdim % 4 == 0 && lc.dim <= 128 && lc.vdim <= 128 &&
+                           lc.conv <= PREP_MAX_TAPS && (al & (4 * sizeof(T) - 1)) == 0;
+      if (by_head) {
+        const int units = lc.heads + (l.Ck ? lc.kv_heads : 0) + (l.Cv ? lc.kv_heads : 0), tok = N > 64 ? 8 : 1;
+        auto kern = lc.conv == 0 ? k_attn_prep_heads<T, 0> : lc.conv == 1 ? k_attn_prep_heads<T, 1> : lc.conv == 2 ? k_attn_prep_heads<T, 2>
+                  : lc.conv == 3 ? k_attn_prep_heads<T, 3> : k_attn_prep_heads<T, 4>;
+        CK(launch(kern, dim3((N + tok - 1) / tok, (units + PREP_WARPS - 1) / PREP_WARPS), dim3(32 * PREP_WARPS), 0, s, a, b, tok, (const T*)m->uq, (const T*)m->uk,
+                  (const T*)m->uv, w(DN_SQ_Q_CONV), w(DN_SQ_K_CONV), w(DN_SQ_V_CONV), w(DN_SQ_Q_NORM), w(DN_SQ_K_NORM), cst, m->conv_stride, (T*)m->qb,
+                  (T*)m->kpool[run.kv_index], (T*)m->vpool[run.kv_index]));
+      } else
+        CK(launch(k_attn_prep<T>, dim3(N), dim3(256), sm, s, a, b, (const T*)m->uq, (const T*)m->uk, (const T*)m->uv, w(DN_SQ_Q_CONV),
+                  w(DN_SQ_K_CONV), w(DN_SQ_V_CONV), w(DN_SQ_Q_NORM), w(DN_SQ_K_NORM), cst, m->conv_stride, (T*)m->qb,
+                  (T*)m->kpool[run.kv_index], (T*)m->vpool[run.kv_index]));
       if (lc.pool > 0)      // blocks that this step's tokens complete get their mean key and value
         CK(launch(k_pool_rows<T>, dim3(N), dim3(128), 0, s, b, lc.pool, Ckk, lc.v_is_k ? 0 : lc.kv_heads * lc.vdim, (const T*)m->kpool[run.kv_index], (const T*)vpl,
                   (T*)pkp, (T*)pvp));

@@ -701,16 +701,88 @@ __device__ __forceinline__ void linear_row(const T* __restrict__ X, const T* __r
     }
   }
 }
-template <class T, bool OUT32>
+// The same sums for NT rows (N <= NT; rows beyond N repeat row N - 1 and are not stored) against one or two weight rows at a
+// time: two rows share the activations' loads.  The second row is the second operand of a two-operand activation (one
+// output feature), or the next output feature (PAIR).  Every output's sum runs in the order of linear_row.
+template <class T, int NT, bool TWO>
+__device__ __forceinline__ void dot_rows(const T* __restrict__ X, const T* __restrict__ wa, const T* __restrict__ wb, int N, int K, bool vec,
+                                         float (&a)[NT], float (&b)[NT]) {
+  constexpr int V = Vec16<T>::n;
+  const int lane = threadIdx.x & 31;
+#pragma unroll
+  for (int i = 0; i < NT; i++) a[i] = b[i] = 0.f;
+  size_t xo[NT];
+#pragma unroll
+  for (int i = 0; i < NT; i++) xo[i] = (size_t)min(i, N - 1) * K;
+  if (vec) {
+#pragma unroll (NT <= 2 ? 4 : 2)
+    for (int k = lane * V; k < K; k += 32 * V) {
+      float wv[V], uv[V];
+      ldv(wa + k, wv);
+      if (TWO) ldv(wb + k, uv);
+#pragma unroll
+      for (int i = 0; i < NT; i++) {
+        float x[V];
+        ldv(X + xo[i] + k, x);
+#pragma unroll
+        for (int j = 0; j < V; j++) {
+          a[i] = fmaf(x[j], wv[j], a[i]);
+          if (TWO) b[i] = fmaf(x[j], uv[j], b[i]);
+        }
+      }
+    }
+  } else {
+    for (int k = lane; k < K; k += 32) {
+      const float w = ldf(wa + k), u = TWO ? ldf(wb + k) : 0.f;
+#pragma unroll
+      for (int i = 0; i < NT; i++) {
+        const float x = ldf(X + xo[i] + k);
+        a[i] = fmaf(x, w, a[i]);
+        if (TWO) b[i] = fmaf(x, u, b[i]);
+      }
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < NT; i++) {
+    a[i] = warp_sum(a[i]);
+    if (TWO) b[i] = warp_sum(b[i]);
+  }
+}
+// output feature o (and o + 1 where `pair`) of one product
+template <class T, int NT, bool TWO>
+__device__ __forceinline__ void linear_rows_at(const T* __restrict__ X, const T* __restrict__ Wt, const T* __restrict__ W2, void* __restrict__ Y, bool out32,
+                                               int N, int O, int K, int actc, int o, float alim, const T* __restrict__ bias) {
+  constexpr int V = Vec16<T>::n;
+  const bool two = act_two(actc);
+  const bool pair = TWO && !two && o + 1 < O;
+  const T* wa = Wt + (size_t)o * K;
+  const T* wb = two ? W2 + (size_t)o * K : pair ? wa + K : wa;
+  const bool vec = (K % V == 0) && ((((uintptr_t)Wt | (uintptr_t)X | (uintptr_t)(two ? W2 : Wt)) & 15) == 0);
+  float a[NT], b[NT];
+  dot_rows<T, NT, TWO>(X, wa, wb, N, K, vec, a, b);
+  if ((threadIdx.x & 31) != 0) return;
+  auto put = [&](int i, int oo, float v) {
+    if (out32) ((float*)Y)[(size_t)i * O + oo] = v;
+    else stf((T*)Y + (size_t)i * O + oo, v);
+  };
+#pragma unroll
+  for (int i = 0; i < NT; i++) {
+    if (i >= N) continue;
+    put(i, o, act_apply(actc, a[i] + (bias ? ldf(bias + o) : 0.f), b[i], alim));
+    if (pair) put(i, o + 1, act_apply(actc, b[i] + (bias ? ldf(bias + o + 1) : 0.f), 0.f, alim));
+  }
+}
+// TWO: two-operand products one output feature a warp, others two (`per` = 1 or 2 output features a warp)
+template <class T, int NT, bool TWO>
 __global__ void __launch_bounds__(256) k_linear_rows(const T* __restrict__ X, const T* __restrict__ Wt, const T* __restrict__ W2,
-                                                     void* __restrict__ Y, int N, int O, int K, int act, float alim,
+                                                     void* __restrict__ Y, int out32, int N, int O, int K, int act, int per, float alim,
                                                      const T* __restrict__ bias) {
-  const int o = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  const int o = (blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5)) * per;
   if (o >= O) return;
-  linear_row<T>(X, Wt, W2, Y, OUT32, N, O, K, act, o, alim, bias);
+  linear_rows_at<T, NT, TWO>(X, Wt, W2, Y, out32 != 0, N, O, K, act, o, alim, bias);
 }
 // several products of the same few rows in one launch (the projections of a mixer in a decode step): blocks are
-// dealt to the products in order, 8 output features each
+// dealt to the products in order, 8 output features each (16 where a warp takes two)
 constexpr int MAX_SEGS = 8;
 struct LinSegs {
   const void* X[MAX_SEGS];   // null: the launch's common input
@@ -722,19 +794,20 @@ struct LinSegs {
   int K[MAX_SEGS];           // 0: the launch's common K
   int n;
 };
-template <class T>
+template <class T, int NT, bool TWO>
 __global__ void __launch_bounds__(256) k_linear_rows_multi(const T* __restrict__ X, LinSegs sg, int N, int K) {
+  constexpr int PER = TWO ? 2 : 1;
   int blk = blockIdx.x, i = 0;
   for (; i < sg.n; i++) {
-    const int nb = (sg.O[i] + 7) / 8;
+    const int nb = (sg.O[i] + 8 * PER - 1) / (8 * PER);
     if (blk < nb) break;
     blk -= nb;
   }
   if (i >= sg.n) return;
-  const int o = blk * 8 + (threadIdx.x >> 5);
+  const int o = (blk * 8 + (threadIdx.x >> 5)) * PER;
   if (o >= sg.O[i]) return;
-  linear_row<T>(sg.X[i] ? (const T*)sg.X[i] : X, (const T*)sg.W[i], (const T*)nullptr, sg.Y[i], sg.out32[i] != 0, N, sg.O[i], sg.K[i] > 0 ? sg.K[i] : K,
-                sg.act[i], o);
+  linear_rows_at<T, NT, TWO>(sg.X[i] ? (const T*)sg.X[i] : X, (const T*)sg.W[i], (const T*)nullptr, sg.Y[i], sg.out32[i] != 0, N, sg.O[i],
+                             sg.K[i] > 0 ? sg.K[i] : K, sg.act[i], o, 0.f, (const T*)nullptr);
 }
 
 // ---------------------------------------------------------------------------------------------------------------
@@ -959,6 +1032,108 @@ __global__ void k_attn_prep(AttnPrep a, Batch b, const T* __restrict__ Uq, const
     T* vr = vpool + ((size_t)page * PAGE + prow) * Cv;
     for (int c = threadIdx.x; c < Cv; c += blockDim.x)
       stf(vr + c, conv(Uv, Cv, cwv, c, Cq + Ck));
+  }
+}
+
+// The same for heads that do not rotate and whose norm (if any) is their own: one warp a head of q, k or v walks `tok`
+// consecutive tokens.  A lane owns four adjacent channels (head sizes up to 128, multiples of 4), keeps their weights and the
+// last TAPS - 1 inputs in registers and reads every input row once; the head's sum of squares runs over a lane's four channels
+// in ascending order, then pairwise over the lanes.  Nothing is shared between warps.
+__device__ __forceinline__ void ld4(const float* p, float (&o)[4]) { *reinterpret_cast<float4*>(o) = *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ void ld4(const bf16* p, float (&o)[4]) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.y));
+  o[0] = a.x; o[1] = a.y; o[2] = b.x; o[3] = b.y;
+}
+__device__ __forceinline__ void st4(float* p, const float (&o)[4]) { *reinterpret_cast<float4*>(p) = make_float4(o[0], o[1], o[2], o[3]); }
+__device__ __forceinline__ void st4(bf16* p, const float (&o)[4]) {
+  uint2 v;
+  *reinterpret_cast<__nv_bfloat162*>(&v.x) = __floats2bfloat162_rn(o[0], o[1]);
+  *reinterpret_cast<__nv_bfloat162*>(&v.y) = __floats2bfloat162_rn(o[2], o[3]);
+  *reinterpret_cast<uint2*>(p) = v;
+}
+constexpr int PREP_MAX_TAPS = 4, PREP_WARPS = 4;
+template <class T, int TAPS>
+__global__ void __launch_bounds__(32 * PREP_WARPS) k_attn_prep_heads(AttnPrep a, Batch b, int tok, const T* __restrict__ Uq, const T* __restrict__ Uk,
+                                                                     const T* __restrict__ Uv, const T* __restrict__ cwq, const T* __restrict__ cwk,
+                                                                     const T* __restrict__ cwv, const T* __restrict__ nq, const T* __restrict__ nk,
+                                                                     T* __restrict__ cstate, size_t slot_stride, T* __restrict__ qout, T* __restrict__ kpool,
+                                                                     T* __restrict__ vpool) {
+  const int Cq = a.H * a.dk, Ck = a.own_kv ? a.G * a.dk : 0, Cv = (a.own_kv && a.own_v) ? a.G * a.dv : 0, ldst = Cq + Ck + Cv;
+  const int units = a.H + (Ck ? a.G : 0) + (Cv ? a.G : 0), unit = blockIdx.y * PREP_WARPS + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (unit >= units) return;
+  const int kind = unit < a.H ? 0 : (Ck && unit < a.H + a.G) ? 1 : 2;      // q, k, v
+  const int hh = kind == 0 ? unit : kind == 1 ? unit - a.H : unit - a.H - a.G, d = kind == 2 ? a.dv : a.dk;
+  const bool live = lane * 4 < d;
+  const int c = hh * d + lane * 4;      // the lane's first channel of its projection
+  const int C = kind == 0 ? Cq : kind == 1 ? Ck : Cv, soff = kind == 0 ? 0 : kind == 1 ? Cq : Cq + Ck;
+  const T* U = (kind == 0 ? Uq : kind == 1 ? Uk : Uv) + c;
+  constexpr int TW = TAPS > 0 ? TAPS : 1, M = TAPS > 1 ? TAPS - 1 : 0, MH = M > 0 ? M : 1;
+  float wl[4 * TW], nwt[4], hist[MH][4];
+  if (TAPS > 0 && live) {
+    const T* cw = (kind == 0 ? cwq : kind == 1 ? cwk : cwv) + (size_t)c * TAPS;
+#pragma unroll
+    for (int j = 0; j < TW; j++) ld4(cw + 4 * j, *reinterpret_cast<float(*)[4]>(wl + 4 * j));
+  }
+  const bool normed = kind < 2 && a.norm == 2;
+  if (normed && live) ld4((kind == 0 ? nq : nk) + lane * 4, nwt);
+  const int n0 = blockIdx.x * tok, n1 = min(b.N, n0 + tok);
+  for (int n = n0; n < n1; n++) {
+    const int slot = b.slot[n], p = b.pos[n], local = n - b.first[n];
+    T* st = cstate + (size_t)slot * slot_stride + soff + c;
+    float x[4] = {0.f, 0.f, 0.f, 0.f}, y[4];
+    if (live) {
+      if (M > 0 && (n == n0 || local == 0)) {      // the inputs before this one: rows of the step, or the slot's carried ones
+#pragma unroll
+        for (int j = 0; j < M; j++) {
+          const int back = M - j;
+          ld4(back <= local ? U + (size_t)(n - back) * C : st + (size_t)(M - (back - local)) * ldst, hist[j]);
+        }
+      }
+      ld4(U + (size_t)n * C, x);
+    }
+    if (TAPS > 0) {
+#pragma unroll
+      for (int i = 0; i < 4; i++) {
+        float s = 0.f;
+#pragma unroll
+        for (int j = 0; j < M; j++) s += wl[i * TW + j] * hist[j][i];
+        y[i] = live ? s + wl[i * TW + TW - 1] * x[i] : 0.f;
+      }
+      if (M > 0 && live) {
+#pragma unroll
+        for (int j = 0; j + 1 < M; j++)
+#pragma unroll
+          for (int i = 0; i < 4; i++) hist[j][i] = hist[j + 1][i];
+#pragma unroll
+        for (int i = 0; i < 4; i++) hist[MH - 1][i] = x[i];
+        if (a.carry) {
+#pragma unroll
+          for (int j = 0; j < M; j++) st4(st + (size_t)j * ldst, hist[j]);
+        }
+      }
+    } else {
+#pragma unroll
+      for (int i = 0; i < 4; i++) y[i] = x[i];
+    }
+    if (normed) {
+      const float ss = warp_sum(y[0] * y[0] + y[1] * y[1] + y[2] * y[2] + y[3] * y[3]);
+      const float r = 1.f / sqrtf(ss / (float)d + a.eps);
+#pragma unroll
+      for (int i = 0; i < 4; i++) y[i] = live ? y[i] * r * nwt[i] : 0.f;
+    }
+    if (!live) continue;
+    if (kind == 0) {
+      if (a.qt_every > 0) {
+        const float qt = 1.f + a.qt_coef * logf((float)((p + 1) / a.qt_every + 1));
+#pragma unroll
+        for (int i = 0; i < 4; i++) y[i] *= qt;
+      }
+      st4(qout + (size_t)n * Cq + c, y);
+    } else {
+      const size_t row = (size_t)b.bt[(size_t)slot * b.max_pages + p / PAGE] * PAGE + p % PAGE;
+      st4((kind == 1 ? kpool : vpool) + row * C + c, y);
+    }
   }
 }
 
