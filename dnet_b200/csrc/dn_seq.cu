@@ -2,6 +2,7 @@
 // bound weight pointers, the page pool and the state slots, the staging of a step's batch description, and the
 // launch sequence of a layer.  All arithmetic is in dn_seq_kernels.cuh.
 #include "dn_seq_kernels.cuh"
+#include "dn_seq_attn_rows.cuh"
 #include "dn_seq_recur.cuh"
 #include "dn_seq_moe.cuh"
 #include "dn_seq_latent.cuh"
@@ -98,6 +99,7 @@ struct dn_seq_model {
   // scratch
   float *xs = nullptr, *y = nullptr, *pa = nullptr, *pb = nullptr, *qn = nullptr, *kn = nullptr, *vv = nullptr, *od = nullptr,
         *beta = nullptr, *decay = nullptr, *y2 = nullptr, *x0 = nullptr, *dz = nullptr, *rwt = nullptr, *eo = nullptr, *sgate = nullptr;
+  unsigned int* attn_count = nullptr; // blocks of a split row that have finished [AT_SPLIT_ROWS][heads]; zero between launches
   int part_dv = 256;            // widest value row (padded to 32) of a split attention row's partials
   void *h = nullptr, *uq = nullptr, *uk = nullptr, *uv = nullptr, *qb = nullptr, *mo = nullptr, *gt = nullptr, *act = nullptr, *cat = nullptr,
        *xm = nullptr, *lr = nullptr, *eact = nullptr;
@@ -203,7 +205,7 @@ extern "C" int dn_seq_model_destroy(dn_seq_model* m) {
   cudaDeviceSynchronize();
   void* ptrs[] = {m->xs, m->y, m->pa, m->pb, m->qn, m->kn, m->vv, m->od, m->beta, m->decay, m->h, m->uq, m->uk, m->uv, m->qb,
                   m->mo, m->gt, m->act, m->conv_state, m->delta_state, m->stage_d, m->bt_d, m->tc_err, m->y2, m->x0, m->dz, m->rwt,
-                  m->eo, m->cat, m->xm, m->lr, m->eact, m->ridx, m->rpos, m->rtok, m->tiles, m->xg, m->attn_part, m->sgate, m->hn, m->un, m->aun};
+                  m->eo, m->cat, m->xm, m->lr, m->eact, m->ridx, m->rpos, m->rtok, m->tiles, m->xg, m->attn_part, m->attn_count, m->sgate, m->hn, m->un, m->aun};
   for (void* p : ptrs) if (p) cudaFree(p);
   for (auto& g : m->graphs) cudaGraphExecDestroy(g.second.first);
   if (m->lg_buf) cudaFree(m->lg_buf);
@@ -483,6 +485,7 @@ extern "C" int dn_seq_model_create(const dn_seq_cfg* cfg, const dn_seq_layer_cfg
   DA(m->beta, MB * mh * 4); DA(m->decay, MB * mh * 4);
   DA(m->y2, MB * W * 4); DA(m->dz, MB * mdq * 4); DA(m->lr, MB * mrank * e);
   DA(m->attn_part, (size_t)AT_SPLIT_ROWS * mh * AT_MAX_SPLITS * (2 + m->part_dv) * 4);
+  DA(m->attn_count, (size_t)AT_SPLIT_ROWS * mh * 4);
   DA(m->sgate, MB * 4);
   if (looped) { DA(m->x0, MB * W * 4); DA(m->cat, MB * 2 * W * e); }
   if (any_wkv) DA(m->xm, (size_t)SHIFT_MAX * MB * W * e);
@@ -502,6 +505,7 @@ extern "C" int dn_seq_model_create(const dn_seq_cfg* cfg, const dn_seq_layer_cfg
   DA(m->stage_d, m->stage_ints * 4); DA(m->bt_d, (size_t)cfg->max_seqs * m->max_pages * 4); DA(m->tc_err, 16);
   DA(m->lg_buf, (size_t)8 * cfg->vocab * 4);
 #undef DA
+  if (rc == DN_OK && cudaMemset(m->attn_count, 0, (size_t)AT_SPLIT_ROWS * mh * 4) != cudaSuccess) rc = fail(DN_ECUDA, "memset failed");
   if (rc == DN_OK && cudaMemset(m->tc_err, 0, 16) != cudaSuccess) rc = fail(DN_ECUDA, "memset failed");
   if (rc == DN_OK && cfg->dtype == DN_SEQ_BF16) {
     make_xmaps(&m->x_h, m->h, m->MB, cfg->width);
@@ -756,6 +760,34 @@ static cudaError_t attn_tiles(cudaStream_t s, const Batch& b, const bf16* q, con
   AT(2, 0, 128, 32) AT(2, 1, 128, 64) AT(2, 2, 128, 128)
 #undef AT
   return cudaErrorInvalidValue;
+}
+
+// few rows: the latency form (k_attn_rows) where the head sizes fit it.  Two stages a warp where a row's keys can exceed what the
+// splits take in one tile a warp.  A function of the model's sizes only, but for the number of rows the scratch holds.
+template <class T>
+static int attn_rows_stages(const dn_seq_layer_cfg& lc, int N) {      // 0: not this kernel
+  const int esz = (int)sizeof(T);
+  if (N > AT_SPLIT_ROWS || lc.pool > 0 || lc.dim > 128 || lc.vdim > 128 || (lc.dim * esz) % 16 || (lc.vdim * esz) % 16) return 0;
+  const bool one = lc.chunk > 0 && lc.chunk <= AT_MAX_SPLITS * AR_KEYS;
+  for (int st = one ? 1 : 2; st > 0; st--)
+    if (ar_smem_bytes(lc.dim, lc.vdim, esz, lc.v_is_k != 0, st) + 1024 <= g_max_smem) return st;
+  return 0;
+}
+template <class T, bool SIG>
+static cudaError_t attn_rows_launch(dn_seq_model* m, cudaStream_t s, const Batch& b, const T* q, const T* kp, const T* vp, const dn_seq_layer_cfg& lc, const AttnExtra& ex,
+                                    int stages, T* out) {
+  const size_t smem = ar_smem_bytes(lc.dim, lc.vdim, (int)sizeof(T), lc.v_is_k != 0, stages);
+  static size_t attr = 40 * 1024;      // (the default limit counts the static part too)
+  if (smem > attr) {
+    cudaError_t e = cudaFuncSetAttribute(k_attn_rows<T, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return e;
+    attr = smem;
+  }
+  const int R = lc.heads / lc.kv_heads, per = (R + AR_HEADS - 1) / AR_HEADS;
+  // (a mask of `chunk` positions bounds the keys of a row, and with them its splits)
+  const int Z = lc.chunk > 0 ? std::min((int)AT_MAX_SPLITS, (lc.chunk + AR_KEYS - 1) / AR_KEYS) : AT_MAX_SPLITS;
+  return launch(k_attn_rows<T, SIG>, dim3(b.N, lc.kv_heads * per, Z), dim3(AR_WARPS * 32), smem, s, b, q, kp, vp, lc.heads, lc.kv_heads, lc.dim, lc.vdim, lc.chunk,
+                lc.scale, stages, ex, out, m->attn_part, m->attn_count);
 }
 
 // latent attention of a step that brings a prompt portion, bf16: the MMA tiles over the cached rows (R + rot numbers a key,
@@ -1119,6 +1151,9 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
       PH(DN_SEQ_PH_ATTN);
       if (attn_tiles_ok<T>(lc, b))
         CK(attn_tiles(s, b, (const bf16*)m->qb, (const bf16*)m->kpool[run.kv_index], (const bf16*)vpl, lc, ex, (bf16*)m->mo));
+      else if (const int st = attn_rows_stages<T>(lc, N))
+        CK(ex.off ? attn_rows_launch<T, true>(m, s, b, (const T*)m->qb, (const T*)m->kpool[run.kv_index], (const T*)vpl, lc, ex, st, (T*)m->mo)
+                  : attn_rows_launch<T, false>(m, s, b, (const T*)m->qb, (const T*)m->kpool[run.kv_index], (const T*)vpl, lc, ex, st, (T*)m->mo));
       else {
         // a small step (decode): long rows are split over up to AT_MAX_SPLITS blocks, joined by k_attn_merge
         // (a mask of `chunk` positions bounds the keys of a row, and with them its splits)

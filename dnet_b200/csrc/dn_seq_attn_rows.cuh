@@ -1,0 +1,219 @@
+// dn_seq_attn_rows.cuh -- attention of a step with few rows (decode steps and small portions), libdnet_b200_seq.so.
+//
+// What k_attn computes, arranged for latency: a block takes one token, up to AR_HEADS query heads of one key / value head
+// and every nz-th run of 128 keys; each of its four warps stages a tile of 32 keys *and* their values in shared memory by
+// asynchronous copies -- one trip to memory after the block table, whole rows, read once for all the block's heads -- and
+// works from there: a lane scores one key, then owns ceil(dv / 32) adjacent output dims.  The warps' partials join in warp
+// order; rows with several splits leave theirs in scratch, and the last block of a row to finish (an atomic count, nobody
+// waits) joins them in split order.  A row's split, tiles and order of sums depend on its own position only.
+// Head sizes up to 128 whose rows start on 16-byte boundaries; no pooled blocks (k_attn does those).
+#pragma once
+#include "dn_seq_kernels.cuh"
+
+namespace dnseq {
+
+constexpr int AR_WARPS = 4, AR_HEADS = 4, AR_KEYS = AR_WARPS * 32;
+__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
+  const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src) : "memory");
+}
+// bytes of one tile (32 keys and values): key rows are padded by 16 bytes, so that the lanes' 16-byte reads of one column
+// of 32 rows fall into different banks
+__host__ __device__ __forceinline__ size_t ar_tile_bytes(int dk, int dv, int esz, bool vk) { return (size_t)32 * (dk * esz + 16) + (vk ? 0 : (size_t)32 * dv * esz); }
+__host__ __device__ __forceinline__ size_t ar_smem_bytes(int dk, int dv, int esz, bool vk, int stages) {
+  const size_t part = (size_t)AR_WARPS * AR_HEADS * (2 + (dv + 31) / 32 * 32) * 4;
+  return (size_t)AR_HEADS * dk * 4 + ((part + 15) & ~(size_t)15) + (size_t)AR_WARPS * stages * ar_tile_bytes(dk, dv, esz, vk);
+}
+__device__ __forceinline__ int ar_splits(int keys, int zmax) { return min(zmax, max(1, (keys + AR_KEYS - 1) / AR_KEYS)); }
+
+template <class T, bool SIG>
+__global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* __restrict__ q, const T* __restrict__ kpool, const T* __restrict__ vpool, int H,
+                                                             int G, int dk, int dv, int chunk, float scale, int stages, AttnExtra ex, T* __restrict__ out,
+                                                             float* __restrict__ part_g, unsigned int* __restrict__ count) {
+  extern __shared__ __align__(16) unsigned char smb[];
+  __shared__ uint32_t rows_s[AR_WARPS][32];
+  __shared__ bool last_s;
+  constexpr int V = Vec16<T>::n, ESZ = (int)sizeof(T);
+  const int VPL = (dv + 31) / 32, dvp = VPL * 32, PL = 2 + dvp;
+  float* qs = reinterpret_cast<float*>(smb);                       // [AR_HEADS][dk]
+  float* part = qs + AR_HEADS * dk;                                // [AR_WARPS][AR_HEADS][2 + dvp]
+  unsigned char* tiles = smb + (size_t)AR_HEADS * dk * 4 + (((size_t)AR_WARPS * AR_HEADS * PL * 4 + 15) & ~(size_t)15);
+  const int n = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int R = H / G, per = (R + AR_HEADS - 1) / AR_HEADS;        // heads of a key head; blocks they take
+  const int g = blockIdx.y / per, h0 = g * R + (blockIdx.y % per) * AR_HEADS, nh = min(AR_HEADS, (g + 1) * R - h0);
+  const int slot = b.slot[n], p = b.pos[n];
+  const int lo = attn_lo(p, chunk, ex.window), nkeys = p - lo + 1;
+  const int zmax = gridDim.z, nz = ar_splits(nkeys, zmax), z = blockIdx.z;
+  if (z >= nz) return;
+  const bool vk = vpool == kpool;
+  const int Ck = G * dk, Cv = ex.v_ld > 0 ? ex.v_ld : G * dv;
+  const int ldk = dk * ESZ + 16, ldv_ = vk ? ldk : dv * ESZ;       // row strides of a tile in bytes
+  const size_t tile_b = ar_tile_bytes(dk, dv, ESZ, vk);
+  unsigned char* mine = tiles + (size_t)warp * stages * tile_b;
+  const int32_t* bt = b.bt + (size_t)slot * b.max_pages;
+  const int step = nz * AR_KEYS, first = (z * AR_WARPS + warp) * 32;
+  auto stage = [&](int s, int j0) {      // this warp's tile at key j0 into buffer s
+    unsigned char* kt = mine + (size_t)s * tile_b;
+    unsigned char* vt = vk ? kt : kt + (size_t)32 * ldk;
+    const int cnt = min(32, nkeys - j0);
+    if (lane < cnt) {
+      const int j = lo + j0 + lane;
+      rows_s[warp][lane] = (uint32_t)bt[j / PAGE] * PAGE + (uint32_t)(j % PAGE);
+    }
+    __syncwarp();
+    const int ck = dk * ESZ / 16, cv = vk ? 0 : dv * ESZ / 16;
+    for (int e = lane; e < cnt * ck; e += 32) {
+      const int r = e / ck, c = e - r * ck;
+      cp_async16(kt + (size_t)r * ldk + c * 16, kpool + (size_t)rows_s[warp][r] * Ck + g * dk + c * V);
+    }
+    for (int e = lane; e < cnt * cv; e += 32) {
+      const int r = e / cv, c = e - r * cv;
+      cp_async16(vt + (size_t)r * ldv_ + c * 16, vpool + (size_t)rows_s[warp][r] * Cv + g * dv + c * V);
+    }
+    cp_async_commit();
+    __syncwarp();
+  };
+  if (first < nkeys) stage(0, first);
+  for (int e = threadIdx.x; e < AR_HEADS * dk; e += blockDim.x) qs[e] = e < nh * dk ? ldf(q + ((size_t)n * H + h0) * dk + e) : 0.f;
+  float r1[AR_HEADS], r2[AR_HEADS], soff[AR_HEADS];
+#pragma unroll
+  for (int i = 0; i < AR_HEADS; i++) {
+    const int h = h0 + min(i, nh - 1);
+    r1[i] = ex.r1 ? ldf((const T*)ex.r1 + h) : 0.f;
+    r2[i] = ex.r1 ? ldf((const T*)ex.r2 + h) : 0.f;
+    soff[i] = SIG ? ldf((const T*)ex.off + h) : 0.f;
+  }
+  __syncthreads();
+  float m[AR_HEADS], l[AR_HEADS], acc[AR_HEADS][4];
+#pragma unroll
+  for (int i = 0; i < AR_HEADS; i++) {
+    m[i] = -INFINITY; l[i] = 0.f;
+#pragma unroll
+    for (int x = 0; x < 4; x++) acc[i][x] = 0.f;
+  }
+  const int vcnt = min(VPL, max(0, dv - lane * VPL));
+  int s = 0;
+  for (int j0 = first; j0 < nkeys; j0 += step) {
+    const bool more = j0 + step < nkeys;
+    if (more && stages > 1) { stage(s ^ 1, j0 + step); cp_async_wait<1>(); }
+    else cp_async_wait<0>();
+    __syncwarp();
+    const unsigned char* kt = mine + (size_t)s * tile_b;
+    const unsigned char* vt = vk ? kt : kt + (size_t)32 * ldk;
+    const int cnt = min(32, nkeys - j0), j = j0 + lane;
+    float sc[AR_HEADS] = {0.f, 0.f, 0.f, 0.f};
+    if (lane < cnt) {
+      const T* kr = reinterpret_cast<const T*>(kt + (size_t)lane * ldk);
+#pragma unroll 4
+      for (int d = 0; d < dk; d += V) {
+        float kv[V];
+        ldv(kr + d, kv);
+#pragma unroll
+        for (int i = 0; i < AR_HEADS; i++) {
+#pragma unroll
+          for (int x = 0; x < V; x += 4) {
+            const float4 q4 = *reinterpret_cast<const float4*>(qs + i * dk + d + x);
+            sc[i] = fmaf(q4.x, kv[x], sc[i]); sc[i] = fmaf(q4.y, kv[x + 1], sc[i]);
+            sc[i] = fmaf(q4.z, kv[x + 2], sc[i]); sc[i] = fmaf(q4.w, kv[x + 3], sc[i]);
+          }
+        }
+      }
+    }
+    float pw[AR_HEADS];
+#pragma unroll
+    for (int i = 0; i < AR_HEADS; i++) {
+      float a = sc[i] * scale;
+      if (ex.softcap > 0.f) a = ex.softcap * tanhf(a / ex.softcap);
+      if (ex.r1) a -= r1[i] * log1pf(r2[i] * (float)max(0, nkeys - 1 - j));
+      if (SIG) { pw[i] = lane < cnt ? sigmoid_f(a + soff[i]) : 0.f; continue; }
+      a = lane < cnt ? a : -INFINITY;
+      const float mn = fmaxf(m[i], warp_max(a)), corr = expf(m[i] - mn);
+      pw[i] = lane < cnt ? expf(a - mn) : 0.f;
+      l[i] = l[i] * corr + warp_sum(pw[i]);
+#pragma unroll
+      for (int x = 0; x < 4; x++) acc[i][x] *= corr;
+      m[i] = mn;
+    }
+#pragma unroll 4
+    for (int t = 0; t < cnt; t++) {
+      const T* vr = reinterpret_cast<const T*>(vt + (size_t)t * ldv_) + lane * VPL;
+      float v[4] = {0.f, 0.f, 0.f, 0.f};
+      if (VPL == 4 && vcnt == 4 && (dv & 3) == 0) ld4(vr, v);
+      else {
+#pragma unroll
+        for (int x = 0; x < 4; x++) if (x < vcnt) v[x] = ldf(vr + x);
+      }
+#pragma unroll
+      for (int i = 0; i < AR_HEADS; i++) {
+        const float pt = __shfl_sync(0xffffffffu, pw[i], t);
+#pragma unroll
+        for (int x = 0; x < 4; x++) acc[i][x] = fmaf(pt, v[x], acc[i][x]);
+      }
+    }
+    __syncwarp();
+    if (stages > 1) s ^= 1;
+    else if (more) stage(0, j0 + step);
+  }
+#pragma unroll
+  for (int i = 0; i < AR_HEADS; i++) {
+    float* pr = part + ((size_t)warp * AR_HEADS + i) * PL;
+    if (lane == 0) { pr[0] = m[i]; pr[1] = l[i]; }
+#pragma unroll
+    for (int x = 0; x < 4; x++) if (x < VPL) pr[2 + lane * VPL + x] = acc[i][x];
+  }
+  __syncthreads();
+  const bool split = nz > 1;
+  // head i's output from `cnt` partials at stride `st` floats (shared memory, or scratch written by other blocks: read past L1)
+  auto finish = [&](int i, int d, const float* pr, size_t st, int cnt, bool global) {
+    auto rd = [&](const float* a) { return global ? __ldcg(a) : *a; };
+    const int h = h0 + i;
+    const float og = ex.gate ? sigmoid_f(ex.gate[(size_t)n * H + h]) : 1.f;
+    float a = 0.f;
+    if (SIG) {
+      for (int w = 0; w < cnt; w++) a += rd(pr + w * st + 2 + d);
+      stf(out + ((size_t)n * H + h) * dv + d, a * og);
+      return;
+    }
+    const float snk = ex.sink ? ldf((const T*)ex.sink + h) : -INFINITY;
+    float M = snk;
+    for (int w = 0; w < cnt; w++) M = fmaxf(M, rd(pr + w * st));
+    float L = ex.sink ? expf(snk - M) : 0.f;
+    for (int w = 0; w < cnt; w++) {
+      const float f = expf(rd(pr + w * st) - M);      // a warp without a tile has maximum -inf and weight 0
+      L += rd(pr + w * st + 1) * f;
+      a += rd(pr + w * st + 2 + d) * f;
+    }
+    stf(out + ((size_t)n * H + h) * dv + d, a / L * og);
+  };
+  if (!split) {
+    for (int e = threadIdx.x; e < nh * dv; e += blockDim.x) finish(e / dv, e % dv, part + (size_t)(e / dv) * PL, (size_t)AR_HEADS * PL, AR_WARPS, false);
+    return;
+  }
+  for (int e = threadIdx.x; e < nh * dv; e += blockDim.x) {
+    const int i = e / dv, d = e % dv;
+    const float* pr = part + (size_t)i * PL;
+    float* pg = part_g + (((size_t)n * H + h0 + i) * zmax + z) * PL;
+    float M = -INFINITY, L = 0.f, a = 0.f;
+    if (!SIG)
+      for (int w = 0; w < AR_WARPS; w++) M = fmaxf(M, pr[(size_t)w * AR_HEADS * PL]);
+    for (int w = 0; w < AR_WARPS; w++) {
+      const float* pq = pr + (size_t)w * AR_HEADS * PL;
+      const float f = SIG ? 1.f : expf(pq[0] - M);
+      if (!SIG) L += pq[1] * f;
+      a += pq[2 + d] * f;
+    }
+    pg[2 + d] = a;
+    if (d == 0) { pg[0] = M; pg[1] = L; }
+  }
+  __threadfence();
+  __syncthreads();
+  if (threadIdx.x == 0) last_s = atomicAdd(count + (size_t)n * gridDim.y + blockIdx.y, 1u) == (unsigned)nz - 1;
+  __syncthreads();
+  if (!last_s) return;
+  __threadfence();
+  if (threadIdx.x == 0) count[(size_t)n * gridDim.y + blockIdx.y] = 0;      // ready for the next launch
+  for (int e = threadIdx.x; e < nh * dv; e += blockDim.x)
+    finish(e / dv, e % dv, part_g + ((size_t)n * H + h0 + e / dv) * zmax * PL, (size_t)PL, nz, true);
+}
+
+}  // namespace dnseq
