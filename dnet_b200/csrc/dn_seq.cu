@@ -8,6 +8,7 @@
 #include "dn_seq_latent.cuh"
 #include "dn_seq_gdelta.cuh"
 #include "dn_gemm_tc.cuh"      // the tcgen05 / TMA GEMM the llama-family prefill runs on (namespace dn)
+#include "dn_seq_attn_tc.cuh"
 #include "../../include/dnet_b200_seq.h"
 
 #include <algorithm>
@@ -107,6 +108,10 @@ struct dn_seq_model {
   int max_tiles = 0;
   // state
   std::vector<void*> kpool, vpool;
+  std::vector<CUtensorMap> kmap, vmap;   // TMA descriptors of the pools (boxes of one page x 64 columns), where map_ok
+  std::vector<char> map_ok;
+  float* dist_tab = nullptr;             // [heads][distance]: the tabled bias of the layer whose attention runs (k_dist_table)
+  std::vector<int> ent_len;              // tokens of the current step's entries
   std::vector<void*> pkpool, pvpool;     // mean-pooled blocks behind a sliding window: [pages][pool_rows][row] (null: the run has none)
   std::vector<int> last_tok;             // per slot: the sequence's last token (-1: none yet), for the bigram row
   void* hn = nullptr;                    // the normed rows before the sublayer's input convolution [MB, W]
@@ -186,6 +191,18 @@ static bool make_tmap(CUtensorMap* out, const void* base, int rows, int cols, in
   return g_encode(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
                   CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
+static int dist_span(const dn_seq_cfg& cfg, const dn_seq_layer_cfg& c) {      // distances a visible key can have: 0 .. span - 1
+  int span = cfg.pool_pages * PAGE;
+  if (cfg.max_positions > 0) span = std::min(span, cfg.max_positions);
+  if (c.chunk > 0) span = std::min(span, c.chunk);
+  return span;
+}
+// layers whose prompt portions take k_sig_attn_tc (as far as their sizes go)
+constexpr size_t DIST_TAB_MAX = (size_t)1 << 24;      // floats
+static bool sig_tc_sizes(const dn_seq_cfg& cfg, const dn_seq_layer_cfg& c) {
+  return cfg.dtype == DN_SEQ_BF16 && (c.mixer == DN_MIX_ATTENTION || c.mixer == DN_MIX_PARALLEL) && c.attn_weight == DN_ATTN_SIGMOID && c.softcap <= 0.f && c.pool == 0 &&
+         (c.dim == 64 || c.dim == 128) && (c.vdim == 64 || c.vdim == 128) && (size_t)c.heads * dist_span(cfg, c) <= DIST_TAB_MAX;
+}
 static void make_xmaps(XMaps* x, const void* base, int rows, int cols) {
   x->ok = true;
   const int br[3] = {32, 64, 128};
@@ -205,7 +222,7 @@ extern "C" int dn_seq_model_destroy(dn_seq_model* m) {
   cudaDeviceSynchronize();
   void* ptrs[] = {m->xs, m->y, m->pa, m->pb, m->qn, m->kn, m->vv, m->od, m->beta, m->decay, m->h, m->uq, m->uk, m->uv, m->qb,
                   m->mo, m->gt, m->act, m->conv_state, m->delta_state, m->stage_d, m->bt_d, m->tc_err, m->y2, m->x0, m->dz, m->rwt,
-                  m->eo, m->cat, m->xm, m->lr, m->eact, m->ridx, m->rpos, m->rtok, m->tiles, m->xg, m->attn_part, m->attn_count, m->sgate, m->hn, m->un, m->aun};
+                  m->eo, m->cat, m->xm, m->lr, m->eact, m->ridx, m->rpos, m->rtok, m->tiles, m->xg, m->attn_part, m->attn_count, m->dist_tab, m->sgate, m->hn, m->un, m->aun};
   for (void* p : ptrs) if (p) cudaFree(p);
   for (auto& g : m->graphs) cudaGraphExecDestroy(g.second.first);
   if (m->lg_buf) cudaFree(m->lg_buf);
@@ -430,7 +447,7 @@ extern "C" int dn_seq_model_create(const dn_seq_cfg* cfg, const dn_seq_layer_cfg
     mh = std::max(mh, c.heads);
   }
   // the order of layer runs, and every run's own pages and state
-  size_t coff = 0, doff = 0;
+  size_t coff = 0, doff = 0, tab = 0;
   if (rc == DN_OK) {
     std::vector<std::pair<int, bool>> order;
     for (int i = 0; i < cfg->n_layers; i++) {
@@ -460,8 +477,18 @@ extern "C" int dn_seq_model_create(const dn_seq_cfg* cfg, const dn_seq_layer_cfg
             if ((rc = dalloc(&m->pkpool.back(), rows * l.Ck * m->esz)) != DN_OK) break;
             if ((rc = dalloc(&m->pvpool.back(), rows * l.Cv * m->esz)) != DN_OK) break;
           }
+          CUtensorMap km, vm;
+          memset(&km, 0, sizeof(km));
+          memset(&vm, 0, sizeof(vm));
+          const int prows = cfg->pool_pages * PAGE;
+          const void* vp = c.v_is_k ? m->kpool.back() : m->vpool.back();
+          const bool ok = sig_tc_sizes(*cfg, c) && make_tmap(&km, m->kpool.back(), prows, l.Ck, PAGE) && make_tmap(&vm, vp, prows, c.v_is_k ? l.Ck : l.Cv, PAGE);
+          m->kmap.push_back(km);
+          m->vmap.push_back(vm);
+          m->map_ok.push_back(ok ? 1 : 0);
         }
       }
+      if (sig_tc_sizes(*cfg, c)) tab = std::max(tab, (size_t)c.heads * dist_span(*cfg, c));
       for (int q = 0; q < 2; q++) {
         r.canon_off[q] = coff;
         if (cfg->canon_taps > 1 && (q == 0 || c.ff > 0)) coff += (size_t)(cfg->canon_taps - 1) * cfg->width;
@@ -486,6 +513,7 @@ extern "C" int dn_seq_model_create(const dn_seq_cfg* cfg, const dn_seq_layer_cfg
   DA(m->y2, MB * W * 4); DA(m->dz, MB * mdq * 4); DA(m->lr, MB * mrank * e);
   DA(m->attn_part, (size_t)AT_SPLIT_ROWS * mh * AT_MAX_SPLITS * (2 + m->part_dv) * 4);
   DA(m->attn_count, (size_t)AT_SPLIT_ROWS * mh * 4);
+  if (tab > 0) DA(m->dist_tab, tab * 4);
   DA(m->sgate, MB * 4);
   if (looped) { DA(m->x0, MB * W * 4); DA(m->cat, MB * 2 * W * e); }
   if (any_wkv) DA(m->xm, (size_t)SHIFT_MAX * MB * W * e);
@@ -760,6 +788,32 @@ static cudaError_t attn_tiles(cudaStream_t s, const Batch& b, const bf16* q, con
   AT(2, 0, 128, 32) AT(2, 1, 128, 64) AT(2, 2, 128, 128)
 #undef AT
   return cudaErrorInvalidValue;
+}
+
+// sigmoid weights, prompt portions: a CTA per (block of tokens, key head, up to SG_HEADS of its query heads)
+template <int DK, int DV>
+static cudaError_t sig_attn_launch(dn_seq_model* m, cudaStream_t s, const Batch& b, int kv, const SigParams& p) {
+  constexpr size_t smem = sg_smem(DK, DV);
+  static bool attr = false;
+  if (!attr) {
+    cudaError_t e = cudaFuncSetAttribute(k_sig_attn_tc<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return e;
+    attr = true;
+  }
+  const int TB = 128 / p.hpc, R = p.H / p.G;
+  int blocks = 0;
+  for (int n : m->ent_len) blocks += (n + TB - 1) / TB;
+  g_launches++;
+  k_sig_attn_tc<DK, DV><<<dim3(blocks, p.G * ((R + p.hpc - 1) / p.hpc)), SG_THREADS, smem, s>>>(m->kmap[kv], m->vmap[kv], b, p);
+  return cudaGetLastError();
+}
+static cudaError_t sig_attn(dn_seq_model* m, cudaStream_t s, const Batch& b, int kv, const bf16* q, const dn_seq_layer_cfg& lc, const AttnExtra& ex, bf16* out) {
+  const int D = dist_span(m->cfg, lc);
+  cudaError_t e = launch(k_dist_table, dim3((D + 255) / 256, lc.heads), dim3(256), 0, s, (const bf16*)ex.r1, (const bf16*)ex.r2, (const bf16*)ex.off, D, m->dist_tab);
+  if (e != cudaSuccess) return e;
+  const SigParams p{q, out, m->dist_tab, ex.gate, lc.heads, lc.kv_heads, lc.chunk, ex.window, D, std::min(lc.heads / lc.kv_heads, SG_HEADS), lc.scale, m->tc_err};
+  if (lc.dim == 64) return lc.vdim == 64 ? sig_attn_launch<64, 64>(m, s, b, kv, p) : sig_attn_launch<64, 128>(m, s, b, kv, p);
+  return lc.vdim == 64 ? sig_attn_launch<128, 64>(m, s, b, kv, p) : sig_attn_launch<128, 128>(m, s, b, kv, p);
 }
 
 // few rows: the latency form (k_attn_rows) where the head sizes fit it.  Two stages a warp where a row's keys can exceed what the
@@ -1149,7 +1203,9 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
         CK(launch(k_pool_rows<T>, dim3(N), dim3(128), 0, s, b, lc.pool, Ckk, lc.v_is_k ? 0 : lc.kv_heads * lc.vdim, (const T*)m->kpool[run.kv_index], (const T*)vpl,
                   (T*)pkp, (T*)pvp));
       PH(DN_SEQ_PH_ATTN);
-      if (attn_tiles_ok<T>(lc, b))
+      if (b.max_len >= 16 && m->map_ok[run.kv_index] && sig_tc_sizes(c, lc))
+        CK(sig_attn(m, s, b, run.kv_index, (const bf16*)m->qb, lc, ex, (bf16*)m->mo));
+      else if (attn_tiles_ok<T>(lc, b))
         CK(attn_tiles(s, b, (const bf16*)m->qb, (const bf16*)m->kpool[run.kv_index], (const bf16*)vpl, lc, ex, (bf16*)m->mo));
       else if (const int st = attn_rows_stages<T>(lc, N))
         CK(ex.off ? attn_rows_launch<T, true>(m, s, b, (const T*)m->qb, (const T*)m->kpool[run.kv_index], (const T*)vpl, lc, ex, st, (T*)m->mo)
@@ -1566,6 +1622,7 @@ extern "C" int dn_seq_step(dn_seq_model* m, int E, const int32_t* slots, const i
   CK(cudaMemcpyAsync(m->stage_d, h, ints * 4, cudaMemcpyHostToDevice, s));
   CK(cudaEventRecord(m->staged, s));
   int32_t* d = m->stage_d;
+  m->ent_len.assign(counts, counts + E);
   int max_len = 0, row_tiles = 0;
   for (int e = 0; e < E; e++) { max_len = counts[e] > max_len ? counts[e] : max_len; row_tiles += (counts[e] + AT_ROWS - 1) / AT_ROWS; }
   Batch b{d, d + N, d + 2 * N, d + 3 * N, d + 5 * N, d + 5 * N + E + 1, d + 5 * N + 2 * E + 1, m->bt_d, N, E, m->max_pages, max_len, row_tiles, d + 4 * N};

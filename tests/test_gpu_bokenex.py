@@ -240,6 +240,33 @@ def test_sizes_that_allow_no_wide_loads(dtype):
         assert off(dtype)(run_schedule(rig, t, [70, 2, 20]), ref) < TOL[dtype]
 
 
+@pytest.mark.parametrize("H,G,dk,dv,size", [(1, 1, 64, 64, 50), (4, 2, 128, 64, 200), (6, 2, 64, 128, 64), (6, 1, 128, 128, 65), (16, 1, 64, 64, 33),
+                                            (20, 1, 64, 64, 300), (8, 8, 64, 64, None), (34, 2, 64, 128, 130), (4, 1, 128, 128, 1)])
+def test_prompt_attention_on_tcgen05(H, G, dk, dv, size):
+    """heads of 64 / 128: one, some and more than 16 query heads a key head (token blocks of 128 down to 8), windows of one token, about
+    a page, several tiles and none; whole, in portions that start inside pages and tiles, and unequal entries side by side"""
+    cfg = config([att(size=size, heads=H, kv_heads=G, dim=dk, vdim=dv, scale=1.5 * dk ** -0.5, conv=2)], width=64)
+    t = toks(330, seed=500 + H)
+    with Rig(cfg, "bfloat16", max_tokens=2048, max_batch_tokens=1024) as rig:
+        ref = rig.oracle(t)
+        assert err16(run_schedule(rig, t, [330]), ref) < TOL["bfloat16"]
+        assert err16(run_schedule(rig, t, [37, 16, 2, 90, 129, 50]), ref) < TOL["bfloat16"]
+        rig.eng.step([("a", t[:100], []), ("b", t[:20], [])])
+        lg = rig.eng.step([("a", t[100:231], list(range(131))), ("b", t[20:21], [0]), ("c", t[:17], list(range(17)))])
+        assert err16(lg, torch.cat([ref[100:231], ref[20:21], ref[:17]])) < TOL["bfloat16"]
+
+
+def test_prompt_attention_in_pages_that_were_used():
+    """the last page of a prompt holds rows of the request that had it before: they must not enter (values four times as large)"""
+    cfg = config([att(DENSE, size=200, heads=4, kv_heads=2, dim=64, vdim=64, scale=0.15)], width=64)
+    w = bo.random_weights(cfg, 520)
+    w["l0.mix.v"] = w["l0.mix.v"] * 4
+    with Rig(cfg, "bfloat16", weights=w, max_tokens=256, max_seqs=2) as rig:
+        for n, k in ((250, 0), (17, 1), (70, 2), (129, 3), (190, 4)):
+            t = toks(n, seed=521 + k)
+            assert err16(run_schedule(rig, t, [n]), rig.oracle(t)) < TOL["bfloat16"]
+
+
 LAYER_SIZED = {
     "w384": config([att({"kind": "dense", "ff": 640}, size=90, heads=6, kv_heads=2, dim=64, vdim=48, scale=0.11, conv=4),
                     att(moe(6, 2, 2.0, 128), size=40, heads=12, kv_heads=4, dim=32, vdim=32, conv=4),
@@ -396,10 +423,10 @@ def opposite_setup(layer, seed, vocab=64):
     return cfg, w
 
 
-def edge_setup(size, token_marks=(0, 40, 64, 104, 127, 170)):
+def edge_setup(size, token_marks=(0, 40, 64, 104, 127, 170), dk=32, dv=16):
     """token 63 stands at every position of `token_marks`, token 62 at mark + size - 1 (it just sees the 63) and at mark + size
     (it just does not); all other tokens are below 62"""
-    cfg, w = opposite_setup(att(size=size, heads=2, kv_heads=1, dim=32, vdim=16, scale=0.5), 70 + size)
+    cfg, w = opposite_setup(att(size=size, heads=2, kv_heads=1, dim=dk, vdim=dv, scale=16.0 / dk), 70 + size)
     n = max(token_marks) + size + 8
     g = torch.Generator().manual_seed(71 + size)
     t = torch.randint(0, 62, (n,), generator=g).tolist()
@@ -414,12 +441,13 @@ def edge_setup(size, token_marks=(0, 40, 64, 104, 127, 170)):
     return cfg, w, t, sorted(set(rows))
 
 
+@pytest.mark.parametrize("dk,dv", [(32, 16), (64, 64)])      # the warp-level tiles, the tcgen05 kernel
 @pytest.mark.parametrize("size", [24, 64, 65, 40, 129])
-def test_keys_just_inside_and_just_outside_the_window(size, monkeypatch):
+def test_keys_just_inside_and_just_outside_the_window(size, dk, dv, monkeypatch):
     """marks at the sequence's start (the first tokens a window keeps and loses), in the middle of pages and where an edge
     falls on a page border; a window that is one token off in either direction changes the marked rows by far more than the
     tolerance.  In prompts (cut at, before and after the edges) and decoded one by one, fp32 and bf16."""
-    cfg, w, t, rows = edge_setup(size)
+    cfg, w, t, rows = edge_setup(size, dk=dk, dv=dv)
     ref = bo.forward(cfg, w, t)
     real = bo.visible
     for d in (-1, 1):
@@ -438,12 +466,13 @@ def test_keys_just_inside_and_just_outside_the_window(size, monkeypatch):
             assert e(got, ref) < TOL[dtype] and e(got[rows], ref[rows]) < TOL[dtype]
 
 
+@pytest.mark.parametrize("dk,dv", [(32, 16), (64, 128)])
 @pytest.mark.parametrize("size", [None, 704])
-def test_far_key_among_hundreds(size):
+def test_far_key_among_hundreds(size, dk, dv):
     """the marked token at position 3 is seen from 700 positions on, through the prompt kernels and through decode rows split
     over several blocks"""
     n = 706
-    cfg, w = opposite_setup(att(size=size, heads=2, kv_heads=1, dim=32, vdim=16, scale=0.5), 170)
+    cfg, w = opposite_setup(att(size=size, heads=2, kv_heads=1, dim=dk, vdim=dv, scale=16.0 / dk), 170)
     g = torch.Generator().manual_seed(171)
     t = torch.randint(0, 62, (n,), generator=g).tolist()
     t[3] = 63
@@ -460,12 +489,13 @@ def test_far_key_among_hundreds(size):
                 assert off(dtype)(got, ref) < TOL[dtype] and off(dtype)(got[-6:], ref[-6:]) < TOL[dtype]
 
 
-def test_distance_bias_and_offset_show(monkeypatch):
+@pytest.mark.parametrize("d", [16, 64])
+def test_distance_bias_and_offset_show(d, monkeypatch):
     """equal scores everywhere (zero queries): a key's weight is sigmoid(offset - r1 ln(1 + r2 d)) alone, so a distance that is
     one off, a bias without its logarithm or a lost offset shows in every row"""
-    cfg = config([att(size=90, heads=3, kv_heads=1, dim=16, vdim=16, conv=2)])
+    cfg = config([att(size=90, heads=3, kv_heads=1, dim=d, vdim=d, conv=2)])
     w = bo.random_weights(cfg, 61)
-    w["l0.mix.q.norm"] = torch.zeros(16)
+    w["l0.mix.q.norm"] = torch.zeros(d)
     w["l0.mix.r1"] = torch.tensor([2.5, 0.75, 1.5])
     w["l0.mix.r2"] = torch.tensor([0.125, 4.0, 0.015625])
     w["l0.mix.pb"] = torch.tensor([1.0, -0.5, -2.0])
@@ -484,9 +514,10 @@ def test_distance_bias_and_offset_show(monkeypatch):
             assert off(dtype)(run_schedule(rig, t, [60, 2, 50, 33]), ref) < TOL[dtype]
 
 
-def test_weights_far_from_one_half():
+@pytest.mark.parametrize("d", [16, 64])
+def test_weights_far_from_one_half(d):
     """offsets that push the sigmoids to both ends: weights near zero do not overflow, weights near one do not sum to one"""
-    cfg = config([att(size=80, heads=3, kv_heads=1, dim=16, vdim=16, scale=2.0)])
+    cfg = config([att(size=80, heads=3, kv_heads=1, dim=d, vdim=d, scale=2.0)])
     w = bo.random_weights(cfg, 63)
     w["l0.mix.pb"] = torch.tensor([40.0, -40.0, -120.0])
     t = toks(150, seed=64)
