@@ -513,7 +513,7 @@ extern "C" int dn_seq_model_create(const dn_seq_cfg* cfg, const dn_seq_layer_cfg
   DA(m->y2, MB * W * 4); DA(m->dz, MB * mdq * 4); DA(m->lr, MB * mrank * e);
   DA(m->attn_part, (size_t)AT_SPLIT_ROWS * mh * AT_MAX_SPLITS * (2 + m->part_dv) * 4);
   DA(m->attn_count, (size_t)AT_SPLIT_ROWS * mh * 4);
-  if (tab > 0) DA(m->dist_tab, tab * 4);
+  if (tab > 0) DA(m->dist_tab, (tab + 32) * 4);      // (rows without a query read up to 32 entries whatever the span)
   DA(m->sgate, MB * 4);
   if (looped) { DA(m->x0, MB * W * 4); DA(m->cat, MB * 2 * W * e); }
   if (any_wkv) DA(m->xm, (size_t)SHIFT_MAX * MB * W * e);

@@ -7,19 +7,19 @@
 // tokens, so that a staged key / value tile serves the whole group.  Per tile of 128 keys (two pages, by TMA through the
 // block table):
 //   S = Q K^T       A = Q [128 x DK] K-major, B = K tile [128 x DK] K-major          TMEM columns 0-127 / 128-255 in turn
-//   P = weights     eight warps, two per TMEM lane quarter (each takes half of the columns): one score = one fused
+//   P = weights     sixteen warps, four per TMEM lane quarter (a quarter of the columns each): one score = one fused
 //                   multiply-add with the tabled bias, one exponential, half a reciprocal (two weights share one)
 //   O += P V        A = P as a bf16 pair hi + lo (16 bits of each weight's mantissa), B = V tile, MN-major     TMEM 256-383
-// S of tile j + 1 is formed while the weights of tile j are; K has two buffers, V and P one each.
+// S of tile j + 1 is formed while the weights of tile j are; S, K and V have two buffers each, P one.
 // Per row the tiles are visited in ascending position; a tile that a row does not see adds zeros.
-// Roles: warp 0 TMA producer, warp 1 MMA issuer, warp 2 TMEM allocator, warps 4-11 weights and output.
+// Roles: warp 0 TMA producer, warp 1 MMA issuer, warp 2 TMEM allocator, warps 4-19 weights and output.
 #pragma once
 #include "dn_gemm_tc.cuh"
 #include "dn_seq_kernels.cuh"
 
 namespace dnseq {
 
-constexpr int SG_HEADS = 16, SG_THREADS = 384, SG_HALF = 16384;      // SG_HALF: bytes of 128 rows x 64 columns
+constexpr int SG_HEADS = 16, SG_THREADS = 640, SG_HALF = 16384;      // SG_HALF: bytes of 128 rows x 64 columns
 constexpr float SG_LOG2E = 1.4426950408889634f;
 
 struct SigParams {
@@ -32,6 +32,24 @@ struct SigParams {
   unsigned int* err;
 };
 
+// exponential and reciprocal of the special-function unit (a few units in the last place of fp32, far inside what the bf16
+// operands carry)
+__device__ __forceinline__ float sg_ex2(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
+__device__ __forceinline__ float sg_rcp(float x) { float y; asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
+// 32 lanes x 32 consecutive fp32 columns of this warp's TMEM quarter
+__device__ __forceinline__ void sg_ld32(uint32_t taddr, float (&v)[32]) {
+  uint32_t r[32];
+  asm volatile(
+      "tcgen05.ld.sync.aligned.32x32b.x32.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"
+      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]),
+        "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]), "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]),
+        "=r"(r[23]), "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
+      : "r"(taddr));
+  asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+#pragma unroll
+  for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
+}
+
 // tab[h][d] = (r1_h ln(1 + r2_h d) - off_h) log2(e)
 __global__ void k_dist_table(const bf16* __restrict__ r1, const bf16* __restrict__ r2, const bf16* __restrict__ off, int D, float* __restrict__ tab) {
   const int h = blockIdx.y, d = blockIdx.x * blockDim.x + threadIdx.x;
@@ -40,18 +58,18 @@ __global__ void k_dist_table(const bf16* __restrict__ r1, const bf16* __restrict
   tab[(size_t)h * D + d] = (b - ldf(off + h)) * SG_LOG2E;
 }
 
-__host__ __device__ constexpr size_t sg_smem(int DK, int DV) { return (size_t)(3 * (DK / 64) + DV / 64 + 4) * SG_HALF + 1024 + 256; }
+__host__ __device__ constexpr size_t sg_smem(int DK, int DV) { return (size_t)(3 * (DK / 64) + 2 * (DV / 64) + 4) * SG_HALF + 1024 + 256; }
 
 template <int DK, int DV>
 __global__ void __launch_bounds__(SG_THREADS, 1) k_sig_attn_tc(const __grid_constant__ CUtensorMap mapK, const __grid_constant__ CUtensorMap mapV, Batch b, SigParams p) {
   constexpr int KB = DK / 64 * SG_HALF, VB = DV / 64 * SG_HALF;      // bytes of a K (Q) and a V tile
   extern __shared__ __align__(1024) unsigned char sg_raw[];
   unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(sg_raw) + 1023) & ~(uintptr_t)1023);
-  unsigned char *sQ = smem, *sK = sQ + KB, *sV = sK + 2 * KB, *sPh = sV + VB, *sPl = sPh + 2 * SG_HALF;
+  unsigned char *sQ = smem, *sK = sQ + KB, *sV = sK + 2 * KB, *sPh = sV + 2 * VB, *sPl = sPh + 2 * SG_HALF;
   uint64_t* bars = reinterpret_cast<uint64_t*>(sPl + 2 * SG_HALF);
-  uint64_t *k_full = bars, *k_empty = bars + 2, *s_full = bars + 4, *s_empty = bars + 6, *v_full = bars + 8, *v_empty = bars + 9, *p_full = bars + 10,
-           *p_empty = bars + 11, *o_full = bars + 12;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 13);
+  uint64_t *k_full = bars, *k_empty = bars + 2, *s_full = bars + 4, *s_empty = bars + 6, *v_full = bars + 8, *v_empty = bars + 10, *p_full = bars + 12,
+           *p_empty = bars + 13, *o_full = bars + 14;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 15);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   // which entry, which of its blocks of TB tokens, which heads
   const int TB = 128 / p.hpc;
@@ -69,8 +87,12 @@ __global__ void __launch_bounds__(SG_THREADS, 1) k_sig_attn_tc(const __grid_cons
   const int page0 = attn_lo(p_first, p.chunk, p.window) / PAGE, pages = (kv_max + PAGE - 1) / PAGE, n_tiles = (pages - page0 + 1) / 2;
 
   if (threadIdx.x == 0) {
-    for (int i = 0; i < 2; i++) { dn::mbar_init(&k_full[i], 1); dn::mbar_init(&k_empty[i], 1); dn::mbar_init(&s_full[i], 1); dn::mbar_init(&s_empty[i], 8); }
-    dn::mbar_init(v_full, 1); dn::mbar_init(v_empty, 1); dn::mbar_init(p_full, 8); dn::mbar_init(p_empty, 1); dn::mbar_init(o_full, 1);
+    constexpr int WW = SG_THREADS / 32 - 4;      // warps that form weights
+    for (int i = 0; i < 2; i++) {
+      dn::mbar_init(&k_full[i], 1); dn::mbar_init(&k_empty[i], 1); dn::mbar_init(&s_full[i], 1); dn::mbar_init(&s_empty[i], WW);
+      dn::mbar_init(&v_full[i], 1); dn::mbar_init(&v_empty[i], 1);
+    }
+    dn::mbar_init(p_full, WW); dn::mbar_init(p_empty, 1); dn::mbar_init(o_full, 1);
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
   if (warp == 2) {
@@ -106,14 +128,15 @@ __global__ void __launch_bounds__(SG_THREADS, 1) k_sig_attn_tc(const __grid_cons
           }
         }
         if (j > 0) {
-          const int jv = j - 1;
+          const int jv = j - 1, st = jv & 1;
+          unsigned char* dst = sV + st * VB;
           const int pg0 = bt[page0 + 2 * jv], pg1 = page0 + 2 * jv + 1 < pages ? bt[page0 + 2 * jv + 1] : pg0;
-          dn::mbar_wait(v_empty, (jv & 1) ^ 1u, p.err);
-          dn::mbar_arrive_expect_tx(v_full, VB);
+          dn::mbar_wait(&v_empty[st], ((jv >> 1) & 1) ^ 1u, p.err);
+          dn::mbar_arrive_expect_tx(&v_full[st], VB);
 #pragma unroll
           for (int hf = 0; hf < DV / 64; hf++) {
-            dn::tma_load_2d(sV + hf * SG_HALF, &mapV, g * DV + hf * 64, pg0 * PAGE, v_full);
-            dn::tma_load_2d(sV + hf * SG_HALF + SG_HALF / 2, &mapV, g * DV + hf * 64, pg1 * PAGE, v_full);
+            dn::tma_load_2d(dst + hf * SG_HALF, &mapV, g * DV + hf * 64, pg0 * PAGE, &v_full[st]);
+            dn::tma_load_2d(dst + hf * SG_HALF + SG_HALF / 2, &mapV, g * DV + hf * 64, pg1 * PAGE, &v_full[st]);
           }
         }
       }
@@ -138,11 +161,11 @@ __global__ void __launch_bounds__(SG_THREADS, 1) k_sig_attn_tc(const __grid_cons
           dn::tc_commit(&s_full[st]);
         }
         if (j > 0) {
-          const uint32_t ph = (j - 1) & 1;
-          dn::mbar_wait(p_full, ph, p.err);
-          dn::mbar_wait(v_full, ph, p.err);
+          const int st = (j - 1) & 1;
+          dn::mbar_wait(p_full, st, p.err);
+          dn::mbar_wait(&v_full[st], ((j - 1) >> 1) & 1, p.err);
           dn::tc_fence_after();
-          const uint64_t vd = dn::tc_smem_desc_mn(sV, SG_HALF, 1024);
+          const uint64_t vd = dn::tc_smem_desc_mn(sV + st * VB, SG_HALF, 1024);
 #pragma unroll
           for (int part = 0; part < 2; part++) {
 #pragma unroll
@@ -151,72 +174,71 @@ __global__ void __launch_bounds__(SG_THREADS, 1) k_sig_attn_tc(const __grid_cons
               dn::tc_mma(tO, ad, vd + (uint64_t)(kk * (2048 >> 4)), idesc_o, (j > 1 || part || kk) ? 1u : 0u);
             }
           }
-          dn::tc_commit(v_empty);
+          dn::tc_commit(&v_empty[st]);
           dn::tc_commit(p_empty);
         }
       }
       dn::tc_commit(o_full);
     }
   } else if (warp >= 4) {
-    const int qd = warp & 3, half = (warp - 4) >> 2, r = qd * 32 + lane;      // TMEM lane quarter, half of the columns, this thread's row
+    const int qd = warp & 3, cq = (warp - 4) >> 2, r = qd * 32 + lane;      // TMEM lane quarter, quarter of the columns, this thread's row
     const int hr = r / TB, tr = r % TB;
     const bool ok = hr < nh && tr < nq;
     const int pos = p_first + tr, lo = ok ? attn_lo(pos, p.chunk, p.window) : 0, hi_pos = ok ? pos : -1;
     const uint32_t lane_off = (uint32_t)(qd * 32) << 16;
     const float ns = -p.scale * SG_LOG2E;
     const float* tab = p.tab + (size_t)(h0 + (ok ? hr : 0)) * p.D;
+    uint32_t hi[16], lw[16];
+    // weights of columns 2 k, 2 k + 1 from z = (bias - offset - score) log2(e): 1 / (1 + 2^z); two denominators share a reciprocal
+    // (z is capped where 2^-60 stands for zero)
+    auto weigh = [&](int k, float za, float zb, bool sa, bool sb) {
+      const float a = 1.f + sg_ex2(fminf(za, 60.f)), c = 1.f + sg_ex2(fminf(zb, 60.f)), rc = sg_rcp(a * c);
+      const float wa = sa ? rc * c : 0.f, wb = sb ? rc * a : 0.f;
+      hi[k] = pack_bf16(wa, wb);
+      lw[k] = pack_bf16(wa - __uint_as_float(hi[k] << 16), wb - __uint_as_float(hi[k] & 0xffff0000u));
+    };
     for (int j = 0; j < n_tiles; j++) {
-      const int st = j & 1, key0 = (page0 + 2 * j) * PAGE + half * 64;      // this thread's 64 keys
+      const int st = j & 1, key0 = (page0 + 2 * j) * PAGE + cq * 32, d0 = pos - key0;      // this thread's 32 keys; the first one's distance
+      // every key of the quarter is seen by every live row of the warp (rows without a query compute something that is not stored)
+      const bool inner = __all_sync(0xffffffffu, !ok || (key0 >= lo && key0 + 31 <= pos));
+      float tv[32], v[32];
+      if (inner) {
+        const float* tp = tab + (ok ? d0 : 31);
+#pragma unroll
+        for (int i = 0; i < 32; i++) tv[i] = __ldg(tp - i);
+      } else {
+#pragma unroll
+        for (int i = 0; i < 32; i++) tv[i] = __ldg(tab + min(max(d0 - i, 0), p.D - 1));
+      }
       dn::mbar_wait(&s_full[st], (j >> 1) & 1, p.err);
       dn::tc_fence_after();
-      uint32_t hi[32], lw[32];
-      // every key of the half seen by every live row of the warp (rows without a query compute something that is not stored)
-      const bool inner = __all_sync(0xffffffffu, !ok || (key0 >= lo && key0 + 63 <= pos));
-#pragma unroll
-      for (int c = 0; c < 4; c++) {
-        float v[16];
-        dn::tc_ld16(tmem + st * 128 + lane_off + half * 64 + c * 16, v);
-        const int d0 = pos - key0 - c * 16;      // distance of the chunk's first key
-#pragma unroll
-        for (int i = 0; i < 16; i += 2) {
-          float za, zb;
-          bool sa = true, sb = true;
-          if (inner && ok) {
-            za = fmaf(v[i], ns, __ldg(tab + d0 - i));
-            zb = fmaf(v[i + 1], ns, __ldg(tab + d0 - i - 1));
-          } else {
-            const int ka = key0 + c * 16 + i;
-            sa = ka >= lo && ka <= hi_pos;
-            sb = ka + 1 >= lo && ka + 1 <= hi_pos;
-            za = fmaf(v[i], ns, __ldg(tab + min(max(d0 - i, 0), p.D - 1)));
-            zb = fmaf(v[i + 1], ns, __ldg(tab + min(max(d0 - i - 1, 0), p.D - 1)));
-          }
-          // weights 1 / (1 + 2^z); two denominators share a reciprocal (z is capped where 2^-60 stands for zero)
-          const float a = 1.f + exp2f(fminf(za, 60.f)), c2 = 1.f + exp2f(fminf(zb, 60.f));
-          const float rc = __fdividef(1.f, a * c2);
-          float wa = sa ? rc * c2 : 0.f, wb = sb ? rc * a : 0.f;
-          const uint32_t hp = pack_bf16(wa, wb);
-          const __nv_bfloat162 hb = *reinterpret_cast<const __nv_bfloat162*>(&hp);
-          hi[c * 8 + i / 2] = hp;
-          lw[c * 8 + i / 2] = pack_bf16(wa - __low2float(hb), wb - __high2float(hb));
-        }
-      }
+      sg_ld32(tmem + st * 128 + lane_off + cq * 32, v);
       dn::tc_fence_before();
       __syncwarp();
       if (lane == 0) dn::mbar_arrive(&s_empty[st]);
+      if (inner) {
+#pragma unroll
+        for (int i = 0; i < 32; i += 2) weigh(i / 2, fmaf(v[i], ns, tv[i]), fmaf(v[i + 1], ns, tv[i + 1]), true, true);
+      } else {
+#pragma unroll
+        for (int i = 0; i < 32; i += 2) {
+          const int ka = key0 + i;
+          weigh(i / 2, fmaf(v[i], ns, tv[i]), fmaf(v[i + 1], ns, tv[i + 1]), ka >= lo && ka <= hi_pos, ka + 1 >= lo && ka + 1 <= hi_pos);
+        }
+      }
       dn::mbar_wait(p_empty, (j & 1) ^ 1u, p.err);      // the product with the previous tile's weights has read them
 #pragma unroll
-      for (int c = 0; c < 8; c++) {
-        *reinterpret_cast<uint4*>(sPh + dn::at_swz(r, half * 8 + c)) = make_uint4(hi[4 * c], hi[4 * c + 1], hi[4 * c + 2], hi[4 * c + 3]);
-        *reinterpret_cast<uint4*>(sPl + dn::at_swz(r, half * 8 + c)) = make_uint4(lw[4 * c], lw[4 * c + 1], lw[4 * c + 2], lw[4 * c + 3]);
+      for (int c = 0; c < 4; c++) {
+        *reinterpret_cast<uint4*>(sPh + dn::at_swz(r, cq * 4 + c)) = make_uint4(hi[4 * c], hi[4 * c + 1], hi[4 * c + 2], hi[4 * c + 3]);
+        *reinterpret_cast<uint4*>(sPl + dn::at_swz(r, cq * 4 + c)) = make_uint4(lw[4 * c], lw[4 * c + 1], lw[4 * c + 2], lw[4 * c + 3]);
       }
       const int valid = kv_max - (page0 + 2 * j) * PAGE;      // value rows from here on belong to no key: whatever the page holds, it must not enter
       if (valid < 128) {
-        dn::mbar_wait(v_full, j & 1, p.err);
+        dn::mbar_wait(&v_full[st], (j >> 1) & 1, p.err);
         const int per_row = 8 * (DV / 64);
-        for (int i = threadIdx.x - 128; i < (128 - valid) * per_row; i += 256) {
+        for (int i = threadIdx.x - 128; i < (128 - valid) * per_row; i += SG_THREADS - 128) {
           const int row = valid + i / per_row, c = i % per_row;
-          *reinterpret_cast<uint4*>(sV + (c >> 3) * SG_HALF + row * 128 + (c & 7) * 16) = make_uint4(0u, 0u, 0u, 0u);
+          *reinterpret_cast<uint4*>(sV + st * VB + (c >> 3) * SG_HALF + row * 128 + (c & 7) * 16) = make_uint4(0u, 0u, 0u, 0u);
         }
       }
       asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
@@ -226,11 +248,11 @@ __global__ void __launch_bounds__(SG_THREADS, 1) k_sig_attn_tc(const __grid_cons
     dn::mbar_wait(o_full, 0, p.err);
     dn::tc_fence_after();
     const float og = ok && p.gate ? sigmoid_f(p.gate[(size_t)(s0 + tr) * p.H + h0 + hr]) : 1.f;
-    bf16* dst = p.out + ((size_t)(s0 + (ok ? tr : 0)) * p.H + h0 + (ok ? hr : 0)) * DV + half * (DV / 2);
+    bf16* dst = p.out + ((size_t)(s0 + (ok ? tr : 0)) * p.H + h0 + (ok ? hr : 0)) * DV + cq * (DV / 4);
 #pragma unroll
-    for (int c = 0; c < DV / 32; c++) {
+    for (int c = 0; c < DV / 64; c++) {
       float v[16];
-      dn::tc_ld16(tO + lane_off + half * (DV / 2) + c * 16, v);
+      dn::tc_ld16(tO + lane_off + cq * (DV / 4) + c * 16, v);
       if (ok) {
 #pragma unroll
         for (int x = 0; x < 2; x++) {
