@@ -824,24 +824,35 @@ static int attn_rows_stages(const dn_seq_layer_cfg& lc, int N) {      // 0: not 
   if (N > AT_SPLIT_ROWS || lc.pool > 0 || lc.dim > 128 || lc.vdim > 128 || (lc.dim * esz) % 16 || (lc.vdim * esz) % 16) return 0;
   const bool one = lc.chunk > 0 && lc.chunk <= AT_MAX_SPLITS * AR_KEYS;
   for (int st = one ? 1 : 2; st > 0; st--)
-    if (ar_smem_bytes(lc.dim, lc.vdim, esz, lc.v_is_k != 0, st) + 1024 <= g_max_smem) return st;
+    if (ar_smem_bytes(lc.dim, lc.vdim, esz, lc.v_is_k != 0, st, 4) + 1024 <= g_max_smem) return st;
   return 0;
 }
-template <class T, bool SIG>
+template <class T, bool SIG, int HB>
 static cudaError_t attn_rows_launch(dn_seq_model* m, cudaStream_t s, const Batch& b, const T* q, const T* kp, const T* vp, const dn_seq_layer_cfg& lc, const AttnExtra& ex,
-                                    int stages, T* out) {
-  const size_t smem = ar_smem_bytes(lc.dim, lc.vdim, (int)sizeof(T), lc.v_is_k != 0, stages);
+                                    int stages, int Z, T* out) {
+  const size_t smem = ar_smem_bytes(lc.dim, lc.vdim, (int)sizeof(T), lc.v_is_k != 0, stages, HB);
   static size_t attr = 40 * 1024;      // (the default limit counts the static part too)
   if (smem > attr) {
-    cudaError_t e = cudaFuncSetAttribute(k_attn_rows<T, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(k_attn_rows<T, SIG, HB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return e;
     attr = smem;
   }
-  const int R = lc.heads / lc.kv_heads, per = (R + AR_HEADS - 1) / AR_HEADS;
+  const int R = lc.heads / lc.kv_heads, per = (R + HB - 1) / HB;
+  return launch(k_attn_rows<T, SIG, HB>, dim3(b.N, lc.kv_heads * per, Z), dim3(AR_WARPS * 32), smem, s, b, q, kp, vp, lc.heads, lc.kv_heads, lc.dim, lc.vdim, lc.chunk,
+                lc.scale, stages, ex, out, m->attn_part, m->attn_count);
+}
+template <class T>
+static cudaError_t attn_rows(dn_seq_model* m, cudaStream_t s, const Batch& b, const T* q, const T* kp, const T* vp, const dn_seq_layer_cfg& lc, const AttnExtra& ex,
+                             int stages, T* out) {
   // (a mask of `chunk` positions bounds the keys of a row, and with them its splits)
   const int Z = lc.chunk > 0 ? std::min((int)AT_MAX_SPLITS, (lc.chunk + AR_KEYS - 1) / AR_KEYS) : AT_MAX_SPLITS;
-  return launch(k_attn_rows<T, SIG>, dim3(b.N, lc.kv_heads * per, Z), dim3(AR_WARPS * 32), smem, s, b, q, kp, vp, lc.heads, lc.kv_heads, lc.dim, lc.vdim, lc.chunk,
-                lc.scale, stages, ex, out, m->attn_part, m->attn_count);
+  const int R = lc.heads / lc.kv_heads;
+  auto blocks = [&](int hb) { return (long long)b.N * lc.kv_heads * ((R + hb - 1) / hb) * Z; };
+  const int hb = R == 1 || blocks(1) <= 2 * g_sms ? 1 : R == 2 || blocks(2) <= 2 * g_sms ? 2 : 4;      // the most blocks that the SMs take at once
+#define AR(SIGv) (hb == 1 ? attn_rows_launch<T, SIGv, 1>(m, s, b, q, kp, vp, lc, ex, stages, Z, out) \
+                : hb == 2 ? attn_rows_launch<T, SIGv, 2>(m, s, b, q, kp, vp, lc, ex, stages, Z, out) : attn_rows_launch<T, SIGv, 4>(m, s, b, q, kp, vp, lc, ex, stages, Z, out))
+  return ex.off ? AR(true) : AR(false);
+#undef AR
 }
 
 // latent attention of a step that brings a prompt portion, bf16: the MMA tiles over the cached rows (R + rot numbers a key,
@@ -1208,8 +1219,7 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
       else if (attn_tiles_ok<T>(lc, b))
         CK(attn_tiles(s, b, (const bf16*)m->qb, (const bf16*)m->kpool[run.kv_index], (const bf16*)vpl, lc, ex, (bf16*)m->mo));
       else if (const int st = attn_rows_stages<T>(lc, N))
-        CK(ex.off ? attn_rows_launch<T, true>(m, s, b, (const T*)m->qb, (const T*)m->kpool[run.kv_index], (const T*)vpl, lc, ex, st, (T*)m->mo)
-                  : attn_rows_launch<T, false>(m, s, b, (const T*)m->qb, (const T*)m->kpool[run.kv_index], (const T*)vpl, lc, ex, st, (T*)m->mo));
+        CK(attn_rows<T>(m, s, b, (const T*)m->qb, (const T*)m->kpool[run.kv_index], (const T*)vpl, lc, ex, st, (T*)m->mo));
       else {
         // a small step (decode): long rows are split over up to AT_MAX_SPLITS blocks, joined by k_attn_merge
         // (a mask of `chunk` positions bounds the keys of a row, and with them its splits)

@@ -1,6 +1,6 @@
 // dn_seq_attn_rows.cuh -- attention of a step with few rows (decode steps and small portions), libdnet_b200_seq.so.
 //
-// What k_attn computes, arranged for latency: a block takes one token, up to AR_HEADS query heads of one key / value head
+// What k_attn computes, arranged for latency: a block takes one token, up to HB (1, 2 or 4) query heads of one key / value head
 // and every nz-th run of 128 keys; each of its four warps stages a tile of 32 keys *and* their values in shared memory by
 // asynchronous copies -- one trip to memory after the block table, whole rows, read once for all the block's heads -- and
 // works from there: a lane scores one key, then owns ceil(dv / 32) adjacent output dims.  The warps' partials join in warp
@@ -12,7 +12,7 @@
 
 namespace dnseq {
 
-constexpr int AR_WARPS = 4, AR_HEADS = 4, AR_KEYS = AR_WARPS * 32;
+constexpr int AR_WARPS = 4, AR_KEYS = AR_WARPS * 32;
 __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
   const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src) : "memory");
@@ -20,13 +20,14 @@ __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
 // bytes of one tile (32 keys and values): key rows are padded by 16 bytes, so that the lanes' 16-byte reads of one column
 // of 32 rows fall into different banks
 __host__ __device__ __forceinline__ size_t ar_tile_bytes(int dk, int dv, int esz, bool vk) { return (size_t)32 * (dk * esz + 16) + (vk ? 0 : (size_t)32 * dv * esz); }
-__host__ __device__ __forceinline__ size_t ar_smem_bytes(int dk, int dv, int esz, bool vk, int stages) {
-  const size_t part = (size_t)AR_WARPS * AR_HEADS * (2 + (dv + 31) / 32 * 32) * 4;
-  return (size_t)AR_HEADS * dk * 4 + ((part + 15) & ~(size_t)15) + (size_t)AR_WARPS * stages * ar_tile_bytes(dk, dv, esz, vk);
+__host__ __device__ __forceinline__ size_t ar_smem_bytes(int dk, int dv, int esz, bool vk, int stages, int HB) {
+  const size_t part = (size_t)AR_WARPS * HB * (2 + (dv + 31) / 32 * 32) * 4;
+  return (size_t)HB * dk * 4 + ((part + 15) & ~(size_t)15) + (size_t)AR_WARPS * stages * ar_tile_bytes(dk, dv, esz, vk);
 }
 __device__ __forceinline__ int ar_splits(int keys, int zmax) { return min(zmax, max(1, (keys + AR_KEYS - 1) / AR_KEYS)); }
 
-template <class T, bool SIG>
+// (a head's result does not depend on HB: small grids take fewer heads a block)
+template <class T, bool SIG, int HB>
 __global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* __restrict__ q, const T* __restrict__ kpool, const T* __restrict__ vpool, int H,
                                                              int G, int dk, int dv, int chunk, float scale, int stages, AttnExtra ex, T* __restrict__ out,
                                                              float* __restrict__ part_g, unsigned int* __restrict__ count) {
@@ -35,12 +36,12 @@ __global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* _
   __shared__ bool last_s;
   constexpr int V = Vec16<T>::n, ESZ = (int)sizeof(T);
   const int VPL = (dv + 31) / 32, dvp = VPL * 32, PL = 2 + dvp;
-  float* qs = reinterpret_cast<float*>(smb);                       // [AR_HEADS][dk]
-  float* part = qs + AR_HEADS * dk;                                // [AR_WARPS][AR_HEADS][2 + dvp]
-  unsigned char* tiles = smb + (size_t)AR_HEADS * dk * 4 + (((size_t)AR_WARPS * AR_HEADS * PL * 4 + 15) & ~(size_t)15);
+  float* qs = reinterpret_cast<float*>(smb);                       // [HB][dk]
+  float* part = qs + HB * dk;                                // [AR_WARPS][HB][2 + dvp]
+  unsigned char* tiles = smb + (size_t)HB * dk * 4 + (((size_t)AR_WARPS * HB * PL * 4 + 15) & ~(size_t)15);
   const int n = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int R = H / G, per = (R + AR_HEADS - 1) / AR_HEADS;        // heads of a key head; blocks they take
-  const int g = blockIdx.y / per, h0 = g * R + (blockIdx.y % per) * AR_HEADS, nh = min(AR_HEADS, (g + 1) * R - h0);
+  const int R = H / G, per = (R + HB - 1) / HB;        // heads of a key head; blocks they take
+  const int g = blockIdx.y / per, h0 = g * R + (blockIdx.y % per) * HB, nh = min(HB, (g + 1) * R - h0);
   const int slot = b.slot[n], p = b.pos[n];
   const int lo = attn_lo(p, chunk, ex.window), nkeys = p - lo + 1;
   const int zmax = gridDim.z, nz = ar_splits(nkeys, zmax), z = blockIdx.z;
@@ -52,6 +53,10 @@ __global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* _
   unsigned char* mine = tiles + (size_t)warp * stages * tile_b;
   const int32_t* bt = b.bt + (size_t)slot * b.max_pages;
   const int step = nz * AR_KEYS, first = (z * AR_WARPS + warp) * 32;
+  // a lane's walk over the 16-byte pieces of a tile's rows: first row and piece, and what 32 pieces further means
+  const int ck = dk * ESZ / 16, cv = dv * ESZ / 16;
+  const int kr0 = lane / ck, kc0 = lane - kr0 * ck, kdr = 32 / ck, kdc = 32 - kdr * ck;
+  const int vr0 = lane / cv, vc0 = lane - vr0 * cv, vdr = 32 / cv, vdc = 32 - vdr * cv;
   auto stage = [&](int s, int j0) {      // this warp's tile at key j0 into buffer s
     unsigned char* kt = mine + (size_t)s * tile_b;
     unsigned char* vt = vk ? kt : kt + (size_t)32 * ldk;
@@ -61,32 +66,34 @@ __global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* _
       rows_s[warp][lane] = (uint32_t)bt[j / PAGE] * PAGE + (uint32_t)(j % PAGE);
     }
     __syncwarp();
-    const int ck = dk * ESZ / 16, cv = vk ? 0 : dv * ESZ / 16;
-    for (int e = lane; e < cnt * ck; e += 32) {
-      const int r = e / ck, c = e - r * ck;
-      cp_async16(kt + (size_t)r * ldk + c * 16, kpool + (size_t)rows_s[warp][r] * Ck + g * dk + c * V);
+    for (int r = kr0, c = kc0; r < cnt;) {
+      cp_async16(kt + r * ldk + c * 16, kpool + (size_t)rows_s[warp][r] * Ck + g * dk + c * V);
+      r += kdr; c += kdc;
+      if (c >= ck) { c -= ck; r++; }
     }
-    for (int e = lane; e < cnt * cv; e += 32) {
-      const int r = e / cv, c = e - r * cv;
-      cp_async16(vt + (size_t)r * ldv_ + c * 16, vpool + (size_t)rows_s[warp][r] * Cv + g * dv + c * V);
-    }
+    if (!vk)
+      for (int r = vr0, c = vc0; r < cnt;) {
+        cp_async16(vt + r * ldv_ + c * 16, vpool + (size_t)rows_s[warp][r] * Cv + g * dv + c * V);
+        r += vdr; c += vdc;
+        if (c >= cv) { c -= cv; r++; }
+      }
     cp_async_commit();
     __syncwarp();
   };
   if (first < nkeys) stage(0, first);
-  for (int e = threadIdx.x; e < AR_HEADS * dk; e += blockDim.x) qs[e] = e < nh * dk ? ldf(q + ((size_t)n * H + h0) * dk + e) : 0.f;
-  float r1[AR_HEADS], r2[AR_HEADS], soff[AR_HEADS];
+  for (int e = threadIdx.x; e < HB * dk; e += blockDim.x) qs[e] = e < nh * dk ? ldf(q + ((size_t)n * H + h0) * dk + e) : 0.f;
+  float r1[HB], r2[HB], soff[HB];
 #pragma unroll
-  for (int i = 0; i < AR_HEADS; i++) {
+  for (int i = 0; i < HB; i++) {
     const int h = h0 + min(i, nh - 1);
     r1[i] = ex.r1 ? ldf((const T*)ex.r1 + h) : 0.f;
     r2[i] = ex.r1 ? ldf((const T*)ex.r2 + h) : 0.f;
     soff[i] = SIG ? ldf((const T*)ex.off + h) : 0.f;
   }
   __syncthreads();
-  float m[AR_HEADS], l[AR_HEADS], acc[AR_HEADS][4];
+  float m[HB], l[HB], acc[HB][4];
 #pragma unroll
-  for (int i = 0; i < AR_HEADS; i++) {
+  for (int i = 0; i < HB; i++) {
     m[i] = -INFINITY; l[i] = 0.f;
 #pragma unroll
     for (int x = 0; x < 4; x++) acc[i][x] = 0.f;
@@ -101,7 +108,9 @@ __global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* _
     const unsigned char* kt = mine + (size_t)s * tile_b;
     const unsigned char* vt = vk ? kt : kt + (size_t)32 * ldk;
     const int cnt = min(32, nkeys - j0), j = j0 + lane;
-    float sc[AR_HEADS] = {0.f, 0.f, 0.f, 0.f};
+    float sc[HB];
+#pragma unroll
+    for (int i = 0; i < HB; i++) sc[i] = 0.f;
     if (lane < cnt) {
       const T* kr = reinterpret_cast<const T*>(kt + (size_t)lane * ldk);
 #pragma unroll 4
@@ -109,7 +118,7 @@ __global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* _
         float kv[V];
         ldv(kr + d, kv);
 #pragma unroll
-        for (int i = 0; i < AR_HEADS; i++) {
+        for (int i = 0; i < HB; i++) {
 #pragma unroll
           for (int x = 0; x < V; x += 4) {
             const float4 q4 = *reinterpret_cast<const float4*>(qs + i * dk + d + x);
@@ -119,9 +128,9 @@ __global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* _
         }
       }
     }
-    float pw[AR_HEADS];
+    float pw[HB];
 #pragma unroll
-    for (int i = 0; i < AR_HEADS; i++) {
+    for (int i = 0; i < HB; i++) {
       float a = sc[i] * scale;
       if (ex.softcap > 0.f) a = ex.softcap * tanhf(a / ex.softcap);
       if (ex.r1) a -= r1[i] * log1pf(r2[i] * (float)max(0, nkeys - 1 - j));
@@ -144,7 +153,7 @@ __global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* _
         for (int x = 0; x < 4; x++) if (x < vcnt) v[x] = ldf(vr + x);
       }
 #pragma unroll
-      for (int i = 0; i < AR_HEADS; i++) {
+      for (int i = 0; i < HB; i++) {
         const float pt = __shfl_sync(0xffffffffu, pw[i], t);
 #pragma unroll
         for (int x = 0; x < 4; x++) acc[i][x] = fmaf(pt, v[x], acc[i][x]);
@@ -155,8 +164,8 @@ __global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* _
     else if (more) stage(0, j0 + step);
   }
 #pragma unroll
-  for (int i = 0; i < AR_HEADS; i++) {
-    float* pr = part + ((size_t)warp * AR_HEADS + i) * PL;
+  for (int i = 0; i < HB; i++) {
+    float* pr = part + ((size_t)warp * HB + i) * PL;
     if (lane == 0) { pr[0] = m[i]; pr[1] = l[i]; }
 #pragma unroll
     for (int x = 0; x < 4; x++) if (x < VPL) pr[2 + lane * VPL + x] = acc[i][x];
@@ -186,7 +195,7 @@ __global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* _
     stf(out + ((size_t)n * H + h) * dv + d, a / L * og);
   };
   if (!split) {
-    for (int e = threadIdx.x; e < nh * dv; e += blockDim.x) finish(e / dv, e % dv, part + (size_t)(e / dv) * PL, (size_t)AR_HEADS * PL, AR_WARPS, false);
+    for (int e = threadIdx.x; e < nh * dv; e += blockDim.x) finish(e / dv, e % dv, part + (size_t)(e / dv) * PL, (size_t)HB * PL, AR_WARPS, false);
     return;
   }
   for (int e = threadIdx.x; e < nh * dv; e += blockDim.x) {
@@ -195,9 +204,9 @@ __global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* _
     float* pg = part_g + (((size_t)n * H + h0 + i) * zmax + z) * PL;
     float M = -INFINITY, L = 0.f, a = 0.f;
     if (!SIG)
-      for (int w = 0; w < AR_WARPS; w++) M = fmaxf(M, pr[(size_t)w * AR_HEADS * PL]);
+      for (int w = 0; w < AR_WARPS; w++) M = fmaxf(M, pr[(size_t)w * HB * PL]);
     for (int w = 0; w < AR_WARPS; w++) {
-      const float* pq = pr + (size_t)w * AR_HEADS * PL;
+      const float* pq = pr + (size_t)w * HB * PL;
       const float f = SIG ? 1.f : expf(pq[0] - M);
       if (!SIG) L += pq[1] * f;
       a += pq[2 + d] * f;
