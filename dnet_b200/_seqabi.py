@@ -22,7 +22,7 @@ DN_ATTN_SOFTMAX, DN_ATTN_SIGMOID = 0, 1
 DN_QKNORM_NONE, DN_QKNORM_WHOLE, DN_QKNORM_HEAD = 0, 1, 2
 DN_RIGHT_GLA, DN_RIGHT_GDELTA = 0, 1
 DN_MLP_DENSE, DN_MLP_MOE = 0, 1
-DN_FF_GEGLU, DN_FF_RELU2 = 0, 1
+DN_FF_GEGLU, DN_FF_RELU2, DN_FF_SWIGLU = 0, 1, 2
 DN_ROUTER_TOPK, DN_ROUTER_SCORED = 0, 1
 DN_SCORE_SOFTMAX, DN_SCORE_SIGMOID = 0, 1
 DN_EXPERT_CGLU, DN_EXPERT_SWIGLU, DN_EXPERT_RELU2 = 0, 1, 2
@@ -40,15 +40,17 @@ _LAYER_SLOTS = ["norm1", "norm2", "mix.q", "mix.k", "mix.v", "mix.o", "mix.q.con
                 "mix.dq", "mix.dq.norm", "mix.dkv", "mix.dkv.norm", "mix.uk", "mix.uv",
                 "mlp.up.b", "mlp.down.b", "router.corr", "shared.sg",
                 "canon1", "canon2", "l.out", "r.out", "r.a", "r.ab",
-                "mix.r1", "mix.r2", "mix.pb"]
+                "mix.r1", "mix.r2", "mix.pb",
+                "ls1", "ls2", "mix.lq1", "mix.lk1", "mix.lq2", "mix.lk2", "side.gate", "side.proj", "side.norm"]
 LAYER_SLOT = {n: i for i, n in enumerate(_LAYER_SLOTS)}
 MODEL_SLOT = {"embed": 100, "final.norm": 101, "head": 102, "final.norm.b": 103, "final.norm.alpha": 104,
-              "embed.norm": 105, "embed.norm.b": 106, "embed.norm.alpha": 107, "loop.in": 108, "bigram": 109, "pos": 110}
+              "embed.norm": 105, "embed.norm.b": 106, "embed.norm.alpha": 107, "loop.in": 108, "bigram": 109, "pos": 110,
+              "side.embed": 111}
 EXPERT_SLOT = {"gate": 0, "up": 1, "down": 2}
 # phases of a step, in the header's order (dn_seq_profile_read)
 PHASES = ["embed", "norm", "proj", "attn_prep", "attn", "delta_prep", "delta_rule", "delta_out", "conv_carry", "out_proj",
           "write_back", "ff_up", "ff_down", "head", "other", "recur_prep", "recur", "recur_out", "router", "moe_up", "moe_down",
-          "latent_in", "latent_out", "canon"]
+          "latent_in", "latent_out", "canon", "side"]
 
 
 class LayerCfg(C.Structure):
@@ -66,7 +68,9 @@ class LayerCfg(C.Structure):
                 ("v_is_k", C.c_int32), ("qtemp_coef", C.c_float), ("qtemp_every", C.c_int32), ("pool", C.c_int32),
                 ("yarn_factor", C.c_float), ("yarn_original", C.c_float), ("yarn_fast", C.c_float), ("yarn_slow", C.c_float),
                 ("r_kind", C.c_int32), ("branch_norm", C.c_int32),
-                ("attn_weight", C.c_int32), ("dist_bias", C.c_int32), ("score_kind", C.c_int32)]
+                ("attn_weight", C.c_int32), ("dist_bias", C.c_int32), ("score_kind", C.c_int32),
+                ("band_factor", C.c_float), ("band_low", C.c_float), ("band_high", C.c_float), ("band_original", C.c_float),
+                ("keep_first", C.c_int32), ("maps", C.c_int32), ("diff", C.c_float)]
 
 
 class SeqCfg(C.Structure):
@@ -76,7 +80,8 @@ class SeqCfg(C.Structure):
                 ("norm_kind", C.c_int32), ("post_norm", C.c_int32), ("embed_norm", C.c_int32), ("logit_softcap", C.c_float),
                 ("loop_start", C.c_int32), ("loop_stop", C.c_int32), ("loop_times", C.c_int32), ("no_pre_norm", C.c_int32),
                 ("canon_taps", C.c_int32), ("bigram_buckets", C.c_int32), ("bigram_mul_prev", C.c_int32), ("bigram_mul_cur", C.c_int32),
-                ("logit_scale", C.c_float), ("parallel_ff", C.c_int32), ("residual_mult", C.c_float), ("max_positions", C.c_int32)]
+                ("logit_scale", C.c_float), ("parallel_ff", C.c_int32), ("residual_mult", C.c_float), ("max_positions", C.c_int32),
+                ("layer_scale", C.c_int32), ("side_dim", C.c_int32)]
 
 
 def declared_symbols() -> List[str]:

@@ -65,6 +65,17 @@ by side, windowed attention whose weights are sigmoids of distance-biased scores
                  "mixer": {"heads", "kv_heads", "dim", "vdim", "conv", "scale", "mask": {"size"}},
                  "mlp": {"kind": "dense", "ff": F}
                       | {"kind": "moe", "router": {"experts", "top", "scale"}, "expert": {"ff"}} | null}, ...]}
+
+``TuguvikRingModel``: dynamic-tanh norms before the sublayers, outputs scaled per channel, latent attention with a sink beside
+differential attention whose window keeps the first tokens, and a gated row of a token table at the end of every layer:
+
+    {"architecture": "Tuguvik", "vocab": V, "width": W, "norm": {"eps": e}, "token_side": {"dim": D},
+     "layers": [{"type": "latent_attention",
+                 "mixer": {"heads", "dim", "rot_dim", "vdim", "kv_rank", "q_rank", "scale", "mask": {"size"}, "kv_from": j,
+                           "rot": {"base", "dims", "scaling": {"factor", "original", "fast", "slow"}}}, "mlp": ...},
+                {"type": "attention",
+                 "mixer": {"heads", "kv_heads", "dim", "vdim", "scale", "diff", "mask": {"size", "keep_first"},
+                           "rot": {"base", "dims", "scaling": {"factor", "low", "high", "original"}}}, "mlp": ...}, ...]}
 """
 from __future__ import annotations
 
@@ -111,9 +122,12 @@ def _attention_cfg(lc: _seqabi.LayerCfg, mx: dict, qk_norm, mask: str = "block",
     lc.rot_base = float(rot.get("base", 10000.0))
     lc.rot_layout = _seqabi.DN_ROT_HALF if rot_layout == "half" else _seqabi.DN_ROT_INTERLEAVED
     sc = rot.get("scaling")
-    if sc:
+    if sc and "high" in sc:         # by wavelength bands
+        lc.band_factor, lc.band_low, lc.band_high, lc.band_original = (float(sc[k]) for k in ("factor", "low", "high", "original"))
+    elif sc:                        # by a ramp over the pairs
         lc.yarn_factor, lc.yarn_original = float(sc["factor"]), float(sc["original"])
         lc.yarn_fast, lc.yarn_slow = float(sc["fast"]), float(sc["slow"])
+    lc.keep_first = int((mx.get("mask") or {}).get("keep_first", 0) or 0)
     qt = mx.get("q_temp")
     if qt:
         lc.qtemp_coef, lc.qtemp_every = float(qt["coef"]), int(qt["every"])
@@ -126,6 +140,7 @@ def _attention_cfg(lc: _seqabi.LayerCfg, mx: dict, qk_norm, mask: str = "block",
 
 
 _NORM_KIND = {"rms": _seqabi.DN_NORM_RMS, "dyt": _seqabi.DN_NORM_DYT, "layer": _seqabi.DN_NORM_LAYER, "rms_scalar": _seqabi.DN_NORM_RMS_SCALAR}
+_FF_ACT = {"geglu": _seqabi.DN_FF_GEGLU, "relu2": _seqabi.DN_FF_RELU2, "swiglu": _seqabi.DN_FF_SWIGLU}
 _EXPERT_ACT = {"cglu": _seqabi.DN_EXPERT_CGLU, "swiglu": _seqabi.DN_EXPERT_SWIGLU, "relu2": _seqabi.DN_EXPERT_RELU2}
 
 
@@ -138,6 +153,7 @@ def parse_layer_list(cfg: dict, family: Optional[dict] = None,
            "mask": "block", "ff_act": "geglu", "router": "topk", "expert_act": "cglu", "shared_gate": False}
     fam.update({"v_is_k": False, "rot_layout": "interleaved", "right": "gla", "branch_norm": False})
     fam.update({"attn_weight": "softmax", "dist_bias": False, "parallel_ff": False, "router_score": "softmax"})
+    fam.update({"differential": False, "layer_scale": False, "latent": {}})
     fam.update(family or {})
     shapes = shapes or {}
 
@@ -165,16 +181,17 @@ def parse_layer_list(cfg: dict, family: Optional[dict] = None,
             lc.sink, lc.out_gate, lc.v_is_k = int(per("sink", kind)), int(per("head_gate", kind)), int(per("v_is_k", kind))
             lc.attn_weight = _seqabi.DN_ATTN_SIGMOID if fam["attn_weight"] == "sigmoid" else _seqabi.DN_ATTN_SOFTMAX
             lc.dist_bias = int(per("dist_bias", kind))
+            if per("differential", kind):
+                lc.maps, lc.diff = 2, float(mx["diff"])
         elif kind in ("latent_attention", "latent_attention_2"):
-            # the second type sends its queries through a normed latent too, pairs rotary dims half apart and gates its heads
-            second = kind == "latent_attention_2"
+            # what a type does beyond the plain form: queries through a normed latent too, pairing of rotary dims, gated heads, a sink
+            v = fam["latent"].get(kind, {})
             lc.mixer = _seqabi.DN_MIX_LATENT
-            _attention_cfg(lc, {**mx, "kv_heads": 1}, False, fam["mask"])
+            _attention_cfg(lc, {**mx, "kv_heads": 1}, False, fam["mask"], v.get("rot_layout", "interleaved"))
             lc.rot_part = int(mx.get("rot_dim", lc.rot_dims))
             lc.kv_rank = int(mx["kv_rank"])
-            lc.q_rank = from_shape(f"l{i}.mix.dq", 0, mx, "q_rank", f"layer {i}") if second else 0
-            lc.rot_layout = _seqabi.DN_ROT_HALF if second else _seqabi.DN_ROT_INTERLEAVED
-            lc.out_gate = int(second)
+            lc.q_rank = from_shape(f"l{i}.mix.dq", 0, mx, "q_rank", f"layer {i}") if v.get("q_latent") else 0
+            lc.out_gate, lc.sink = int(v.get("gate", False)), int(v.get("sink", False))
         elif kind == "delta":
             lc.mixer = _seqabi.DN_MIX_DELTA
             lc.heads, lc.kv_heads = int(mx["heads"]), int(mx.get("kv_heads", mx["heads"]))
@@ -213,7 +230,7 @@ def parse_layer_list(cfg: dict, family: Optional[dict] = None,
             mk = mlp.get("kind", "dense")
             if mk == "dense":
                 lc.mlp_kind, lc.ff = _seqabi.DN_MLP_DENSE, int(mlp["ff"])
-                lc.ff_act = _seqabi.DN_FF_RELU2 if fam["ff_act"] == "relu2" else _seqabi.DN_FF_GEGLU
+                lc.ff_act = _FF_ACT[fam["ff_act"]]
             elif mk == "moe":
                 lc.mlp_kind = _seqabi.DN_MLP_MOE
                 lc.expert_act = _EXPERT_ACT[fam["expert_act"]]
@@ -243,6 +260,7 @@ def parse_layer_list(cfg: dict, family: Optional[dict] = None,
     sc.norm_kind = _NORM_KIND[fam["norm"]]
     sc.parallel_ff, sc.residual_mult = int(fam["parallel_ff"]), float(cfg.get("residual_mult", 1.0))
     sc.max_positions = int(cfg.get("max_positions", 0) or 0)
+    sc.layer_scale, sc.side_dim = int(fam["layer_scale"]), int((cfg.get("token_side") or {}).get("dim", 0) or 0)
     sc.canon_taps = int((cfg.get("canon") or {}).get("taps", 0) or 0)
     bg = (cfg.get("embedding") or {}).get("bigram")
     if bg:
@@ -318,6 +336,8 @@ class SeqMixRingModel(BaseRingModel):
             out["pos"] = (sc.max_positions, W)
         if sc.bigram_buckets > 0:
             out["bigram"] = (sc.bigram_buckets + 1, W)
+        if sc.side_dim > 0:
+            out["side.embed"] = (V, len(self._layer_structs) * sc.side_dim)
         if not self.family.get("tied_head"):
             out["head"] = (V, W)
 
@@ -338,7 +358,9 @@ class SeqMixRingModel(BaseRingModel):
             att = lc.mixer in (_seqabi.DN_MIX_ATTENTION, _seqabi.DN_MIX_PARALLEL)
             latent = lc.mixer == _seqabi.DN_MIX_LATENT
             cq = (lc.heads if lc.mixer != _seqabi.DN_MIX_DELTA else lc.kv_heads) * lc.dim
-            ck, cv = lc.kv_heads * lc.dim, (lc.kv_heads if att else lc.heads) * lc.vdim
+            maps = max(1, lc.maps)
+            cq *= maps
+            ck, cv = lc.kv_heads * lc.dim * maps, (lc.kv_heads if att else lc.heads) * lc.vdim
             co = lc.heads * lc.vdim
             own = not (att and lc.kv_from >= 0) and not latent
             if not sc.no_pre_norm:
@@ -349,6 +371,15 @@ class SeqMixRingModel(BaseRingModel):
                     out[p + "canon2"] = (W, sc.canon_taps)
             if sc.post_norm:
                 norm(p + "post1")
+            if sc.layer_scale:
+                out[p + "ls1"] = (W,)
+                if lc.ff > 0:
+                    out[p + "ls2"] = (W,)
+            if sc.side_dim > 0:
+                out[p + "side.gate"], out[p + "side.proj"], out[p + "side.norm"] = (sc.side_dim, W), (W, sc.side_dim), (W,)
+            if maps > 1:
+                for q in ("lq1", "lk1", "lq2", "lk2"):
+                    out[f"{p}mix.{q}"] = (lc.dim,)
             out[p + "mix.q"] = (cq, W)
             out[p + "mix.o"] = (W, co)
             if own:
@@ -360,7 +391,10 @@ class SeqMixRingModel(BaseRingModel):
                 out[p + "mix.q"] = (cq, lc.q_rank if lc.q_rank > 0 else W)
                 if lc.q_rank > 0:
                     out[p + "mix.dq"], out[p + "mix.dq.norm"] = (lc.q_rank, W), (lc.q_rank,)
-                out[p + "mix.dkv"], out[p + "mix.dkv.norm"] = (lc.kv_rank + lc.rot_part, W), (lc.kv_rank,)
+                if lc.kv_from < 0:
+                    out[p + "mix.dkv"], out[p + "mix.dkv.norm"] = (lc.kv_rank + lc.rot_part, W), (lc.kv_rank,)
+                if lc.sink:
+                    out[p + "sink"] = (lc.heads,)
                 out[p + "mix.uk"], out[p + "mix.uv"] = (lc.heads * lc.dim, lc.kv_rank), (co, lc.kv_rank)
                 if lc.out_gate:
                     out[p + "head_gate"] = (lc.heads, W)
@@ -620,7 +654,8 @@ class LutesunRingModel(SeqMixRingModel):
     expert; scaled embedding whose table is also the output head."""
 
     model_type = "lutesun"
-    family = {"norm": "rms", "post_norm": True, "pre_norm": False, "qk_norm": False, "tied_head": True, "mask": "window",
+    family = {"latent": {"latent_attention_2": {"q_latent": True, "rot_layout": "half", "gate": True}},
+              "norm": "rms", "post_norm": True, "pre_norm": False, "qk_norm": False, "tied_head": True, "mask": "window",
               "ff_act": "relu2", "router": "scored", "expert_act": "swiglu", "shared_gate": True}
     tensor_alias = {
         "*": {"norm1": "post1", "norm2": "post2", **_MOE_ALIAS, "mlp.correction": "router.corr", "mlp.shared.sg": "shared.sg"},
@@ -660,3 +695,17 @@ class BokenexRingModel(SeqMixRingModel):
     family = {"norm": "rms_scalar", "parallel_ff": True, "qk_norm": "head", "mask": "window", "attn_weight": "sigmoid", "dist_bias": True,
               "ff_act": "relu2", "ff_bias": False, "router": "scored", "router_score": "sigmoid", "router_corr": False, "expert_act": "relu2"}
     tensor_alias = {"*": _MOE_ALIAS}
+
+
+class TuguvikRingModel(SeqMixRingModel):
+    """Tuguvik: dynamic-tanh norms before every sublayer, whose output joins the residual times a learned vector; layers are
+    either latent attention under a sliding window (queries through a normed latent, interpolated rotary frequencies, a sink,
+    gated heads; a layer may read the rows an earlier one cached) or GQA differential attention (two maps a head over one
+    value, subtracted and normed) under a window that keeps the sequence's first tokens, with rotary frequencies scaled by
+    wavelength; a dense silu-gated feed-forward; every layer ends with its columns of a per-token table, gated by the residual,
+    projected and normed."""
+
+    model_type = "tuguvik"
+    family = {"norm": "dyt", "layer_scale": True, "qk_norm": False, "mask": "window", "rot_layout": "half", "ff_act": "swiglu",
+              "differential": {"attention": True}, "latent": {"latent_attention": {"q_latent": True, "gate": True, "sink": True}}}
+    tensor_alias = {"latent_attention": {"mix.uq": "mix.q", "mix.g": "head_gate", "mix.sink": "sink"}}

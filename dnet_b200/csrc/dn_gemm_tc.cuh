@@ -24,6 +24,9 @@
 //   EPI_SGLU   : two weight tiles; y = T(silu(acc_g) * acc_u), in fp32 with one rounding
 //   EPI_RELU2  : y = T(relu(acc + bias)^2)
 //   (EPI_STORE_F32 adds the bias too when there is one)
+//   EPI_GELU_TAB : y = T(gelu_tanh(acc) * tab[row[t] tab_ld + n]), in fp32 with one rounding
+//   EPI_JOIN   : an fp32 residual takes the product in, x[t][n] += acc mul ls[n], and the norm that follows is elementwise:
+//                nh[t][n] = T(tanh(alpha x) w + b), or T(x) without an alpha (ls, nh optional; no Y)
 //
 // GROUPED: one launch over many weight matrices of one shape (routed experts).  The token rows are sorted by matrix
 // into tiles of BN rows that never span two matrices; a device table gives every token tile its matrix, first row
@@ -35,7 +38,7 @@
 
 namespace dn {
 
-enum { EPI_STORE = 0, EPI_RESID = 1, EPI_SWIGLU = 2, EPI_STORE_F32 = 3, EPI_GEGLU = 4, EPI_CGLU = 5, EPI_TANH = 6, EPI_SGLU = 7, EPI_RELU2 = 8 };
+enum { EPI_STORE = 0, EPI_RESID = 1, EPI_SWIGLU = 2, EPI_STORE_F32 = 3, EPI_GEGLU = 4, EPI_CGLU = 5, EPI_TANH = 6, EPI_SGLU = 7, EPI_RELU2 = 8, EPI_GELU_TAB = 9, EPI_JOIN = 10 };
 __host__ __device__ constexpr bool epi_two_weights(int epi) { return epi == EPI_SWIGLU || epi == EPI_GEGLU || epi == EPI_CGLU || epi == EPI_SGLU; }
 
 constexpr int TC_BM = 128;        // weight rows per tile (MMA M)
@@ -51,6 +54,8 @@ struct TcParams {
   const bf16* bias;               // [N] or null
   unsigned int* err;
   float limit;                    // EPI_CGLU
+  const bf16* tab; const int32_t* row; int tab_ld;       // EPI_GELU_TAB
+  float* x; const bf16* ls; float mul; const bf16 *nw, *nb, *nalpha; bf16* nh;      // EPI_JOIN, leading dimension ldy
   // GROUPED: token tile tt uses the matrix g_tile_e[tt] on the rows [g_tile_r0[tt], + g_tile_rows[tt]) of X and Y
   const int32_t *g_tile_e, *g_tile_r0, *g_tile_rows, *g_ntiles;
   const CUtensorMap *g_mapW, *g_mapW2;      // [matrices], 64-byte aligned, in global memory
@@ -213,6 +218,11 @@ k_gemm_tc(const __grid_constant__ CUtensorMap mapW, const __grid_constant__ CUte
       const uint32_t trow = tmem_base + ab * ACC_COLS + ((uint32_t)(ew * 32) << 16);
       float bias = 0.f;
       if ((EPI == EPI_STORE || EPI == EPI_STORE_F32 || EPI == EPI_RELU2) && p.bias != nullptr && n < p.N) bias = __bfloat162float(p.bias[n]);
+      float jls = 0.f, jw = 0.f, jb = 0.f, ja = 0.f;
+      if (EPI == EPI_JOIN && n < p.N) {
+        jls = p.ls ? p.mul * __bfloat162float(p.ls[n]) : p.mul;
+        if (p.nalpha) { ja = __bfloat162float(*p.nalpha); jw = __bfloat162float(p.nw[n]); jb = __bfloat162float(p.nb[n]); }
+      }
       const int t_base = GROUPED ? p.g_tile_r0[tt] : tt * BN;
       const int t_end = GROUPED ? t_base + p.g_tile_rows[tt] : p.T;
 #pragma unroll 1
@@ -220,6 +230,29 @@ k_gemm_tc(const __grid_constant__ CUtensorMap mapW, const __grid_constant__ CUte
         float v[16], v2[16];
         tc_ld16(trow + c, v);
         if (NA == 2) tc_ld16(trow + BN + c, v2);
+        if (EPI == EPI_JOIN || EPI == EPI_GELU_TAB) {      // all of the chunk's loads first
+          if (n < p.N) {
+#pragma unroll
+            for (int j = 0; j < 16; ++j) {
+              const int t = t_base + c + j;
+              if (t < t_end) v2[j] = EPI == EPI_JOIN ? p.x[(size_t)t * p.ldy + n] : __bfloat162float(p.tab[(size_t)p.row[t] * p.tab_ld + n]);
+            }
+#pragma unroll
+            for (int j = 0; j < 16; ++j) {
+              const int t = t_base + c + j;
+              if (t >= t_end) continue;
+              if (EPI == EPI_JOIN) {
+                const float xn = v2[j] + v[j] * jls;
+                p.x[(size_t)t * p.ldy + n] = xn;
+                if (p.nh) p.nh[(size_t)t * p.ldy + n] = __float2bfloat16_rn(p.nalpha ? tanhf(ja * xn) * jw + jb : xn);
+              } else {
+                const float g = v[j];
+                p.Y[(size_t)t * p.ldy + p.col0 + n] = __float2bfloat16_rn(0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * v2[j]);
+              }
+            }
+          }
+          continue;
+        }
         if (n < p.N) {
 #pragma unroll
           for (int j = 0; j < 16; ++j) {

@@ -67,6 +67,7 @@ struct SeqLayer {
   int Rc, Rv;                   // linear-attention half of a parallel mixer: q / k width, v / output width
   int Cql, Col;                 // latent attention: widths of the absorbed queries [H (R + rot)] and of the output in latent space [H R]
   float* inv_freq;              // [rot/2] device
+  float* lam;                   // differential attention: lambda, computed on the device when its vectors have been bound
   std::vector<const void*> etab_h;   // routed experts: [3][E] gate, up, down
   const void** etab_d;
   CUtensorMap* emaps_d;              // [3][E] TMA descriptors of the experts' matrices, in device memory (bf16 mode)
@@ -94,7 +95,9 @@ struct dn_seq_model {
   bool tm_loop_ok = false, x_xg_ok = false;
   void* xg = nullptr;
   float* attn_part = nullptr;         // partials of split attention rows [AT_SPLIT_ROWS][heads][AT_MAX_SPLITS][2 + vdim padded]
-  XMaps x_cat, x_xm[SHIFT_MAX];
+  XMaps x_cat, x_xm[SHIFT_MAX], x_side;
+  bool lam_stale = true;
+  float* maps32 = nullptr;            // differential attention of steps or sizes without a fused kernel: the maps' outputs [MB][2 heads][vdim]
   size_t esz = 2;
   int S1 = 1, MB = 0, max_pages = 0;
   // scratch
@@ -200,7 +203,7 @@ static int dist_span(const dn_seq_cfg& cfg, const dn_seq_layer_cfg& c) {      //
 // layers whose prompt portions take k_sig_attn_tc (as far as their sizes go)
 constexpr size_t DIST_TAB_MAX = (size_t)1 << 24;      // floats
 static bool sig_tc_sizes(const dn_seq_cfg& cfg, const dn_seq_layer_cfg& c) {
-  return cfg.dtype == DN_SEQ_BF16 && (c.mixer == DN_MIX_ATTENTION || c.mixer == DN_MIX_PARALLEL) && c.attn_weight == DN_ATTN_SIGMOID && c.softcap <= 0.f && c.pool == 0 &&
+  return cfg.dtype == DN_SEQ_BF16 && (c.mixer == DN_MIX_ATTENTION || c.mixer == DN_MIX_PARALLEL) && c.attn_weight == DN_ATTN_SIGMOID && c.softcap <= 0.f && c.pool == 0 && c.keep_first == 0 &&
          (c.dim == 64 || c.dim == 128) && (c.vdim == 64 || c.vdim == 128) && (size_t)c.heads * dist_span(cfg, c) <= DIST_TAB_MAX;
 }
 static void make_xmaps(XMaps* x, const void* base, int rows, int cols) {
@@ -208,6 +211,39 @@ static void make_xmaps(XMaps* x, const void* base, int rows, int cols) {
   const int br[3] = {32, 64, 128};
   for (int i = 0; i < 3; i++) x->ok = x->ok && make_tmap(&x->m[i], base, rows, cols, br[i]);
 }
+
+static int n_maps(const dn_seq_layer_cfg& c) { return c.maps == 2 ? 2 : 1; }
+// rotary frequencies base^(-2j/dims), j = 0 .. dims/2 - 1, optionally scaled.  By a ramp over the pairs (yarn_*): pairs that turn fast
+// within the original context keep theirs, slow ones are divided by the factor, a line between.  By wavelength (band_*): short ones keep
+// theirs, long ones are divided, a blend between.
+static std::vector<float> rot_freqs(const dn_seq_layer_cfg& c) {
+  std::vector<float> f(c.rot_dims / 2);
+  const double dims = c.rot_dims, base = c.rot_base;
+  double lo = 0, hi = 0;
+  if (c.yarn_factor > 0.f) {
+    auto dim_of = [&](double turns) { return dims * std::log((double)c.yarn_original / (2.0 * M_PI * turns)) / (2.0 * std::log(base)); };
+    lo = std::max(std::floor(dim_of(c.yarn_fast)), 0.0);
+    hi = std::min(std::ceil(dim_of(c.yarn_slow)), dims - 1.0);
+  }
+  for (int j = 0; j < c.rot_dims / 2; j++) {
+    double fj = std::pow(base, -2.0 * j / dims);
+    if (c.yarn_factor > 0.f) {
+      const double ramp = std::min(1.0, std::max(0.0, ((double)j - lo) / std::max(hi - lo, 0.001)));
+      fj = fj / (double)c.yarn_factor * ramp + fj * (1.0 - ramp);
+    }
+    if (c.band_factor > 0.f) {
+      const double wl = 2.0 * M_PI / fj, orig = c.band_original, low = c.band_low, high = c.band_high;
+      if (wl > orig / low) fj /= (double)c.band_factor;
+      else if (!(wl < orig / high)) {
+        const double s = (orig / wl - low) / (high - low);
+        fj = (1.0 - s) * fj / (double)c.band_factor + s * fj;
+      }
+    }
+    f[j] = (float)fj;
+  }
+  return f;
+}
+static float rot_mscale(const dn_seq_layer_cfg& c) { return c.yarn_factor > 0.f ? 0.1f * logf(c.yarn_factor) + 1.f : 1.f; }
 
 template <class P>
 static int dalloc(P** p, size_t bytes) {
@@ -222,7 +258,7 @@ extern "C" int dn_seq_model_destroy(dn_seq_model* m) {
   cudaDeviceSynchronize();
   void* ptrs[] = {m->xs, m->y, m->pa, m->pb, m->qn, m->kn, m->vv, m->od, m->beta, m->decay, m->h, m->uq, m->uk, m->uv, m->qb,
                   m->mo, m->gt, m->act, m->conv_state, m->delta_state, m->stage_d, m->bt_d, m->tc_err, m->y2, m->x0, m->dz, m->rwt,
-                  m->eo, m->cat, m->xm, m->lr, m->eact, m->ridx, m->rpos, m->rtok, m->tiles, m->xg, m->attn_part, m->attn_count, m->dist_tab, m->sgate, m->hn, m->un, m->aun};
+                  m->eo, m->cat, m->xm, m->lr, m->eact, m->ridx, m->rpos, m->rtok, m->tiles, m->xg, m->attn_part, m->attn_count, m->dist_tab, m->sgate, m->hn, m->un, m->aun, m->maps32};
   for (void* p : ptrs) if (p) cudaFree(p);
   for (auto& g : m->graphs) cudaGraphExecDestroy(g.second.first);
   if (m->lg_buf) cudaFree(m->lg_buf);
@@ -232,7 +268,7 @@ extern "C" int dn_seq_model_destroy(dn_seq_model* m) {
   for (void* p : m->vpool) if (p) cudaFree(p);
   for (void* p : m->pkpool) if (p) cudaFree(p);
   for (void* p : m->pvpool) if (p) cudaFree(p);
-  for (auto& l : m->L) { if (l.inv_freq) cudaFree(l.inv_freq); if (l.etab_d) cudaFree((void*)l.etab_d); if (l.emaps_d) cudaFree(l.emaps_d); }
+  for (auto& l : m->L) { if (l.inv_freq) cudaFree(l.inv_freq); if (l.lam) cudaFree(l.lam); if (l.etab_d) cudaFree((void*)l.etab_d); if (l.emaps_d) cudaFree(l.emaps_d); }
   if (m->stage_h) cudaFreeHost(m->stage_h);
   if (m->bt_h) cudaFreeHost(m->bt_h);
   if (m->staged) cudaEventDestroy(m->staged);
@@ -275,14 +311,15 @@ extern "C" int dn_seq_model_create(const dn_seq_cfg* cfg, const dn_seq_layer_cfg
     rc = fail(DN_EINVAL, "bigram table of %d buckets with multipliers %d / %d unsupported", cfg->bigram_buckets, cfg->bigram_mul_prev, cfg->bigram_mul_cur);
   if (rc == DN_OK && cfg->norm_kind == DN_NORM_RMS && cfg->post_norm && cfg->streams > 0)
     rc = fail(DN_EINVAL, "an RMS norm after a sublayer joins the plain residual only (streams = 0)");
+  if (rc == DN_OK && (cfg->layer_scale || cfg->side_dim != 0) && (cfg->side_dim < 0 || cfg->post_norm || cfg->no_pre_norm || cfg->streams > 0 || cfg->parallel_ff))
+    rc = fail(DN_EINVAL, "scaled outputs and a token input of %d numbers after a layer need the plain residual with norms before the sublayers only", cfg->side_dim);
+  mff = std::max(mff, cfg->side_dim);
+  for (auto& l : m->L) { l.inv_freq = nullptr; l.lam = nullptr; l.etab_d = nullptr; l.emaps_d = nullptr; }
   for (int i = 0; i < cfg->n_layers && rc == DN_OK; i++) {
     SeqLayer& l = m->L[i];
     l.c = layers[i];
     memset(l.w, 0, sizeof(l.w));
     memset(l.tm_ok, 0, sizeof(l.tm_ok));
-    l.inv_freq = nullptr;
-    l.etab_d = nullptr;
-    l.emaps_d = nullptr;
     l.x_eact_ok = false;
     l.Rc = l.Rv = l.Cql = l.Col = 0;
     const dn_seq_layer_cfg& c = l.c;
@@ -291,22 +328,38 @@ extern "C" int dn_seq_model_create(const dn_seq_cfg* cfg, const dn_seq_layer_cfg
       break;
     }
     if (c.conv < 0 || c.conv > 9) { rc = fail(DN_EINVAL, "layer %d: conv taps %d unsupported (0..9)", i, c.conv); break; }
+    if (c.keep_first < 0 || (c.keep_first > 0 && (c.mask_kind != DN_MASK_WINDOW || c.pool > 0 || c.mixer == DN_MIX_LATENT))) {
+      rc = fail(DN_EINVAL, "layer %d: %d kept first tokens stand behind a sliding window of plain keys without pooled blocks", i, c.keep_first);
+      break;
+    }
+    if (c.maps < 0 || c.maps > 2 || (c.maps == 2 && (c.mixer != DN_MIX_ATTENTION || c.attn_weight != DN_ATTN_SOFTMAX || c.sink || c.out_gate || c.dist_bias ||
+                                                     c.v_is_k || c.pool > 0))) {
+      rc = fail(DN_EINVAL, "layer %d: %d maps a head unsupported (2: softmax attention with values of its own, no sink, gates, distance bias or pooled blocks)", i, c.maps);
+      break;
+    }
+    if (c.rot_dims > 0 && ((c.yarn_factor > 0.f && c.band_factor > 0.f) || (c.band_factor > 0.f && !(c.band_low > 0.f && c.band_high > 0.f && c.band_original > 0.f)))) {
+      rc = fail(DN_EINVAL, "layer %d: rotary frequencies scaled by factor %g / low %g / high %g / original %g unsupported", i, c.band_factor, c.band_low, c.band_high, c.band_original);
+      break;
+    }
     if (c.mixer == DN_MIX_ATTENTION || c.mixer == DN_MIX_PARALLEL) {
       if (c.vdim > 256) { rc = fail(DN_EINVAL, "layer %d: vdim %d > 256", i, c.vdim); break; }
       if (c.rot_dims < 0 || c.rot_dims > c.dim || (c.rot_dims & 1)) { rc = fail(DN_EINVAL, "layer %d: rot dims %d unsupported", i, c.rot_dims); break; }
-      l.Cq = c.heads * c.dim;
+      l.Cq = c.heads * c.dim * n_maps(c);
       l.Co = c.heads * c.vdim;
+      mh = std::max(mh, c.heads * n_maps(c));
       if (c.kv_from >= 0) {
         if (c.kv_from >= i || m->L[c.kv_from].c.mixer != DN_MIX_ATTENTION || m->L[c.kv_from].c.kv_from >= 0 ||
-            m->L[c.kv_from].c.kv_heads != c.kv_heads || m->L[c.kv_from].c.dim != c.dim || m->L[c.kv_from].c.vdim != c.vdim) {
+            m->L[c.kv_from].c.kv_heads != c.kv_heads || m->L[c.kv_from].c.dim != c.dim || m->L[c.kv_from].c.vdim != c.vdim ||
+            n_maps(m->L[c.kv_from].c) != n_maps(c)) {
           rc = fail(DN_EINVAL, "layer %d: kv_from %d must name an earlier attention layer with its own keys and the same head sizes", i, c.kv_from);
           break;
         }
         l.Ck = l.Cv = 0;
       } else {
-        l.Ck = c.kv_heads * c.dim;
+        l.Ck = c.kv_heads * c.dim * n_maps(c);
         l.Cv = c.kv_heads * c.vdim;
       }
+      if (n_maps(c) == 2 && (rc = dalloc(&l.lam, 4)) != DN_OK) break;
       if (c.v_is_k) {
         if (c.vdim != c.dim || c.kv_from >= 0 || c.conv > 0) { rc = fail(DN_EINVAL, "layer %d: values that are the keys need vdim = dim, own keys and no convolutions", i); break; }
         l.Cv = 0;      // one pool: the value of a token is its key row
@@ -323,24 +376,7 @@ extern "C" int dn_seq_model_create(const dn_seq_cfg* cfg, const dn_seq_layer_cfg
       if (cfg->parallel_ff && c.mixer == DN_MIX_PARALLEL) { rc = fail(DN_EINVAL, "layer %d: a parallel mixer beside the feed-forward is unsupported", i); break; }
       if (c.qtemp_every < 0 || (c.rot_layout == DN_ROT_HALF && c.dim < c.rot_dims)) { rc = fail(DN_EINVAL, "layer %d: query scale / rotary layout unsupported", i); break; }
       if (c.rot_dims > 0) {
-        // frequencies base^(-2j/dims); scaled: dims that turn fast within the original context keep theirs, slow ones are
-        // divided by the factor, a linear ramp over the dim index between
-        std::vector<float> f(c.rot_dims / 2);
-        const double dims = c.rot_dims, base = c.rot_base;
-        double lo = 0, hi = 0;
-        if (c.yarn_factor > 0.f) {
-          auto dim_of = [&](double turns) { return dims * std::log((double)c.yarn_original / (2.0 * M_PI * turns)) / (2.0 * std::log(base)); };
-          lo = std::max(std::floor(dim_of(c.yarn_fast)), 0.0);
-          hi = std::min(std::ceil(dim_of(c.yarn_slow)), dims - 1.0);
-        }
-        for (int j = 0; j < c.rot_dims / 2; j++) {
-          double fj = std::pow(base, -2.0 * j / dims);
-          if (c.yarn_factor > 0.f) {
-            const double ramp = std::min(1.0, std::max(0.0, ((double)j - lo) / std::max(hi - lo, 0.001)));
-            fj = fj / (double)c.yarn_factor * ramp + fj * (1.0 - ramp);
-          }
-          f[j] = (float)fj;
-        }
+        const std::vector<float> f = rot_freqs(c);
         if ((rc = dalloc(&l.inv_freq, f.size() * 4)) != DN_OK) break;
         if (cudaMemcpy(l.inv_freq, f.data(), f.size() * 4, cudaMemcpyHostToDevice) != cudaSuccess) { rc = fail(DN_ECUDA, "inv_freq upload failed"); break; }
       }
@@ -373,9 +409,14 @@ extern "C" int dn_seq_model_create(const dn_seq_cfg* cfg, const dn_seq_layer_cfg
       }
     } else if (c.mixer == DN_MIX_LATENT) {
       if (c.kv_rank <= 0 || c.kv_rank > 512 || c.q_rank < 0 || c.rot_part < 0 || c.rot_dims < 0 || c.rot_dims > c.rot_part || (c.rot_dims & 1) ||
-          c.kv_heads != 1 || c.conv > 0 || c.kv_from >= 0 || c.sink || c.qk_norm) {
+          c.kv_heads != 1 || c.conv > 0 || c.qk_norm) {
         rc = fail(DN_EINVAL, "layer %d: latent attention with kv_rank %d (1..512) / q_rank %d / rotated part %d of which %d turn unsupported", i,
                   c.kv_rank, c.q_rank, c.rot_part, c.rot_dims);
+        break;
+      }
+      if (c.kv_from >= 0 && (c.kv_from >= i || m->L[c.kv_from].c.mixer != DN_MIX_LATENT || m->L[c.kv_from].c.kv_from >= 0 ||
+                             m->L[c.kv_from].c.kv_rank != c.kv_rank || m->L[c.kv_from].c.rot_part != c.rot_part)) {
+        rc = fail(DN_EINVAL, "layer %d: kv_from %d must name an earlier latent-attention layer with its own rows of the same size", i, c.kv_from);
         break;
       }
       l.Cq = c.heads * (c.dim + c.rot_part);
@@ -387,8 +428,7 @@ extern "C" int dn_seq_model_create(const dn_seq_cfg* cfg, const dn_seq_layer_cfg
       mrank = std::max(mrank, c.q_rank);
       m->part_dv = std::max(m->part_dv, (c.kv_rank + 31) / 32 * 32);
       if (c.rot_dims > 0) {
-        std::vector<float> f(c.rot_dims / 2);
-        for (int j = 0; j < c.rot_dims / 2; j++) f[j] = (float)std::pow((double)c.rot_base, -2.0 * j / (double)c.rot_dims);
+        const std::vector<float> f = rot_freqs(c);
         if ((rc = dalloc(&l.inv_freq, f.size() * 4)) != DN_OK) break;
         if (cudaMemcpy(l.inv_freq, f.data(), f.size() * 4, cudaMemcpyHostToDevice) != cudaSuccess) { rc = fail(DN_ECUDA, "inv_freq upload failed"); break; }
       }
@@ -438,7 +478,7 @@ extern "C" int dn_seq_model_create(const dn_seq_cfg* cfg, const dn_seq_layer_cfg
       rc = fail(DN_EINVAL, "layer %d: feed-forward kind %d unknown", i, c.mlp_kind);
       break;
     } else {
-      if (c.ff > 0 && c.ff_act != DN_FF_GEGLU && c.ff_act != DN_FF_RELU2) { rc = fail(DN_EINVAL, "layer %d: feed-forward activation %d unknown", i, c.ff_act); break; }
+      if (c.ff > 0 && c.ff_act != DN_FF_GEGLU && c.ff_act != DN_FF_RELU2 && c.ff_act != DN_FF_SWIGLU) { rc = fail(DN_EINVAL, "layer %d: feed-forward activation %d unknown", i, c.ff_act); break; }
       mff = std::max(mff, c.ff);
     }
     mq = std::max(mq, l.Cql); mo = std::max(mo, l.Col);
@@ -515,6 +555,11 @@ extern "C" int dn_seq_model_create(const dn_seq_cfg* cfg, const dn_seq_layer_cfg
   DA(m->attn_count, (size_t)AT_SPLIT_ROWS * mh * 4);
   if (tab > 0) DA(m->dist_tab, (tab + 32) * 4);      // (rows without a query read up to 32 entries whatever the span)
   DA(m->sgate, MB * 4);
+  {
+    size_t mm = 0;
+    for (auto& l : m->L) if (n_maps(l.c) == 2) mm = std::max(mm, (size_t)2 * l.Co);
+    if (mm) DA(m->maps32, MB * mm * 4);
+  }
   if (looped) { DA(m->x0, MB * W * 4); DA(m->cat, MB * 2 * W * e); }
   if (any_wkv) DA(m->xm, (size_t)SHIFT_MAX * MB * W * e);
   if (cfg->canon_taps > 0) DA(m->hn, MB * W * e);
@@ -551,6 +596,7 @@ extern "C" int dn_seq_model_create(const dn_seq_cfg* cfg, const dn_seq_layer_cfg
         if (l.c.mlp_kind == DN_MLP_MOE && l.c.ff > 0)
           l.x_eact_ok = make_tmap(&l.x_eact[0], m->eact, m->MB * l.c.top, l.c.ff, 64) && make_tmap(&l.x_eact[1], m->eact, m->MB * l.c.top, l.c.ff, 128);
     }
+    if (cfg->side_dim > 0) make_xmaps(&m->x_side, m->act, m->MB, cfg->side_dim);
     if (m->cat) make_xmaps(&m->x_cat, m->cat, m->MB, 2 * cfg->width);
     if (m->xm) for (int i = 0; i < SHIFT_MAX; i++) make_xmaps(&m->x_xm[i], (char*)m->xm + (size_t)i * MB * W * e, m->MB, cfg->width);
   }
@@ -578,7 +624,7 @@ extern "C" int dn_seq_bind(dn_seq_model* m, int layer, int which, const void* p)
     else if (which == DN_SQ_HEAD) {
       m->head = p;
       m->tm_head_ok = b16 && make_tmap(&m->tm_head, p, m->cfg.vocab, m->cfg.width, dn::TC_BM);
-    } else if (which > DN_SQ_HEAD && which <= DN_SQ_POS) {
+    } else if (which > DN_SQ_HEAD && which <= DN_SQ_SIDE_EMBED) {
       m->mw[which - DN_SQ_EMBED] = p;
       if (which == DN_SQ_LOOP_IN) m->tm_loop_ok = b16 && make_tmap(&m->tm_loop_in, p, m->cfg.width, 2 * m->cfg.width, dn::TC_BM);
     } else return fail(DN_EINVAL, "tensor %d is not a model tensor", which);
@@ -587,6 +633,7 @@ extern "C" int dn_seq_bind(dn_seq_model* m, int layer, int which, const void* p)
   if (layer >= (int)m->L.size() || which < 0 || which >= DN_SQ_COUNT) return fail(DN_EINVAL, "layer %d / tensor %d out of range", layer, which);
   SeqLayer& l = m->L[layer];
   l.w[which] = p;
+  if (which == DN_SQ_LQ1 || which == DN_SQ_LK1 || which == DN_SQ_LQ2 || which == DN_SQ_LK2) m->lam_stale = true;
   int rows = 0, cols = m->cfg.width;
   switch (which) {
     case DN_SQ_Q: rows = l.Cq; if (l.c.mixer == DN_MIX_LATENT && l.c.q_rank > 0) cols = l.c.q_rank; break;
@@ -600,6 +647,8 @@ extern "C" int dn_seq_bind(dn_seq_model* m, int layer, int which, const void* p)
     case DN_SQ_O: rows = m->cfg.width; cols = l.Co; break;
     case DN_SQ_DOWN: rows = m->cfg.width; cols = l.c.ff; break;
     case DN_SQ_HEAD_GATE: rows = l.c.heads; break;
+    case DN_SQ_SIDE_GATE: rows = m->cfg.side_dim; break;
+    case DN_SQ_SIDE_PROJ: rows = m->cfg.width; cols = m->cfg.side_dim; break;
     case DN_SQ_R_Q: case DN_SQ_R_K: case DN_SQ_R_A: rows = l.Rc; break;
     case DN_SQ_R_V: case DN_SQ_R_G: rows = l.Rv; break;
     case DN_SQ_R_O: rows = m->cfg.width; cols = l.Rv; break;
@@ -731,10 +780,11 @@ constexpr int ROWS_PAIR = 2048;      // output features from which a warp of the
 struct LinMaps { const CUtensorMap* w; const CUtensorMap* w2; const XMaps* x; };
 template <class T>
 static cudaError_t linear(dn_seq_model* m, cudaStream_t s, const T* X, const void* W, const void* W2, void* Y, int N, int O, int K, bool out32,
-                          int act, LinMaps tm = LinMaps{nullptr, nullptr, nullptr}, float alim = 0.f, const void* bias = nullptr) {
+                          int act, LinMaps tm = LinMaps{nullptr, nullptr, nullptr}, float alim = 0.f, const void* bias = nullptr, const LinEpi<T>* ep = nullptr) {
+  const LinEpi<T> epi = ep ? *ep : LinEpi<T>{nullptr, nullptr, 0, nullptr, nullptr, 1.f, {nullptr, nullptr, nullptr, nullptr}};
   // (a weight of fewer than 128 rows fills part of a tile: still far ahead of the CUDA-core tiles once K is in the thousands)
   if (std::is_same<T, bf16>::value && N >= 16 && O >= 16 && tm.w && tm.x && tm.x->ok && (!bias || act == ACT_RELU2 || (act == ACT_NONE && out32)) &&
-      (act == ACT_NONE || act == ACT_TANH || act == ACT_RELU2 || (act_two(act) && tm.w2))) {
+      (act == ACT_NONE || act == ACT_TANH || act == ACT_RELU2 || act == ACT_GELU_TAB || act == ACT_JOIN || (act_two(act) && tm.w2))) {
     dn::TcParams p;
     memset(&p, 0, sizeof(p));
     p.T = N; p.N = O; p.K = K; p.ldy = O; p.Y = (dn::bf16*)Y; p.err = m->tc_err; p.limit = alim; p.bias = (const dn::bf16*)bias;
@@ -742,6 +792,15 @@ static cudaError_t linear(dn_seq_model* m, cudaStream_t s, const T* X, const voi
     if (act == ACT_SWIGLU) return gemm_tc<dn::EPI_SGLU>(*tm.w, *tm.w2, *tm.x, p, s);
     if (act == ACT_RELU2) return gemm_tc<dn::EPI_RELU2>(*tm.w, *tm.w, *tm.x, p, s);
     if (act == ACT_TANH) return gemm_tc<dn::EPI_TANH>(*tm.w, *tm.w, *tm.x, p, s);
+    if (act == ACT_GELU_TAB) {
+      p.tab = (const dn::bf16*)epi.tab; p.row = epi.row; p.tab_ld = epi.ld;
+      return gemm_tc<dn::EPI_GELU_TAB>(*tm.w, *tm.w, *tm.x, p, s);
+    }
+    if (act == ACT_JOIN) {
+      p.x = epi.x; p.ls = (const dn::bf16*)epi.ls; p.mul = epi.mul;
+      p.nw = (const dn::bf16*)epi.nx.w; p.nb = (const dn::bf16*)epi.nx.b; p.nalpha = (const dn::bf16*)epi.nx.alpha; p.nh = (dn::bf16*)epi.nx.h;
+      return gemm_tc<dn::EPI_JOIN>(*tm.w, *tm.w, *tm.x, p, s);
+    }
     if (act) return gemm_tc<dn::EPI_GEGLU>(*tm.w, *tm.w2, *tm.x, p, s);
     if (out32) return gemm_tc<dn::EPI_STORE_F32>(*tm.w, *tm.w, *tm.x, p, s);
     return gemm_tc<dn::EPI_STORE>(*tm.w, *tm.w, *tm.x, p, s);
@@ -750,14 +809,14 @@ static cudaError_t linear(dn_seq_model* m, cudaStream_t s, const T* X, const voi
     const bool two = act_two(act), pair = !two && O >= ROWS_PAIR;
     const int per = pair ? 2 : 1;
     dim3 grid((O + 8 * per - 1) / (8 * per));
-#define LR(NT) (two || pair ? launch(k_linear_rows<T, NT, true>, grid, dim3(256), 0, s, X, (const T*)W, (const T*)W2, Y, out32 ? 1 : 0, N, O, K, act, per, alim, (const T*)bias) \
-                            : launch(k_linear_rows<T, NT, false>, grid, dim3(256), 0, s, X, (const T*)W, (const T*)W2, Y, out32 ? 1 : 0, N, O, K, act, per, alim, (const T*)bias))
+#define LR(NT) (two || pair ? launch(k_linear_rows<T, NT, true>, grid, dim3(256), 0, s, X, (const T*)W, (const T*)W2, Y, out32 ? 1 : 0, N, O, K, act, per, alim, (const T*)bias, epi) \
+                            : launch(k_linear_rows<T, NT, false>, grid, dim3(256), 0, s, X, (const T*)W, (const T*)W2, Y, out32 ? 1 : 0, N, O, K, act, per, alim, (const T*)bias, epi))
     return N == 1 ? LR(1) : N == 2 ? LR(2) : N <= 4 ? LR(4) : LR(8);
 #undef LR
   }
   dim3 grid((O + 63) / 64, (N + 63) / 64);
-  if (out32) return launch(k_linear<T, true>, grid, dim3(256), 0, s, X, (const T*)W, (const T*)W2, Y, N, O, K, act, alim, (const T*)bias);
-  return launch(k_linear<T, false>, grid, dim3(256), 0, s, X, (const T*)W, (const T*)W2, Y, N, O, K, act, alim, (const T*)bias);
+  if (out32) return launch(k_linear<T, true>, grid, dim3(256), 0, s, X, (const T*)W, (const T*)W2, Y, N, O, K, act, alim, (const T*)bias, epi);
+  return launch(k_linear<T, false>, grid, dim3(256), 0, s, X, (const T*)W, (const T*)W2, Y, N, O, K, act, alim, (const T*)bias, epi);
 }
 
 // Attention of a step: bf16 steps that bring a prompt portion (an entry of 16 tokens or more) run on the MMA tiles when
@@ -766,24 +825,27 @@ template <class T>
 static bool attn_tiles_ok(const dn_seq_layer_cfg& lc, const Batch& b) {
   return std::is_same<T, bf16>::value && b.max_len >= 16 && lc.dim % 8 == 0 && lc.vdim % 8 == 0 && lc.dim <= 128 && lc.vdim <= 128;
 }
-template <int DKP, int DVP, bool SIG>
+template <int DKP, int DVP, bool SIG, int MAPS>
 static cudaError_t attn_tiles_launch(cudaStream_t s, const Batch& b, const bf16* q, const bf16* kp, const bf16* vp, const dn_seq_layer_cfg& lc,
                                      const AttnExtra& ex, bf16* out) {
-  constexpr size_t smem = ((size_t)2 * AT_ROWS * (DKP + 8) + (size_t)AT_ROWS * (DVP + 8)) * 2;
+  constexpr size_t smem = ((size_t)2 * MAPS * AT_ROWS * (DKP + 8) + (size_t)AT_ROWS * (DVP + 8)) * 2;
+  static_assert(MAPS == 1 || smem >= (size_t)AT_ROWS * (DVP + 4) * 4, "the second map's rows pass through the tiles' memory");
   static bool attr = false;
   if (!attr) {
-    cudaError_t e = cudaFuncSetAttribute(k_attn_tiles<DKP, DVP, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(k_attn_tiles<DKP, DVP, SIG, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return e;
     attr = true;
   }
   g_launches++;
-  k_attn_tiles<DKP, DVP, SIG><<<dim3(b.row_tiles, lc.heads), 128, smem, s>>>(b, q, kp, vp, lc.heads, lc.kv_heads, lc.dim, lc.vdim, lc.chunk, lc.scale, ex, out);
+  k_attn_tiles<DKP, DVP, SIG, MAPS><<<dim3(b.row_tiles, lc.heads), 128 * MAPS, smem, s>>>(b, q, kp, vp, lc.heads * MAPS, lc.kv_heads * MAPS, lc.dim, lc.vdim, lc.chunk,
+                                                                                          lc.scale, ex, out);
   return cudaGetLastError();
 }
 static cudaError_t attn_tiles(cudaStream_t s, const Batch& b, const bf16* q, const bf16* kp, const bf16* vp, const dn_seq_layer_cfg& lc,
                               const AttnExtra& ex, bf16* out) {
   const int kq = lc.dim <= 32 ? 0 : lc.dim <= 64 ? 1 : 2, vq = lc.vdim <= 32 ? 0 : lc.vdim <= 64 ? 1 : 2;
-#define AT(a, c, A, Cc) if (kq == a && vq == c) return ex.off ? attn_tiles_launch<A, Cc, true>(s, b, q, kp, vp, lc, ex, out) : attn_tiles_launch<A, Cc, false>(s, b, q, kp, vp, lc, ex, out);
+#define AT(a, c, A, Cc) if (kq == a && vq == c) return ex.maps == 2 ? attn_tiles_launch<A, Cc, false, 2>(s, b, q, kp, vp, lc, ex, out) \
+                                     : ex.off ? attn_tiles_launch<A, Cc, true, 1>(s, b, q, kp, vp, lc, ex, out) : attn_tiles_launch<A, Cc, false, 1>(s, b, q, kp, vp, lc, ex, out);
   AT(0, 0, 32, 32) AT(0, 1, 32, 64) AT(0, 2, 32, 128) AT(1, 0, 64, 32) AT(1, 1, 64, 64) AT(1, 2, 64, 128)
   AT(2, 0, 128, 32) AT(2, 1, 128, 64) AT(2, 2, 128, 128)
 #undef AT
@@ -822,36 +884,36 @@ template <class T>
 static int attn_rows_stages(const dn_seq_layer_cfg& lc, int N) {      // 0: not this kernel
   const int esz = (int)sizeof(T);
   if (N > AT_SPLIT_ROWS || lc.pool > 0 || lc.dim > 128 || lc.vdim > 128 || (lc.dim * esz) % 16 || (lc.vdim * esz) % 16) return 0;
-  const bool one = lc.chunk > 0 && lc.chunk <= AT_MAX_SPLITS * AR_KEYS;
+  const bool one = lc.chunk > 0 && lc.chunk + lc.keep_first <= AT_MAX_SPLITS * AR_KEYS;
   for (int st = one ? 1 : 2; st > 0; st--)
-    if (ar_smem_bytes(lc.dim, lc.vdim, esz, lc.v_is_k != 0, st, 4) + 1024 <= g_max_smem) return st;
+    if (ar_smem_bytes(lc.dim * n_maps(lc), lc.vdim, esz, lc.v_is_k != 0, st, 4, n_maps(lc)) + 1024 <= g_max_smem) return st;
   return 0;
 }
-template <class T, bool SIG, int HB>
+template <class T, bool SIG, int HB, int MAPS>
 static cudaError_t attn_rows_launch(dn_seq_model* m, cudaStream_t s, const Batch& b, const T* q, const T* kp, const T* vp, const dn_seq_layer_cfg& lc, const AttnExtra& ex,
                                     int stages, int Z, T* out) {
-  const size_t smem = ar_smem_bytes(lc.dim, lc.vdim, (int)sizeof(T), lc.v_is_k != 0, stages, HB);
+  const size_t smem = ar_smem_bytes(lc.dim * MAPS, lc.vdim, (int)sizeof(T), lc.v_is_k != 0, stages, HB, MAPS);
   static size_t attr = 40 * 1024;      // (the default limit counts the static part too)
   if (smem > attr) {
-    cudaError_t e = cudaFuncSetAttribute(k_attn_rows<T, SIG, HB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(k_attn_rows<T, SIG, HB, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return e;
     attr = smem;
   }
   const int R = lc.heads / lc.kv_heads, per = (R + HB - 1) / HB;
-  return launch(k_attn_rows<T, SIG, HB>, dim3(b.N, lc.kv_heads * per, Z), dim3(AR_WARPS * 32), smem, s, b, q, kp, vp, lc.heads, lc.kv_heads, lc.dim, lc.vdim, lc.chunk,
+  return launch(k_attn_rows<T, SIG, HB, MAPS>, dim3(b.N, lc.kv_heads * per, Z), dim3(AR_WARPS * 32), smem, s, b, q, kp, vp, lc.heads * MAPS, lc.kv_heads * MAPS, lc.dim, lc.vdim, lc.chunk,
                 lc.scale, stages, ex, out, m->attn_part, m->attn_count);
 }
 template <class T>
 static cudaError_t attn_rows(dn_seq_model* m, cudaStream_t s, const Batch& b, const T* q, const T* kp, const T* vp, const dn_seq_layer_cfg& lc, const AttnExtra& ex,
                              int stages, T* out) {
   // (a mask of `chunk` positions bounds the keys of a row, and with them its splits)
-  const int Z = lc.chunk > 0 ? std::min((int)AT_MAX_SPLITS, (lc.chunk + AR_KEYS - 1) / AR_KEYS) : AT_MAX_SPLITS;
+  const int Z = lc.chunk > 0 ? std::min((int)AT_MAX_SPLITS, (lc.chunk + lc.keep_first + AR_KEYS - 1) / AR_KEYS) : AT_MAX_SPLITS;
   const int R = lc.heads / lc.kv_heads;
   auto blocks = [&](int hb) { return (long long)b.N * lc.kv_heads * ((R + hb - 1) / hb) * Z; };
   const int hb = R == 1 || blocks(1) <= 2 * g_sms ? 1 : R == 2 || blocks(2) <= 2 * g_sms ? 2 : 4;      // the most blocks that the SMs take at once
-#define AR(SIGv) (hb == 1 ? attn_rows_launch<T, SIGv, 1>(m, s, b, q, kp, vp, lc, ex, stages, Z, out) \
-                : hb == 2 ? attn_rows_launch<T, SIGv, 2>(m, s, b, q, kp, vp, lc, ex, stages, Z, out) : attn_rows_launch<T, SIGv, 4>(m, s, b, q, kp, vp, lc, ex, stages, Z, out))
-  return ex.off ? AR(true) : AR(false);
+#define AR(SIGv, MP) (hb == 1 ? attn_rows_launch<T, SIGv, 1, MP>(m, s, b, q, kp, vp, lc, ex, stages, Z, out) \
+                    : hb == 2 ? attn_rows_launch<T, SIGv, 2, MP>(m, s, b, q, kp, vp, lc, ex, stages, Z, out) : attn_rows_launch<T, SIGv, 4, MP>(m, s, b, q, kp, vp, lc, ex, stages, Z, out))
+  return ex.maps == 2 ? AR(false, 2) : ex.off ? AR(true, 1) : AR(false, 1);
 #undef AR
 }
 
@@ -1052,8 +1114,10 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
   };
   // a sublayer's output a y (+ b y2) joins the residual, through the norm after the sublayer where the model has one
   const NextNorm<T> no_next{nullptr, nullptr, nullptr, nullptr};
-  // the norm before the sublayer that follows, when the joining kernel can produce it (plain residual, both norms dynamic tanh)
-  const bool can_fuse_next = c.post_norm && dyt && S <= 0;
+  // sublayer outputs join the plain residual as they are, or scaled per channel: in the product's epilogue where there is one product
+  const bool sjoin = !c.post_norm && pre && S <= 0 && !c.parallel_ff && (dyt || c.layer_scale || c.side_dim > 0);
+  // the norm before the sublayer that follows, when the joining kernel can produce it (plain residual, a dynamic tanh)
+  const bool can_fuse_next = (c.post_norm || sjoin) && dyt && S <= 0;
   auto next_norm = [&](const SeqLayer& nl, int which) {
     return NextNorm<T>{(const T*)nl.w[which], (const T*)nl.w[which == DN_SQ_NORM1 ? DN_SQ_NORM1_B : DN_SQ_NORM2_B],
                        (const T*)nl.w[which == DN_SQ_NORM1 ? DN_SQ_NORM1_ALPHA : DN_SQ_NORM2_ALPHA], (T*)m->h};
@@ -1063,7 +1127,10 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
     auto w = [&](int i) { return (const T*)l.w[i]; };
     if (c.post_norm && !dyt)      // RMS norm of the sublayer's output, added to the plain residual; h = T(x) for a model without norms before
       return launch(k_rms_join<T>, dim3(N), nthr, nsm, s, m->xs, W, ms ? (const float*)nullptr : (const float*)m->y, a, y2, bb,
-                    ms ? *ms : no_moe, w(post), 1, c.eps, pre ? (T*)nullptr : (T*)m->h);
+                    ms ? *ms : no_moe, w(post), 1, c.eps, pre ? (T*)nullptr : (T*)m->h, no_next);
+    if (sjoin)
+      return launch(k_scale_join<T>, dim3(ew), dim3(256), 0, s, m->xs, NW, W, (const float*)m->y, a, y2, bb,
+                    c.layer_scale ? w(post == DN_SQ_POST1 ? DN_SQ_LS1 : DN_SQ_LS2) : (const T*)nullptr, nx);
     if (c.post_norm) {
       if (S <= 0) return launch(k_dyt_add<T>, dim3(ew), dim3(256), 0, s, m->xs, NW, W, (const float*)m->y, a, y2, bb, w(post), w(post + 1), w(post + 2), nx);
       cudaError_t e = launch(k_dyt_inplace<T>, dim3(ew), dim3(256), 0, s, m->y, NW, W, a, y2, bb, w(post), w(post + 1), w(post + 2));
@@ -1100,18 +1167,19 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
     }
     return DN_OK;
   };
-  // a dense feed-forward: h [N, W] -> y [N, W] fp32
-  auto dense_ff = [&](SeqLayer& l, int N, float* y) -> int {
+  // a dense feed-forward: h [N, W] -> y [N, W] fp32, or (ep) straight into the residual
+  auto dense_ff = [&](SeqLayer& l, int N, float* y, const LinEpi<T>* ep = nullptr) -> int {
     const dn_seq_layer_cfg& lc = l.c;
     auto wm = [&](int i) { return l.tm_ok[i] ? &l.tm[i] : (const CUtensorMap*)nullptr; };
     PH(DN_SEQ_PH_FF_UP);
     if (lc.ff_act == DN_FF_RELU2)      // no gate: relu(W_up h + b)^2
       CK(linear<T>(m, s, (const T*)m->h, l.w[DN_SQ_UP], nullptr, m->act, N, lc.ff, W, false, ACT_RELU2, LinMaps{wm(DN_SQ_UP), nullptr, &m->x_h}, 0.f, l.w[DN_SQ_UP_B]));
     else
-      CK(linear<T>(m, s, (const T*)m->h, l.w[DN_SQ_GATE], l.w[DN_SQ_UP], m->act, N, lc.ff, W, false, ACT_GEGLU, LinMaps{wm(DN_SQ_GATE), wm(DN_SQ_UP), &m->x_h}));
+      CK(linear<T>(m, s, (const T*)m->h, l.w[DN_SQ_GATE], l.w[DN_SQ_UP], m->act, N, lc.ff, W, false, lc.ff_act == DN_FF_SWIGLU ? ACT_SWIGLU : ACT_GEGLU,
+                   LinMaps{wm(DN_SQ_GATE), wm(DN_SQ_UP), &m->x_h}));
     PH(DN_SEQ_PH_FF_DOWN);
-    CK(linear<T>(m, s, (const T*)m->act, l.w[DN_SQ_DOWN], nullptr, y, N, W, lc.ff, true, 0, LinMaps{wm(DN_SQ_DOWN), nullptr, &l.x_act}, 0.f,
-                 lc.ff_act == DN_FF_RELU2 ? l.w[DN_SQ_DOWN_B] : nullptr));
+    CK(linear<T>(m, s, (const T*)m->act, l.w[DN_SQ_DOWN], nullptr, y, N, W, lc.ff, true, ep ? ACT_JOIN : ACT_NONE, LinMaps{wm(DN_SQ_DOWN), nullptr, &l.x_act}, 0.f,
+                 lc.ff_act == DN_FF_RELU2 ? l.w[DN_SQ_DOWN_B] : nullptr, ep));
     return DN_OK;
   };
   bool h_ready = !pre;
@@ -1139,6 +1207,11 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
     // what the join after this run's last sublayer can prepare: the next run's first norm, unless a loop pass starts there
     const bool next_ok = can_fuse_next && ri + 1 < (int)m->runs.size() && !m->runs[ri + 1].inject;
     const NextNorm<T> nx_run = next_ok ? next_norm(m->L[m->runs[ri + 1].layer], DN_SQ_NORM1) : no_next;
+    // what follows the layer's last sublayer: the token input, which reads the residual itself, or the next run's norm
+    const NextNorm<T> nx_last = c.side_dim > 0 ? NextNorm<T>{nullptr, nullptr, nullptr, (T*)m->h} : nx_run;
+    auto join_epi = [&](int ls, const NextNorm<T>& nx) {
+      return LinEpi<T>{nullptr, nullptr, 0, m->xs, c.layer_scale ? w(ls) : (const T*)nullptr, rmul, nx};
+    };
     T* cst = (T*)m->conv_state + run.conv_off;
     float* st = m->delta_state + run.state_off;
     const bool few = N <= 8;      // a decode step: all projections of the mixer in one launch of the row kernel
@@ -1181,23 +1254,25 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
       }
     }
     if (lc.mixer == DN_MIX_ATTENTION || lc.mixer == DN_MIX_PARALLEL) {
-      AttnPrep a{lc.heads, lc.kv_heads, lc.dim, lc.vdim, lc.conv, lc.rot_dims, l.Ck ? 1 : 0, lc.qk_norm, c.eps, l.inv_freq,
-                 lc.v_is_k ? 0 : 1, lc.rot_layout == DN_ROT_HALF ? 1 : 0, lc.yarn_factor > 0.f ? 0.1f * logf(lc.yarn_factor) + 1.f : 1.f,
-                 lc.qtemp_coef, lc.qtemp_every, lc.conv > 0 && b.max_len == 1 ? 1 : 0};
+      const int maps = n_maps(lc), Hm = lc.heads * maps, Gm = lc.kv_heads * maps;      // heads and key heads, every map counted
+      AttnPrep a{Hm, Gm, lc.dim, lc.vdim, lc.conv, lc.rot_dims, l.Ck ? 1 : 0, lc.qk_norm, c.eps, l.inv_freq,
+                 lc.v_is_k ? 0 : 1, lc.rot_layout == DN_ROT_HALF ? 1 : 0, rot_mscale(lc),
+                 lc.qtemp_coef, lc.qtemp_every, lc.conv > 0 && b.max_len == 1 ? 1 : 0, lc.kv_heads};
       // values that are the keys: the value pool is the key pool (row stride G dk); the pooled rows likewise
       const void* vpl = lc.v_is_k ? m->kpool[run.kv_index] : m->vpool[run.kv_index];
       void* pkp = m->pkpool[run.kv_index];
       void* pvp = lc.v_is_k ? pkp : m->pvpool[run.kv_index];
-      const int Ckk = lc.kv_heads * lc.dim;
+      const int Ckk = Gm * lc.dim;
       AttnExtra ex{lc.softcap, lc.sink ? l.w[DN_SQ_SINK] : nullptr, lc.out_gate ? (const float*)m->pa : nullptr, lc.mask_kind == DN_MASK_WINDOW ? 1 : 0,
                    lc.v_is_k ? Ckk : 0, lc.pool, pkp, pvp, lc.dist_bias ? l.w[DN_SQ_DIST1] : nullptr, lc.dist_bias ? l.w[DN_SQ_DIST2] : nullptr,
-                   lc.attn_weight == DN_ATTN_SIGMOID ? l.w[DN_SQ_ATTN_OFF] : nullptr};
-      const size_t sm = ((size_t)l.Cq + l.Ck + 40 + lc.heads + lc.kv_heads + lc.rot_dims) * 4;
+                   lc.attn_weight == DN_ATTN_SIGMOID ? l.w[DN_SQ_ATTN_OFF] : nullptr,
+                   lc.keep_first, maps, l.lam, 1.f - lc.diff, c.eps, nullptr};
+      const size_t sm = ((size_t)l.Cq + l.Ck + 40 + Hm + Gm + lc.rot_dims) * 4;
       PH(DN_SEQ_PH_ATTN_PREP);
       // heads that do not rotate and are normed alone (or not at all): a warp a head (a function of the model, not of the batch)
       uintptr_t al = (uintptr_t)cst | (m->conv_stride * sizeof(T));
       for (int q : {DN_SQ_Q_CONV, DN_SQ_K_CONV, DN_SQ_V_CONV, DN_SQ_Q_NORM, DN_SQ_K_NORM}) al |= (uintptr_t)l.w[q];
-      const bool by_head = lc.rot_dims == 0 && lc.qk_norm != DN_QKNORM_WHOLE && lc.dim % 4 == 0 && lc.vdim % 4 == 0 && lc.dim <= 128 && lc.vdim <= 128 &&
+      const bool by_head = lc.rot_dims == 0 && maps == 1 && lc.qk_norm != DN_QKNORM_WHOLE && lc.dim % 4 == 0 && lc.vdim % 4 == 0 && lc.dim <= 128 && lc.vdim <= 128 &&
                            lc.conv <= PREP_MAX_TAPS && (al & (4 * sizeof(T) - 1)) == 0;
       if (by_head) {
         const int units = lc.heads + (l.Ck ? lc.kv_heads : 0) + (l.Cv ? lc.kv_heads : 0), tok = N > 64 ? 8 : 1;
@@ -1223,12 +1298,15 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
       else {
         // a small step (decode): long rows are split over up to AT_MAX_SPLITS blocks, joined by k_attn_merge
         // (a mask of `chunk` positions bounds the keys of a row, and with them its splits)
-        const int zcap = lc.chunk > 0 && lc.pool == 0 ? std::min((int)AT_MAX_SPLITS, (lc.chunk + AT_SPLIT_KEYS - 1) / AT_SPLIT_KEYS) : AT_MAX_SPLITS;
+        const int zcap = lc.chunk > 0 && lc.pool == 0 ? std::min((int)AT_MAX_SPLITS, (lc.chunk + lc.keep_first + AT_SPLIT_KEYS - 1) / AT_SPLIT_KEYS) : AT_MAX_SPLITS;
         const int Z = N <= AT_SPLIT_ROWS ? zcap : 1;
-        CK(launch(ex.off ? k_attn<T, 8, true> : k_attn<T, 8, false>, dim3(N, lc.heads, Z), dim3(AT_WARPS * 32), (size_t)(((lc.dim + 3) & ~3) + AT_WARPS * (2 + (lc.vdim + 31) / 32 * 32)) * 4, s, b,
+        if (maps == 2) ex.out32 = m->maps32;
+        CK(launch(ex.off ? k_attn<T, 8, true> : k_attn<T, 8, false>, dim3(N, Hm, Z), dim3(AT_WARPS * 32), (size_t)(((lc.dim + 3) & ~3) + AT_WARPS * (2 + (lc.vdim + 31) / 32 * 32)) * 4, s, b,
                   (const T*)m->qb, (const T*)m->kpool[run.kv_index],
-                  (const T*)vpl, lc.heads, lc.kv_heads, lc.dim, lc.vdim, lc.chunk, lc.scale, ex, (T*)m->mo, m->attn_part));
-        if (Z > 1) CK(launch(k_attn_merge<T>, dim3(N, lc.heads), dim3(128), 0, s, b, lc.heads, lc.vdim, lc.chunk, Z, ex, (const float*)m->attn_part, (T*)m->mo));
+                  (const T*)vpl, Hm, Gm, lc.dim, lc.vdim, lc.chunk, lc.scale, ex, (T*)m->mo, m->attn_part));
+        if (Z > 1) CK(launch(k_attn_merge<T>, dim3(N, Hm), dim3(128), 0, s, b, Hm, lc.vdim, lc.chunk, Z, ex, (const float*)m->attn_part, (T*)m->mo));
+        if (maps == 2)
+          CK(launch(k_diff_join<T>, dim3((N * lc.heads + 7) / 8), dim3(256), 0, s, (const float*)m->maps32, N * lc.heads, lc.vdim, (const float*)l.lam, ex.post, c.eps, (T*)m->mo));
       }
     } else if (lc.mixer == DN_MIX_LATENT) {
       // projections: q (or its latent, normed, then up), the key/value latent row, the heads' gates
@@ -1237,12 +1315,13 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
       void* q1 = lc.q_rank > 0 ? m->lr : m->uq;
       const int q1w = lc.q_rank > 0 ? lc.q_rank : l.Cq, q1t = lc.q_rank > 0 ? DN_SQ_DQ : DN_SQ_Q;
       if (few) {
-        add(nullptr, q1t, q1, q1w, 0); add(nullptr, DN_SQ_DKV, m->uk, l.Ck, 0);
+        add(nullptr, q1t, q1, q1w, 0);
+        if (lc.kv_from < 0) add(nullptr, DN_SQ_DKV, m->uk, l.Ck, 0);
         if (lc.out_gate) add(nullptr, DN_SQ_HEAD_GATE, m->pa, lc.heads, 1);
         CK(run_segs());
       } else {
         CK(linear<T>(m, s, (const T*)m->h, l.w[q1t], nullptr, q1, N, q1w, W, false, 0, LinMaps{wm(q1t), nullptr, &m->x_h}));
-        CK(linear<T>(m, s, (const T*)m->h, l.w[DN_SQ_DKV], nullptr, m->uk, N, l.Ck, W, false, 0, LinMaps{wm(DN_SQ_DKV), nullptr, &m->x_h}));
+        if (lc.kv_from < 0) CK(linear<T>(m, s, (const T*)m->h, l.w[DN_SQ_DKV], nullptr, m->uk, N, l.Ck, W, false, 0, LinMaps{wm(DN_SQ_DKV), nullptr, &m->x_h}));
         if (lc.out_gate)
           CK(linear<T>(m, s, (const T*)m->h, l.w[DN_SQ_HEAD_GATE], nullptr, m->pa, N, lc.heads, W, true, 0, LinMaps{wm(DN_SQ_HEAD_GATE), nullptr, &m->x_h}));
       }
@@ -1251,7 +1330,7 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
         CK(linear<T>(m, s, (const T*)m->lr, l.w[DN_SQ_Q], nullptr, m->uq, N, l.Cq, lc.q_rank, false, 0, LinMaps{wm(DN_SQ_Q), nullptr, &l.x_lr}));
       }
       PH(DN_SEQ_PH_LATENT_IN);
-      LatentPrep a{lc.heads, lc.dim, dr, R, lc.rot_dims, lc.rot_layout == DN_ROT_HALF ? 1 : 0, c.eps, l.inv_freq};
+      LatentPrep a{lc.heads, lc.dim, dr, R, lc.rot_dims, lc.rot_layout == DN_ROT_HALF ? 1 : 0, c.eps, l.inv_freq, rot_mscale(lc), lc.kv_from < 0 ? 1 : 0};
       T* pool = (T*)m->kpool[run.kv_index];
       CK(launch(k_latent_prep<T>, dim3(N), dim3(256), 0, s, a, b, (const T*)m->uq, (const T*)m->uk, w(DN_SQ_DKV_NORM), (T*)m->qb, pool));
       // the unrotated query parts into the latent space: qb[n, h, 0:R] = W_uk,h^T q[n, h, 0:dim]
@@ -1268,7 +1347,7 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
                   HeadsGeom{l.Cq, dq, l.Cql, l.Ck, (size_t)lc.dim * R, 1, R}));
       // multi-query attention of all heads over the cached rows: keys [R + dr], values = their first R numbers
       PH(DN_SEQ_PH_ATTN);
-      AttnExtra ex{lc.softcap, nullptr, lc.out_gate ? (const float*)m->pa : nullptr, lc.mask_kind == DN_MASK_WINDOW ? 1 : 0, l.Ck};
+      AttnExtra ex{lc.softcap, lc.sink ? l.w[DN_SQ_SINK] : nullptr, lc.out_gate ? (const float*)m->pa : nullptr, lc.mask_kind == DN_MASK_WINDOW ? 1 : 0, l.Ck};
       if (std::is_same<T, bf16>::value && latent_tiles_ok(b, l.Ck, R) && (b.max_len >= 16 || b.max_len == 1))
         CK(latent_tiles(s, b, (const bf16*)m->qb, (const bf16*)pool, lc.heads, l.Ck, R, lc.chunk, lc.scale, ex, (bf16*)m->gt, m->attn_part, 2 + m->part_dv));
       else {
@@ -1355,7 +1434,12 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
       CK(launch(k_conv_carry<T>, dim3((std::max(l.Cq, std::max(l.Ck, l.Cv)) + 127) / 128, b.E, 3), dim3(128), 0, s, cs, lc.conv, b, cst, m->conv_stride));
     }
     PH(DN_SEQ_PH_OUT_PROJ);
-    if (ride) {
+    const NextNorm<T> nx_mix = lc.ff > 0 ? (can_fuse_next ? next_norm(l, DN_SQ_NORM2) : no_next) : nx_last;
+    const bool out_joins = sjoin && lc.mixer != DN_MIX_PARALLEL;
+    if (out_joins) {
+      const LinEpi<T> ep = join_epi(DN_SQ_LS1, nx_mix);
+      CK(linear<T>(m, s, (const T*)m->mo, l.w[DN_SQ_O], nullptr, nullptr, N, W, l.Co, true, ACT_JOIN, LinMaps{wm(DN_SQ_O), nullptr, &l.x_mo}, 0.f, nullptr, &ep));
+    } else if (ride) {
       memset(&sg, 0, sizeof(sg));
       add(m->mo, DN_SQ_O, m->y, W, 1, ACT_NONE, l.Co); add(m->act, DN_SQ_DOWN, m->y2, W, 1, ACT_NONE, lc.ff);
       CK(run_segs());
@@ -1469,8 +1553,8 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
       ja = rmul * lc.left_scale; jb = rmul * lc.right_scale; jy2 = m->y2;
     }
     PH(DN_SEQ_PH_WRITE_BACK);
-    const NextNorm<T> nx_mix = lc.ff > 0 ? (can_fuse_next ? next_norm(l, DN_SQ_NORM2) : no_next) : nx_run;
-    if (lc.mixer == DN_MIX_PARALLEL && lc.branch_norm)
+    if (out_joins) {
+    } else if (lc.mixer == DN_MIX_PARALLEL && lc.branch_norm)
       CK(launch(k_rms2_join<T>, dim3(N), nthr, 0, s, m->xs, W, (const float*)m->y, ja, w(DN_SQ_L_OUT), jy2, jb, w(DN_SQ_R_OUT), c.eps));
     else
       CK(join(l, DN_SQ_POST1, DN_SQ_HC1_MIX, DN_SQ_HC1_OUT, ja, jy2, jb, nx_mix));
@@ -1492,15 +1576,26 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
           const MoeSrc<T> ms{m->eo, m->rwt, m->rpos, m->ridx, lc.top, scored ? lc.experts : INT32_MAX, (const T*)m->h,
                              lc.shared_ff > 0 ? (const float*)m->y2 : (const float*)nullptr, lc.shared_gate ? (const float*)m->sgate : (const float*)nullptr};
           CK(join(l, DN_SQ_POST2, DN_SQ_HC2_MIX, DN_SQ_HC2_OUT, 1.f, nullptr, 0.f, no_next, &ms));
-        } else if (!fused) CK(join(l, DN_SQ_POST2, DN_SQ_HC2_MIX, DN_SQ_HC2_OUT, rmul, lc.shared_ff > 0 ? (const float*)m->y2 : nullptr, rmul, nx_run));
+        } else if (!fused) CK(join(l, DN_SQ_POST2, DN_SQ_HC2_MIX, DN_SQ_HC2_OUT, rmul, lc.shared_ff > 0 ? (const float*)m->y2 : nullptr, rmul, nx_last));
         h_ready = nx_run.alpha != nullptr || !pre;
       } else {
-        const int rc = dense_ff(l, N, m->y);
+        const LinEpi<T> ep = join_epi(DN_SQ_LS2, nx_last);
+        const int rc = dense_ff(l, N, m->y, sjoin ? &ep : nullptr);
         if (rc != DN_OK) return rc;
         PH(DN_SEQ_PH_WRITE_BACK);
-        CK(join(l, DN_SQ_POST2, DN_SQ_HC2_MIX, DN_SQ_HC2_OUT, rmul, nullptr, 0.f, nx_run));
-        h_ready = (nx_run.alpha != nullptr && c.post_norm && S <= 0) || !pre;
+        if (!sjoin) CK(join(l, DN_SQ_POST2, DN_SQ_HC2_MIX, DN_SQ_HC2_OUT, rmul, nullptr, 0.f, nx_run));
+        h_ready = (nx_run.alpha != nullptr && can_fuse_next) || !pre;
       }
+    }
+    // ---- token input: x <- x + rms(W_p (gelu(W_g x) * e)) w, and the next run's norm
+    if (c.side_dim > 0) {
+      PH(DN_SEQ_PH_SIDE);
+      const LinEpi<T> ep{mwp(DN_SQ_SIDE_EMBED) + (size_t)run.layer * c.side_dim, b.tok, c.n_layers * c.side_dim, nullptr, nullptr, 1.f, no_next};
+      CK(linear<T>(m, s, (const T*)m->h, l.w[DN_SQ_SIDE_GATE], nullptr, m->act, N, c.side_dim, W, false, ACT_GELU_TAB, LinMaps{wm(DN_SQ_SIDE_GATE), nullptr, &m->x_h}, 0.f,
+                   nullptr, &ep));
+      CK(linear<T>(m, s, (const T*)m->act, l.w[DN_SQ_SIDE_PROJ], nullptr, m->y, N, W, c.side_dim, true, ACT_NONE, LinMaps{wm(DN_SQ_SIDE_PROJ), nullptr, &m->x_side}));
+      CK(launch(k_rms_join<T>, dim3(N), nthr, nsm, s, m->xs, W, (const float*)m->y, 1.f, (const float*)nullptr, 0.f, no_moe, w(DN_SQ_SIDE_NORM), 0, c.eps, (T*)nullptr, nx_run));
+      h_ready = nx_run.alpha != nullptr;
     }
     PH(DN_SEQ_PH_OTHER);
     if (trace) CK(launch(k_stream_sum, dim3(ew), dim3(256), 0, s, (const float*)m->xs, N, W, S1, trace + (size_t)ri * N * W));
@@ -1554,6 +1649,7 @@ extern "C" int dn_seq_step(dn_seq_model* m, int E, const int32_t* slots, const i
   if (m->cfg.loop_times > 0 && !mhas(DN_SQ_LOOP_IN)) return fail(DN_ENOENT, "the loop's input matrix is not bound");
   if (m->cfg.norm_kind == DN_NORM_LAYER && !mhas(DN_SQ_FINAL_NORM_B)) return fail(DN_ENOENT, "the final norm's bias is not bound");
   if (m->cfg.max_positions > 0 && !mhas(DN_SQ_POS)) return fail(DN_ENOENT, "the position table is not bound");
+  if (m->cfg.side_dim > 0 && !mhas(DN_SQ_SIDE_EMBED)) return fail(DN_ENOENT, "the layers' token table is not bound");
   if (m->cfg.bigram_buckets > 0 && !mhas(DN_SQ_BIGRAM)) return fail(DN_ENOENT, "the bigram table is not bound");
   for (int i = 0; i < m->cfg.n_layers; i++) {
     const SeqLayer& l = m->L[i];
@@ -1572,7 +1668,11 @@ extern "C" int dn_seq_step(dn_seq_model* m, int E, const int32_t* slots, const i
     if (dyt) ok = ok && has(DN_SQ_NORM1_B) && has(DN_SQ_NORM1_ALPHA) && (l.c.ff == 0 || (has(DN_SQ_NORM2_B) && has(DN_SQ_NORM2_ALPHA)));
     if (m->cfg.post_norm) ok = ok && has(DN_SQ_POST1) && (l.c.ff == 0 || has(DN_SQ_POST2));
     if (m->cfg.post_norm && dyt) ok = ok && has(DN_SQ_POST1_B) && has(DN_SQ_POST1_ALPHA) && (l.c.ff == 0 || (has(DN_SQ_POST2_B) && has(DN_SQ_POST2_ALPHA)));
-    if (mx == DN_MIX_LATENT) ok = ok && has(DN_SQ_DKV) && has(DN_SQ_DKV_NORM) && has(DN_SQ_UK) && has(DN_SQ_UV) && (!l.c.out_gate || has(DN_SQ_HEAD_GATE)) &&
+    if (m->cfg.layer_scale) ok = ok && has(DN_SQ_LS1) && (l.c.ff == 0 || has(DN_SQ_LS2));
+    if (m->cfg.side_dim > 0) ok = ok && has(DN_SQ_SIDE_GATE) && has(DN_SQ_SIDE_PROJ) && has(DN_SQ_SIDE_NORM);
+    if (n_maps(l.c) == 2) ok = ok && has(DN_SQ_LQ1) && has(DN_SQ_LK1) && has(DN_SQ_LQ2) && has(DN_SQ_LK2);
+    if (mx == DN_MIX_LATENT && l.c.sink) ok = ok && has(DN_SQ_SINK);
+    if (mx == DN_MIX_LATENT) ok = ok && (l.c.kv_from >= 0 || (has(DN_SQ_DKV) && has(DN_SQ_DKV_NORM))) && has(DN_SQ_UK) && has(DN_SQ_UV) && (!l.c.out_gate || has(DN_SQ_HEAD_GATE)) &&
                                   (l.c.q_rank == 0 || (has(DN_SQ_DQ) && has(DN_SQ_DQ_NORM)));
     else if (l.Ck) ok = ok && has(DN_SQ_K) && (l.c.v_is_k || has(DN_SQ_V));
     if (m->cfg.norm_kind == DN_NORM_LAYER) ok = ok && has(DN_SQ_NORM1_B) && (l.c.ff == 0 || m->cfg.parallel_ff || has(DN_SQ_NORM2_B));
@@ -1637,6 +1737,18 @@ extern "C" int dn_seq_step(dn_seq_model* m, int E, const int32_t* slots, const i
   for (int e = 0; e < E; e++) { max_len = counts[e] > max_len ? counts[e] : max_len; row_tiles += (counts[e] + AT_ROWS - 1) / AT_ROWS; }
   Batch b{d, d + N, d + 2 * N, d + 3 * N, d + 5 * N, d + 5 * N + E + 1, d + 5 * N + 2 * E + 1, m->bt_d, N, E, m->max_pages, max_len, row_tiles, d + 4 * N};
   const int32_t* want_dev = d + 5 * N + 3 * E + 1;
+  if (m->lam_stale) {      // lambda of the differential-attention layers, once after their vectors have been bound
+    for (auto& l : m->L)
+      if (n_maps(l.c) == 2) {
+        if (m->cfg.dtype == DN_SEQ_F32)
+          CK(launch(k_diff_lambda<float>, dim3(1), dim3(32), 0, s, (const float*)l.w[DN_SQ_LQ1], (const float*)l.w[DN_SQ_LK1], (const float*)l.w[DN_SQ_LQ2],
+                    (const float*)l.w[DN_SQ_LK2], l.c.dim, l.c.diff, l.lam));
+        else
+          CK(launch(k_diff_lambda<bf16>, dim3(1), dim3(32), 0, s, (const bf16*)l.w[DN_SQ_LQ1], (const bf16*)l.w[DN_SQ_LK1], (const bf16*)l.w[DN_SQ_LQ2],
+                    (const bf16*)l.w[DN_SQ_LK2], l.c.dim, l.c.diff, l.lam));
+      }
+    m->lam_stale = false;
+  }
   auto run = [&](float* lg) {
     if (m->cfg.dtype == DN_SEQ_F32) return step_T<float>(m, b, n_want, want_dev, lg, trace, s);
     return step_T<bf16>(m, b, n_want, want_dev, lg, trace, s);

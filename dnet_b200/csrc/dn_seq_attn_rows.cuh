@@ -6,7 +6,9 @@
 // works from there: a lane scores one key, then owns ceil(dv / 32) adjacent output dims.  The warps' partials join in warp
 // order; rows with several splits leave theirs in scratch, and the last block of a row to finish (an atomic count, nobody
 // waits) joins them in split order.  A row's split, tiles and order of sums depend on its own position only.
-// Head sizes up to 128 whose rows start on 16-byte boundaries; no pooled blocks (k_attn does those).
+// MAPS = 2 (differential attention): heads 2 i and 2 i + 1 are one pair of maps, key heads 2 g and 2 g + 1 lie side by side in a key
+// row and share value head g; a block stages both maps' keys as one row, and the join subtracts the maps and norms the head.
+// Head sizes up to 128 (a pair's keys count as one row) whose rows start on 16-byte boundaries; no pooled blocks (k_attn does those).
 #pragma once
 #include "dn_seq_kernels.cuh"
 
@@ -20,30 +22,34 @@ __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
 // bytes of one tile (32 keys and values): key rows are padded by 16 bytes, so that the lanes' 16-byte reads of one column
 // of 32 rows fall into different banks
 __host__ __device__ __forceinline__ size_t ar_tile_bytes(int dk, int dv, int esz, bool vk) { return (size_t)32 * (dk * esz + 16) + (vk ? 0 : (size_t)32 * dv * esz); }
-__host__ __device__ __forceinline__ size_t ar_smem_bytes(int dk, int dv, int esz, bool vk, int stages, int HB) {
-  const size_t part = (size_t)AR_WARPS * HB * (2 + (dv + 31) / 32 * 32) * 4;
+// (dk: the whole staged key row; HB heads of `maps` rows of partials each)
+__host__ __device__ __forceinline__ size_t ar_smem_bytes(int dk, int dv, int esz, bool vk, int stages, int HB, int maps) {
+  const size_t part = (size_t)AR_WARPS * HB * maps * (2 + (dv + 31) / 32 * 32) * 4;
   return (size_t)HB * dk * 4 + ((part + 15) & ~(size_t)15) + (size_t)AR_WARPS * stages * ar_tile_bytes(dk, dv, esz, vk);
 }
 __device__ __forceinline__ int ar_splits(int keys, int zmax) { return min(zmax, max(1, (keys + AR_KEYS - 1) / AR_KEYS)); }
 
 // (a head's result does not depend on HB: small grids take fewer heads a block)
-template <class T, bool SIG, int HB>
+template <class T, bool SIG, int HB, int MAPS>
 __global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* __restrict__ q, const T* __restrict__ kpool, const T* __restrict__ vpool, int H,
                                                              int G, int dk, int dv, int chunk, float scale, int stages, AttnExtra ex, T* __restrict__ out,
                                                              float* __restrict__ part_g, unsigned int* __restrict__ count) {
   extern __shared__ __align__(16) unsigned char smb[];
   __shared__ uint32_t rows_s[AR_WARPS][32];
   __shared__ bool last_s;
-  constexpr int V = Vec16<T>::n, ESZ = (int)sizeof(T);
+  constexpr int V = Vec16<T>::n, ESZ = (int)sizeof(T), NV = HB * MAPS;      // NV: score rows of the block (head i, map m: i MAPS + m)
+  H /= MAPS; G /= MAPS;                                      // heads and key heads with all their maps
+  const int dk1 = dk;
+  dk *= MAPS;                                                // numbers of a staged key row, and of a head's query
   const int VPL = (dv + 31) / 32, dvp = VPL * 32, PL = 2 + dvp;
   float* qs = reinterpret_cast<float*>(smb);                       // [HB][dk]
-  float* part = qs + HB * dk;                                // [AR_WARPS][HB][2 + dvp]
-  unsigned char* tiles = smb + (size_t)HB * dk * 4 + (((size_t)AR_WARPS * HB * PL * 4 + 15) & ~(size_t)15);
+  float* part = qs + HB * dk;                                // [AR_WARPS][NV][2 + dvp]
+  unsigned char* tiles = smb + (size_t)HB * dk * 4 + (((size_t)AR_WARPS * NV * PL * 4 + 15) & ~(size_t)15);
   const int n = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int R = H / G, per = (R + HB - 1) / HB;        // heads of a key head; blocks they take
   const int g = blockIdx.y / per, h0 = g * R + (blockIdx.y % per) * HB, nh = min(HB, (g + 1) * R - h0);
   const int slot = b.slot[n], p = b.pos[n];
-  const int lo = attn_lo(p, chunk, ex.window), nkeys = p - lo + 1;
+  const int lo = attn_lo(p, chunk, ex.window), kept = attn_kept(lo, ex), nkeys = kept + p - lo + 1;
   const int zmax = gridDim.z, nz = ar_splits(nkeys, zmax), z = blockIdx.z;
   if (z >= nz) return;
   const bool vk = vpool == kpool;
@@ -62,7 +68,7 @@ __global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* _
     unsigned char* vt = vk ? kt : kt + (size_t)32 * ldk;
     const int cnt = min(32, nkeys - j0);
     if (lane < cnt) {
-      const int j = lo + j0 + lane;
+      const int v = j0 + lane, j = v < kept ? v : lo + v - kept;      // kept first tokens, then the tokens lo .. p
       rows_s[warp][lane] = (uint32_t)bt[j / PAGE] * PAGE + (uint32_t)(j % PAGE);
     }
     __syncwarp();
@@ -91,9 +97,9 @@ __global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* _
     soff[i] = SIG ? ldf((const T*)ex.off + h) : 0.f;
   }
   __syncthreads();
-  float m[HB], l[HB], acc[HB][4];
+  float m[NV], l[NV], acc[NV][4];
 #pragma unroll
-  for (int i = 0; i < HB; i++) {
+  for (int i = 0; i < NV; i++) {
     m[i] = -INFINITY; l[i] = 0.f;
 #pragma unroll
     for (int x = 0; x < 4; x++) acc[i][x] = 0.f;
@@ -108,33 +114,38 @@ __global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* _
     const unsigned char* kt = mine + (size_t)s * tile_b;
     const unsigned char* vt = vk ? kt : kt + (size_t)32 * ldk;
     const int cnt = min(32, nkeys - j0), j = j0 + lane;
-    float sc[HB];
+    float sc[NV];
 #pragma unroll
-    for (int i = 0; i < HB; i++) sc[i] = 0.f;
+    for (int i = 0; i < NV; i++) sc[i] = 0.f;
     if (lane < cnt) {
       const T* kr = reinterpret_cast<const T*>(kt + (size_t)lane * ldk);
+#pragma unroll
+      for (int mp = 0; mp < MAPS; mp++) {
 #pragma unroll 4
-      for (int d = 0; d < dk; d += V) {
-        float kv[V];
-        ldv(kr + d, kv);
+        for (int d1 = 0; d1 < dk1; d1 += V) {
+          const int d = mp * dk1 + d1;
+          float kv[V];
+          ldv(kr + d, kv);
 #pragma unroll
-        for (int i = 0; i < HB; i++) {
+          for (int i = 0; i < HB; i++) {
+            float& s1 = sc[i * MAPS + mp];
 #pragma unroll
-          for (int x = 0; x < V; x += 4) {
-            const float4 q4 = *reinterpret_cast<const float4*>(qs + i * dk + d + x);
-            sc[i] = fmaf(q4.x, kv[x], sc[i]); sc[i] = fmaf(q4.y, kv[x + 1], sc[i]);
-            sc[i] = fmaf(q4.z, kv[x + 2], sc[i]); sc[i] = fmaf(q4.w, kv[x + 3], sc[i]);
+            for (int x = 0; x < V; x += 4) {
+              const float4 q4 = *reinterpret_cast<const float4*>(qs + i * dk + d + x);
+              s1 = fmaf(q4.x, kv[x], s1); s1 = fmaf(q4.y, kv[x + 1], s1);
+              s1 = fmaf(q4.z, kv[x + 2], s1); s1 = fmaf(q4.w, kv[x + 3], s1);
+            }
           }
         }
       }
     }
-    float pw[HB];
+    float pw[NV];
 #pragma unroll
-    for (int i = 0; i < HB; i++) {
+    for (int i = 0; i < NV; i++) {
       float a = sc[i] * scale;
       if (ex.softcap > 0.f) a = ex.softcap * tanhf(a / ex.softcap);
-      if (ex.r1) a -= r1[i] * log1pf(r2[i] * (float)max(0, nkeys - 1 - j));
-      if (SIG) { pw[i] = lane < cnt ? sigmoid_f(a + soff[i]) : 0.f; continue; }
+      if (ex.r1) a -= r1[i / MAPS] * log1pf(r2[i / MAPS] * (float)max(0, j < kept ? p - j : nkeys - 1 - j));
+      if (SIG) { pw[i] = lane < cnt ? sigmoid_f(a + soff[i / MAPS]) : 0.f; continue; }
       a = lane < cnt ? a : -INFINITY;
       const float mn = fmaxf(m[i], warp_max(a)), corr = expf(m[i] - mn);
       pw[i] = lane < cnt ? expf(a - mn) : 0.f;
@@ -153,7 +164,7 @@ __global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* _
         for (int x = 0; x < 4; x++) if (x < vcnt) v[x] = ldf(vr + x);
       }
 #pragma unroll
-      for (int i = 0; i < HB; i++) {
+      for (int i = 0; i < NV; i++) {
         const float pt = __shfl_sync(0xffffffffu, pw[i], t);
 #pragma unroll
         for (int x = 0; x < 4; x++) acc[i][x] = fmaf(pt, v[x], acc[i][x]);
@@ -164,17 +175,29 @@ __global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* _
     else if (more) stage(0, j0 + step);
   }
 #pragma unroll
-  for (int i = 0; i < HB; i++) {
-    float* pr = part + ((size_t)warp * HB + i) * PL;
+  for (int i = 0; i < NV; i++) {
+    float* pr = part + ((size_t)warp * NV + i) * PL;
     if (lane == 0) { pr[0] = m[i]; pr[1] = l[i]; }
 #pragma unroll
     for (int x = 0; x < 4; x++) if (x < VPL) pr[2 + lane * VPL + x] = acc[i][x];
   }
   __syncthreads();
   const bool split = nz > 1;
-  // head i's output from `cnt` partials at stride `st` floats (shared memory, or scratch written by other blocks: read past L1)
+  // row i's (head's) output from `cnt` partials at stride `st` floats (shared memory, or scratch written by other blocks: read past L1)
+  float* os = reinterpret_cast<float*>(tiles);      // MAPS = 2: [NV][dv], the maps' outputs (the tiles have been read out)
   auto finish = [&](int i, int d, const float* pr, size_t st, int cnt, bool global) {
     auto rd = [&](const float* a) { return global ? __ldcg(a) : *a; };
+    if (MAPS == 2) {
+      float M = -INFINITY, L = 0.f, a = 0.f;
+      for (int w = 0; w < cnt; w++) M = fmaxf(M, rd(pr + w * st));
+      for (int w = 0; w < cnt; w++) {
+        const float f = expf(rd(pr + w * st) - M);
+        L += rd(pr + w * st + 1) * f;
+        a += rd(pr + w * st + 2 + d) * f;
+      }
+      os[i * dv + d] = a / L;
+      return;
+    }
     const int h = h0 + i;
     const float og = ex.gate ? sigmoid_f(ex.gate[(size_t)n * H + h]) : 1.f;
     float a = 0.f;
@@ -194,19 +217,33 @@ __global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* _
     }
     stf(out + ((size_t)n * H + h) * dv + d, a / L * og);
   };
+  // MAPS = 2: a warp a head subtracts the maps, norms and stores
+  auto diff_out = [&]() {
+    __syncthreads();
+    const float lm = *ex.lam;
+    for (int i = warp; i < nh; i += AR_WARPS) {
+      const float *a1 = os + 2 * i * dv, *a2 = a1 + dv;
+      float ss = 0.f;
+      for (int d = lane; d < dv; d += 32) { const float o = a1[d] - lm * a2[d]; ss += o * o; }
+      const float f = ex.post / sqrtf(warp_sum(ss) / (float)dv + ex.eps);
+      for (int d = lane; d < dv; d += 32) stf(out + ((size_t)n * H + h0 + i) * dv + d, (a1[d] - lm * a2[d]) * f);
+    }
+  };
+  const int nrows = nh * MAPS;
   if (!split) {
-    for (int e = threadIdx.x; e < nh * dv; e += blockDim.x) finish(e / dv, e % dv, part + (size_t)(e / dv) * PL, (size_t)HB * PL, AR_WARPS, false);
+    for (int e = threadIdx.x; e < nrows * dv; e += blockDim.x) finish(e / dv, e % dv, part + (size_t)(e / dv) * PL, (size_t)NV * PL, AR_WARPS, false);
+    if (MAPS == 2) diff_out();
     return;
   }
-  for (int e = threadIdx.x; e < nh * dv; e += blockDim.x) {
+  for (int e = threadIdx.x; e < nrows * dv; e += blockDim.x) {
     const int i = e / dv, d = e % dv;
     const float* pr = part + (size_t)i * PL;
-    float* pg = part_g + (((size_t)n * H + h0 + i) * zmax + z) * PL;
+    float* pg = part_g + (((size_t)n * H * MAPS + h0 * MAPS + i) * zmax + z) * PL;
     float M = -INFINITY, L = 0.f, a = 0.f;
     if (!SIG)
-      for (int w = 0; w < AR_WARPS; w++) M = fmaxf(M, pr[(size_t)w * HB * PL]);
+      for (int w = 0; w < AR_WARPS; w++) M = fmaxf(M, pr[(size_t)w * NV * PL]);
     for (int w = 0; w < AR_WARPS; w++) {
-      const float* pq = pr + (size_t)w * HB * PL;
+      const float* pq = pr + (size_t)w * NV * PL;
       const float f = SIG ? 1.f : expf(pq[0] - M);
       if (!SIG) L += pq[1] * f;
       a += pq[2 + d] * f;
@@ -221,8 +258,9 @@ __global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* _
   if (!last_s) return;
   __threadfence();
   if (threadIdx.x == 0) count[(size_t)n * gridDim.y + blockIdx.y] = 0;      // ready for the next launch
-  for (int e = threadIdx.x; e < nh * dv; e += blockDim.x)
-    finish(e / dv, e % dv, part_g + ((size_t)n * H + h0 + e / dv) * zmax * PL, (size_t)PL, nz, true);
+  for (int e = threadIdx.x; e < nrows * dv; e += blockDim.x)
+    finish(e / dv, e % dv, part_g + ((size_t)n * H * MAPS + h0 * MAPS + e / dv) * zmax * PL, (size_t)PL, nz, true);
+  if (MAPS == 2) diff_out();
 }
 
 }  // namespace dnseq

@@ -29,6 +29,8 @@
 //   * a learned position row added to the embedding; RMS norm with one number for all coordinates; mixer and feed-forward
 //     side by side on one normed input, joined with a factor and the next layer's norm in one pass
 //   * attention without a softmax: sigmoid weights with an offset per head; scores that fall with the logarithm of the distance
+//   * a sliding window behind which the sequence's first tokens stay visible; differential attention (two maps a head over one
+//     value, subtracted and RMS-normed); outputs scaled per channel as they join the residual; a gated row of a per-layer token table
 // T is the storage type of weights and activations (bf16 or float); sums, norms, scores, positions, gates and
 // states are fp32 in both.
 #pragma once
@@ -111,8 +113,9 @@ __device__ __forceinline__ float clamped_glu_f(float g, float u, float limit) {
   return g * sigmoid_f(1.702f * g) * (u + 1.f);
 }
 // activation of a product's epilogue: 0 none; 1 gelu_tanh(a) * b; 2 tanh(a); 3 clamped GLU of (a, b) with `lim`;
-// 4 silu(a) * b; 5 relu(a)^2.  A bias, where a product has one, is added to a before the activation.
-constexpr int ACT_NONE = 0, ACT_GEGLU = 1, ACT_TANH = 2, ACT_CGLU = 3, ACT_SWIGLU = 4, ACT_RELU2 = 5;
+// 4 silu(a) * b; 5 relu(a)^2; 6 gelu_tanh(a) * b with b out of a table (LinEpi).  A bias, where a product has one, is added to a
+// before the activation.  7: the result joins the residual (LinEpi)
+constexpr int ACT_NONE = 0, ACT_GEGLU = 1, ACT_TANH = 2, ACT_CGLU = 3, ACT_SWIGLU = 4, ACT_RELU2 = 5, ACT_GELU_TAB = 6, ACT_JOIN = 7;
 __host__ __device__ __forceinline__ bool act_two(int act) { return act == ACT_GEGLU || act == ACT_CGLU || act == ACT_SWIGLU; }
 __device__ __forceinline__ float act_apply(int act, float a, float b, float lim) {
   if (act == ACT_GEGLU) return gelu_tanh_f(a) * b;
@@ -120,6 +123,7 @@ __device__ __forceinline__ float act_apply(int act, float a, float b, float lim)
   if (act == ACT_CGLU) return clamped_glu_f(a, b, lim);
   if (act == ACT_SWIGLU) return silu_f(a) * b;
   if (act == ACT_RELU2) { const float r = fmaxf(a, 0.f); return r * r; }
+  if (act == ACT_GELU_TAB) return gelu_tanh_f(a) * b;
   return a;
 }
 // sum += v with the rounding error of the addition carried in c (compensated summation)
@@ -358,7 +362,7 @@ __global__ void k_write_back(float* __restrict__ xs, int N, int W, int S, const 
 //   x <- x + dyt(a y + b y2)        (y2 optional: two branches of a mixer, or routed + shared experts)
 // and, since the norm before the next sublayer is elementwise too, its output in the same pass: h <- dyt'(x)
 template <class T>
-struct NextNorm { const T *w, *b, *alpha; T* h; };      // alpha == null: none
+struct NextNorm { const T *w, *b, *alpha; T* h; };      // alpha == null: none (where the kernel says so: T(x) into h)
 template <class T>
 __global__ void k_dyt_add(float* __restrict__ x, size_t NW, int W, const float* __restrict__ y, float a, const float* __restrict__ y2, float b,
                           const T* __restrict__ nw, const T* __restrict__ nb, const T* __restrict__ nalpha, NextNorm<T> nx) {
@@ -370,6 +374,25 @@ __global__ void k_dyt_add(float* __restrict__ x, size_t NW, int W, const float* 
   const float xn = x[i] + dyt_f(v, ldf(nalpha), nw, nb, c);
   x[i] = xn;
   if (nx.alpha) stf(nx.h + i, dyt_f(xn, ldf(nx.alpha), nx.w, nx.b, c));
+}
+// what follows a residual value xn of column c: the next sublayer's dynamic tanh, or (no alpha) xn itself in the products' format
+template <class T>
+__device__ __forceinline__ void next_norm_at(const NextNorm<T>& nx, size_t at, int c, float xn) {
+  stf(nx.h + at, nx.alpha ? dyt_f(xn, ldf(nx.alpha), nx.w, nx.b, c) : xn);
+}
+// a sublayer's output joins the plain residual, scaled per channel, and the next elementwise norm with it:
+//   x <- x + ls (a y + b y2);   h <- dyt'(x) or T(x)        (ls, y2, h optional)
+template <class T>
+__global__ void k_scale_join(float* __restrict__ x, size_t NW, int W, const float* __restrict__ y, float a, const float* __restrict__ y2, float b,
+                             const T* __restrict__ ls, NextNorm<T> nx) {
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= NW) return;
+  const int c = (int)(i % W);
+  float v = a * y[i];
+  if (y2) v += b * y2[i];
+  const float xn = x[i] + (ls ? v * ldf(ls + c) : v);
+  x[i] = xn;
+  if (nx.h) next_norm_at(nx, i, c, xn);
 }
 // the same, in place, for models with residual streams (the write-back follows): y <- dyt(a y + b y2)
 template <class T>
@@ -431,7 +454,7 @@ struct MoeSrc {
 };
 template <class T>
 __global__ void k_rms_join(float* __restrict__ x, int W, const float* __restrict__ y, float a, const float* __restrict__ y2, float b, MoeSrc<T> ms,
-                           const T* __restrict__ nw, int one_plus, float eps, T* __restrict__ hout) {
+                           const T* __restrict__ nw, int one_plus, float eps, T* __restrict__ hout, NextNorm<T> nx) {
   extern __shared__ __align__(16) float sm[];
   float* v = sm;            // [W]
   float* red = sm + W;      // [33]
@@ -457,6 +480,7 @@ __global__ void k_rms_join(float* __restrict__ x, int W, const float* __restrict
     const float xn = x[base + c] + v[c] * rinv * (ldf(nw + c) + (one_plus ? 1.f : 0.f));
     x[base + c] = xn;
     if (hout) stf(hout + base + c, xn);
+    if (nx.h) next_norm_at(nx, base + c, c, xn);
   }
 }
 
@@ -570,10 +594,24 @@ __global__ void k_stream_sum(const float* __restrict__ xs, int N, int W, int S1,
 // error of a long reduction stays that of one block -- the fp32 mode's products then match the few-row kernel's
 // (lane partials + tree) to the last bits, whatever the step's size.
 // OUT32: write fp32 (residual-side outputs), else T.  act: ACT_* (the two-operand ones read W2 as well).
+// Epilogues of a product with operands of their own:
+//   ACT_GELU_TAB   y[n, o] = gelu_tanh(a) tab[row[n] ld + o]
+//   ACT_JOIN       x[n, o] += a mul ls[o];  h[n, o] = dyt'(x[n, o]) or T(x[n, o])      (no y; ls, h optional)
+template <class T>
+struct LinEpi {
+  const T* tab; const int32_t* row; int ld;
+  float* x; const T* ls; float mul; NextNorm<T> nx;
+};
+template <class T>
+__device__ __forceinline__ void lin_join(const LinEpi<T>& ep, size_t at, int o, float a) {
+  const float xn = ep.x[at] + a * (ep.ls ? ep.mul * ldf(ep.ls + o) : ep.mul);
+  ep.x[at] = xn;
+  if (ep.nx.h) next_norm_at(ep.nx, at, o, xn);
+}
 template <class T, bool OUT32>
 __global__ void __launch_bounds__(256) k_linear(const T* __restrict__ X, const T* __restrict__ Wt, const T* __restrict__ W2,
                                                 void* __restrict__ Y, int N, int O, int K, int act, float alim,
-                                                const T* __restrict__ bias) {
+                                                const T* __restrict__ bias, LinEpi<T> ep) {
   const bool two = act_two(act);
   constexpr int BM = 64, BN = 64, BK = 16;
   __shared__ float Xs[BK][BM + 4], Ws[BK][BN + 4], Vs[BK][BN + 4];
@@ -634,7 +672,8 @@ __global__ void __launch_bounds__(256) k_linear(const T* __restrict__ X, const T
     for (int j = 0; j < 4; j++) {
       const int o = o0 + tx * 4 + j;
       if (o >= O) continue;
-      const float v = act_apply(act, acc[i][j] + (bias ? ldf(bias + o) : 0.f), acc2[i][j], alim);
+      if (act == ACT_JOIN) { lin_join(ep, (size_t)n * O + o, o, acc[i][j] + (bias ? ldf(bias + o) : 0.f)); continue; }
+      const float v = act_apply(act, acc[i][j] + (bias ? ldf(bias + o) : 0.f), act == ACT_GELU_TAB ? ldf(ep.tab + (size_t)ep.row[n] * ep.ld + o) : acc2[i][j], alim);
       if (OUT32) ((float*)Y)[(size_t)n * O + o] = v;
       else stf((T*)Y + (size_t)n * O + o, v);
     }
@@ -751,7 +790,8 @@ __device__ __forceinline__ void dot_rows(const T* __restrict__ X, const T* __res
 // output feature o (and o + 1 where `pair`) of one product
 template <class T, int NT, bool TWO>
 __device__ __forceinline__ void linear_rows_at(const T* __restrict__ X, const T* __restrict__ Wt, const T* __restrict__ W2, void* __restrict__ Y, bool out32,
-                                               int N, int O, int K, int actc, int o, float alim, const T* __restrict__ bias) {
+                                               int N, int O, int K, int actc, int o, float alim, const T* __restrict__ bias,
+                                               const LinEpi<T>* ep = nullptr) {
   constexpr int V = Vec16<T>::n;
   const bool two = act_two(actc);
   const bool pair = TWO && !two && o + 1 < O;
@@ -759,6 +799,35 @@ __device__ __forceinline__ void linear_rows_at(const T* __restrict__ X, const T*
   const T* wb = two ? W2 + (size_t)o * K : pair ? wa + K : wa;
   const bool vec = (K % V == 0) && ((((uintptr_t)Wt | (uintptr_t)X | (uintptr_t)(two ? W2 : Wt)) & 15) == 0);
   float a[NT], b[NT];
+  if (ep) {
+    // an epilogue with operands of its own: lane i takes row i (lane NT + i the second output feature's), and what the epilogue reads
+    // is asked for before the product
+    const int lane = threadIdx.x & 31, i = lane % NT, oo = o + lane / NT;
+    const bool live = i < N && (lane < NT || (pair && lane < 2 * NT));
+    const size_t at = (size_t)i * O + oo;
+    float x = 0.f, s = 1.f, nw = 0.f, nb = 0.f, na = 0.f;
+    if (live && actc == ACT_JOIN) {
+      x = ep->x[at];
+      s = ep->ls ? ep->mul * ldf(ep->ls + oo) : ep->mul;
+      if (ep->nx.alpha) { na = ldf(ep->nx.alpha); nw = ldf(ep->nx.w + oo); nb = ldf(ep->nx.b + oo); }
+    } else if (live && actc == ACT_GELU_TAB) x = ldf(ep->tab + (size_t)ep->row[i] * ep->ld + oo);
+    dot_rows<T, NT, TWO>(X, wa, wb, N, K, vec, a, b);
+    if (!live) return;
+    float v = 0.f;
+#pragma unroll
+    for (int k = 0; k < NT; k++) if (k == i) v = lane < NT ? a[k] : b[k];
+    if (bias) v += ldf(bias + oo);
+    if (actc == ACT_JOIN) {
+      const float xn = x + v * s;
+      ep->x[at] = xn;
+      if (ep->nx.h) stf(ep->nx.h + at, ep->nx.alpha ? tanhf(na * xn) * nw + nb : xn);
+      return;
+    }
+    v = act_apply(actc, v, x, alim);
+    if (out32) ((float*)Y)[at] = v;
+    else stf((T*)Y + at, v);
+    return;
+  }
   dot_rows<T, NT, TWO>(X, wa, wb, N, K, vec, a, b);
   if ((threadIdx.x & 31) != 0) return;
   auto put = [&](int i, int oo, float v) {
@@ -776,10 +845,10 @@ __device__ __forceinline__ void linear_rows_at(const T* __restrict__ X, const T*
 template <class T, int NT, bool TWO>
 __global__ void __launch_bounds__(256) k_linear_rows(const T* __restrict__ X, const T* __restrict__ Wt, const T* __restrict__ W2,
                                                      void* __restrict__ Y, int out32, int N, int O, int K, int act, int per, float alim,
-                                                     const T* __restrict__ bias) {
+                                                     const T* __restrict__ bias, LinEpi<T> ep) {
   const int o = (blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5)) * per;
   if (o >= O) return;
-  linear_rows_at<T, NT, TWO>(X, Wt, W2, Y, out32 != 0, N, O, K, act, o, alim, bias);
+  linear_rows_at<T, NT, TWO>(X, Wt, W2, Y, out32 != 0, N, O, K, act, o, alim, bias, act == ACT_JOIN || act == ACT_GELU_TAB ? &ep : nullptr);
 }
 // several products of the same few rows in one launch (the projections of a mixer in a decode step): blocks are
 // dealt to the products in order, 8 output features each (16 where a warp takes two)
@@ -928,6 +997,7 @@ struct AttnPrep {
   float mscale;                      // cos and sin are multiplied by this
   float qt_coef; int qt_every;       // q times 1 + qt_coef ln(floor((p + 1) / qt_every) + 1) (qt_every 0: no)
   int carry;                         // 1: every entry brings one token, and the kernel carries its inputs itself (no k_conv_carry)
+  int gv;                            // value heads (fewer than G where several keys share a value)
 };
 
 // attention mixer, between the projections and the scores: conv -> RMS norm (over the whole q / k projection or per
@@ -940,7 +1010,7 @@ __global__ void k_attn_prep(AttnPrep a, Batch b, const T* __restrict__ Uq, const
                             T* __restrict__ kpool, T* __restrict__ vpool) {
   extern __shared__ float sm[];
   // a layer that borrows its keys and values projects and carries q only
-  const int Cq = a.H * a.dk, Ck = a.own_kv ? a.G * a.dk : 0, Cv = (a.own_kv && a.own_v) ? a.G * a.dv : 0, ldst = Cq + Ck + Cv;
+  const int Cq = a.H * a.dk, Ck = a.own_kv ? a.G * a.dk : 0, Cv = (a.own_kv && a.own_v) ? a.gv * a.dv : 0, ldst = Cq + Ck + Cv;
   const int HG = a.H + (a.own_kv ? a.G : 0);
   float* qs = sm;
   float* ks = sm + Cq;
@@ -1188,6 +1258,13 @@ struct AttnExtra {
   const void* r1;  // [H] with r2: r1_h ln(1 + r2_h (p - j)) is taken off the score (after scale and cap) of the key at j (null: no)
   const void* r2;
   const void* off; // [H] sigmoid weights: added to the score inside the sigmoid
+  int keep;        // with window: positions 0 .. keep - 1 stay visible behind it
+  // maps = 2, differential attention: the H heads and G key heads are pairs of maps, heads 2 i and 2 i + 1 of one pair share a value
+  // head and give (1 - diff) rms(a_2i - lambda a_2i+1), H / 2 heads of the output
+  int maps;
+  const float* lam;    // lambda, one number in device memory
+  float post, eps;     // 1 - diff; of the norm
+  float* out32;        // k_attn, k_attn_merge: fp32 output [N, H, dv] of every map (null: T)
 };
 // keys a query at p sees: the pooled blocks first (virtual indices 0 .. nb - 1), then the tokens lo .. p
 __device__ __forceinline__ int attn_pooled(int p, int chunk, const AttnExtra& ex) { return ex.pool > 0 ? pooled_seen(p, chunk, ex.pool) : 0; }
@@ -1196,6 +1273,15 @@ __device__ __forceinline__ int attn_lo(int p, int chunk, int window) {
   if (chunk <= 0) return 0;
   return window ? max(0, p - chunk + 1) : (p / chunk) * chunk;
 }
+// a query whose window starts at lo sees the positions 0 .. attn_kept(lo) - 1 before it; how many keys a query at p sees in all
+__device__ __forceinline__ int attn_kept(int lo, const AttnExtra& ex) { return min(ex.keep, lo); }
+__device__ __forceinline__ int attn_keys(int p, int chunk, const AttnExtra& ex) {
+  const int lo = attn_lo(p, chunk, ex.window);
+  return attn_pooled(p, chunk, ex) + attn_kept(lo, ex) + p - lo + 1;
+}
+// key and value head of head h
+__device__ __forceinline__ int attn_key_head(int h, int H, int G, int maps) { const int R = H / G; return maps == 2 ? 2 * ((h >> 1) / R) + (h & 1) : h / R; }
+__device__ __forceinline__ int attn_value_head(int h, int H, int G, int maps) { const int R = H / G; return maps == 2 ? (h >> 1) / R : h / R; }
 // Long rows of a small step are split over gridDim.z blocks: a row that sees n keys uses ceil(n / AT_SPLIT_KEYS) of
 // them (at most gridDim.z), split z taking every nz-th group of AT_WARPS tiles; each writes its partial (maximum,
 // sum, output) to scratch and k_attn_merge joins them in the order of z.  The split depends on the row's own
@@ -1237,12 +1323,12 @@ __global__ void __launch_bounds__(AT_WARPS * 32) k_attn(Batch b, const T* __rest
   float* qs = sm;                                   // [dk rounded up to 4]
   float* part = sm + ((dk + 3) & ~3);               // [AT_WARPS][2 + dvp]
   const int n = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int g = h / (H / G), slot = b.slot[n], p = b.pos[n];
-  const int lo = attn_lo(p, chunk, ex.window);
-  const int nb = attn_pooled(p, chunk, ex), nkeys = nb + p - lo + 1;
+  const int g = attn_key_head(h, H, G, ex.maps), gv = attn_value_head(h, H, G, ex.maps), slot = b.slot[n], p = b.pos[n];
+  const int lo = attn_lo(p, chunk, ex.window), kept = attn_kept(lo, ex);
+  const int nb = attn_pooled(p, chunk, ex), nkeys = attn_keys(p, chunk, ex);
   const int nz = attn_splits(nkeys, (int)gridDim.z), z = blockIdx.z;
   if (z >= nz) return;
-  const int Ck = G * dk, Cv = ex.v_ld > 0 ? ex.v_ld : G * dv;
+  const int Ck = G * dk, Cv = ex.v_ld > 0 ? ex.v_ld : (ex.maps == 2 ? G / 2 : G) * dv;
   for (int d = threadIdx.x; d < dk; d += blockDim.x) qs[d] = ldf(q + ((size_t)n * H + h) * dk + d);
   __syncthreads();
   const int32_t* bt = b.bt + (size_t)slot * b.max_pages;
@@ -1256,11 +1342,11 @@ __global__ void __launch_bounds__(AT_WARPS * 32) k_attn(Batch b, const T* __rest
   float m = -INFINITY, l = 0.f, acc[MAXV];
 #pragma unroll
   for (int i = 0; i < MAXV; i++) acc[i] = 0.f;
-  // virtual key v (pooled blocks first, then the tokens lo .. p) lives in row row_of(v) of the token pools, or, with bit 31
+  // virtual key v (pooled blocks or kept first tokens, then the tokens lo .. p) lives in row row_of(v) of the token pools, or, with bit 31
   // set, of the pooled pools; a lane finds its own key's row once and the value loop takes the rows from the lanes
   auto row_of = [&](int v) -> uint32_t {
     if (v < nb) return 0x80000000u | (uint32_t)pooled_row(bt, v, ex.pool);
-    const int j = lo + v - nb;
+    const int u = v - nb, j = u < kept ? u : lo + u - kept;
     return (uint32_t)bt[j / PAGE] * PAGE + (uint32_t)(j % PAGE);
   };
   const T* kpl = (const T*)ex.pk;
@@ -1275,7 +1361,7 @@ __global__ void __launch_bounds__(AT_WARPS * 32) k_attn(Batch b, const T* __rest
       myrow = row_of(j);
       const T* kr = ((myrow >> 31) ? kpl : kpool) + (size_t)(myrow & 0x7fffffffu) * Ck + g * dk;
       {   // the key's value row is needed after the scores: ask for its lines now, so that the value loop finds them in L2
-        const char* vrow = reinterpret_cast<const char*>(((myrow >> 31) ? vpl : vpool) + (size_t)(myrow & 0x7fffffffu) * Cv + g * dv);
+        const char* vrow = reinterpret_cast<const char*>(((myrow >> 31) ? vpl : vpool) + (size_t)(myrow & 0x7fffffffu) * Cv + gv * dv);
         if (vrow != reinterpret_cast<const char*>(kr))
           for (int o = 0; o < dv * (int)sizeof(T); o += 128) asm volatile("prefetch.global.L2 [%0];" ::"l"(vrow + o));
       }
@@ -1293,7 +1379,7 @@ __global__ void __launch_bounds__(AT_WARPS * 32) k_attn(Batch b, const T* __rest
       }
       s = d0 * scale;
       if (ex.softcap > 0.f) s = ex.softcap * tanhf(s / ex.softcap);
-      if (ex.r1) s -= r1 * log1pf(r2 * (float)(nkeys - 1 - j));      // (no pooled blocks here: the last key is the query's own)
+      if (ex.r1) s -= r1 * log1pf(r2 * (float)(j < kept ? p - j : nkeys - 1 - j));      // (no pooled blocks here: the last key is the query's own)
     }
     float mn = 0.f, pj;
     if (SIG) pj = j < nkeys ? sigmoid_f(s + soff) : 0.f;
@@ -1317,7 +1403,7 @@ __global__ void __launch_bounds__(AT_WARPS * 32) k_attn(Batch b, const T* __rest
           const int t = min(t0 + u, cnt - 1);
           const uint32_t rw = __shfl_sync(0xffffffffu, myrow, t);
           pt[u] = t0 + u < cnt ? __shfl_sync(0xffffffffu, pj, t) : 0.f;
-          const T* vr = ((rw >> 31) ? vpl : vpool) + (size_t)(rw & 0x7fffffffu) * Cv + g * dv + lane * VPL;
+          const T* vr = ((rw >> 31) ? vpl : vpool) + (size_t)(rw & 0x7fffffffu) * Cv + gv * dv + lane * VPL;
           if (vbytes == 16) raw[u] = *reinterpret_cast<const uint4*>(vr);
           else if (vbytes == 8) { const uint2 r2 = *reinterpret_cast<const uint2*>(vr); raw[u] = make_uint4(r2.x, r2.y, 0u, 0u); }
           else raw[u] = make_uint4(*reinterpret_cast<const uint32_t*>(vr), 0u, 0u, 0u);
@@ -1337,7 +1423,7 @@ __global__ void __launch_bounds__(AT_WARPS * 32) k_attn(Batch b, const T* __rest
     for (int t = 0; t < cnt; t++) {
       const float pt = __shfl_sync(0xffffffffu, pj, t);
       const uint32_t rw = __shfl_sync(0xffffffffu, myrow, t);
-      const T* vr = ((rw >> 31) ? vpl : vpool) + (size_t)(rw & 0x7fffffffu) * Cv + g * dv + lane * VPL;
+      const T* vr = ((rw >> 31) ? vpl : vpool) + (size_t)(rw & 0x7fffffffu) * Cv + gv * dv + lane * VPL;
 #pragma unroll
       for (int i0 = 0; i0 < MAXV; i0 += 8) {
         if (i0 < vcnt) {
@@ -1381,7 +1467,8 @@ __global__ void __launch_bounds__(AT_WARPS * 32) k_attn(Batch b, const T* __rest
     if (split) {
       pg[2 + d] = a;
       if (d == 0) { pg[0] = M; pg[1] = L; }
-    } else stf(out + ((size_t)n * H + h) * dv + d, a / L * og);
+    } else if (ex.out32) ex.out32[((size_t)n * H + h) * dv + d] = a / L * og;
+    else stf(out + ((size_t)n * H + h) * dv + d, a / L * og);
   }
 }
 // joins the partials of the rows that k_attn split (rows with one split are complete already); grid (N, H, 1)
@@ -1389,8 +1476,7 @@ template <class T>
 __global__ void k_attn_merge(Batch b, int H, int dv, int chunk, int zmax, AttnExtra ex, const float* __restrict__ part_g, T* __restrict__ out) {
   const int n = blockIdx.x, h = blockIdx.y, p = b.pos[n];
   const bool sig = ex.off != nullptr;      // sigmoid weights: the partials add
-  const int lo = attn_lo(p, chunk, ex.window);
-  const int nz = attn_splits(attn_pooled(p, chunk, ex) + p - lo + 1, zmax);
+  const int nz = attn_splits(attn_keys(p, chunk, ex), zmax);
   if (nz <= 1) return;
   const int dvp = (dv + 31) / 32 * 32;
   const float* pg = part_g + ((size_t)n * H + h) * zmax * (2 + dvp);
@@ -1413,8 +1499,30 @@ __global__ void k_attn_merge(Batch b, int H, int dv, int chunk, int zmax, AttnEx
       L += pz[1] * f;
       a += pz[2 + d] * f;
     }
-    stf(out + ((size_t)n * H + h) * dv + d, a / L * og);
+    if (ex.out32) ex.out32[((size_t)n * H + h) * dv + d] = a / L * og;
+    else stf(out + ((size_t)n * H + h) * dv + d, a / L * og);
   }
+}
+// differential attention behind k_attn: the two maps' outputs [N, 2 H, dv] subtracted, RMS-normed over a head's dv numbers without a
+// weight and scaled; one warp per (token, head), a lane's partial sum over its own columns in ascending order
+template <class T>
+__global__ void k_diff_join(const float* __restrict__ a, int rows, int dv, const float* __restrict__ lam, float post, float eps, T* __restrict__ out) {
+  const int r = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (r >= rows) return;
+  const float *a1 = a + (size_t)r * 2 * dv, *a2 = a1 + dv, lm = *lam;
+  float ss = 0.f;
+  for (int d = lane; d < dv; d += 32) { const float o = a1[d] - lm * a2[d]; ss += o * o; }
+  const float f = post / sqrtf(warp_sum(ss) / (float)dv + eps);
+  for (int d = lane; d < dv; d += 32) stf(out + (size_t)r * dv + d, (a1[d] - lm * a2[d]) * f);
+}
+// lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff (one warp)
+template <class T>
+__global__ void k_diff_lambda(const T* __restrict__ lq1, const T* __restrict__ lk1, const T* __restrict__ lq2, const T* __restrict__ lk2, int dk, float diff,
+                              float* __restrict__ lam) {
+  float a = 0.f, c = 0.f;
+  for (int d = threadIdx.x; d < dk; d += 32) { a += ldf(lq1 + d) * ldf(lk1 + d); c += ldf(lq2 + d) * ldf(lk2 + d); }
+  a = warp_sum(a); c = warp_sum(c);
+  if (threadIdx.x == 0) *lam = expf(a) - expf(c) + diff;
 }
 
 // ---------------------------------------------------------------------------------------------------------------
@@ -1428,6 +1536,8 @@ __global__ void k_attn_merge(Batch b, int H, int dv, int chunk, int zmax, AttnEx
 // DKP / DVP: head sizes rounded up to the template's; the padding is zero in shared memory.
 // A distance bias depends on p - key alone, of which a tile has 127 values: they are tabled in shared memory once a tile.
 // SIG: sigmoid weights (see k_attn): no running maximum, no sum; the head's offset rides in the table.
+// MAPS = 2 (differential attention): a block owns one pair of maps, warps 0-3 the first and 4-7 the second; the value tile is staged
+// once for both, and at the end the second map's rows pass through shared memory to the first's, which subtract, norm and store.
 __device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], const void* p) {
   const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
@@ -1471,18 +1581,20 @@ __device__ __forceinline__ void load_tile64_rows(bf16* __restrict__ dst, const b
 }
 
 constexpr int AT_ROWS = 64;      // query rows of a block, and keys of a tile (= PAGE)
-template <int DKP, int DVP, bool SIG = false>
-__global__ void __launch_bounds__(128) k_attn_tiles(Batch b, const bf16* __restrict__ q, const bf16* __restrict__ kpool,
+template <int DKP, int DVP, bool SIG = false, int MAPS = 1>
+__global__ void __launch_bounds__(128 * MAPS) k_attn_tiles(Batch b, const bf16* __restrict__ q, const bf16* __restrict__ kpool,
                                                     const bf16* __restrict__ vpool, int H, int G, int dk, int dv, int chunk, float scale,
                                                     AttnExtra ex, bf16* __restrict__ out) {
   static_assert(PAGE == AT_ROWS, "a key tile is one page");
   constexpr int LQ = DKP + 8, LV = DVP + 8;
   extern __shared__ __align__(16) unsigned char smraw[];
-  bf16* Qs = reinterpret_cast<bf16*>(smraw);
-  bf16* Ks = Qs + AT_ROWS * LQ;
+  const int lane = threadIdx.x & 31, map = MAPS == 2 ? threadIdx.x >> 7 : 0, warp = (threadIdx.x >> 5) & 3;
+  bf16* Q0 = reinterpret_cast<bf16*>(smraw);
+  bf16* K0 = Q0 + MAPS * AT_ROWS * LQ;
+  bf16 *Qs = Q0 + map * AT_ROWS * LQ, *Ks = K0 + map * AT_ROWS * LQ;      // this warp's map's
   // values that are the keys (one pool, equal tile shapes): the key tile is the value tile, nothing is staged twice
   const bool vk = DKP == DVP && dk == dv && vpool == kpool && ex.pv == ex.pk;
-  bf16* Vs = vk ? Ks : Ks + AT_ROWS * LQ;
+  bf16* Vs = vk ? K0 : K0 + MAPS * AT_ROWS * LQ;
   // which entry and which of its 64-row tiles
   int e = 0, t = blockIdx.x;
   for (; e < b.E; e++) {
@@ -1491,13 +1603,14 @@ __global__ void __launch_bounds__(128) k_attn_tiles(Batch b, const bf16* __restr
     t -= nt;
   }
   if (e >= b.E) return;
-  const int h = blockIdx.y, g = h / (H / G);
+  // the block's (first map's) head and key head; its value head
+  const int h = MAPS * blockIdx.y, g = attn_key_head(h, H, G, MAPS), gv = attn_value_head(h, H, G, MAPS);
   const int s0 = b.ent_start[e] + t * AT_ROWS, s1 = b.ent_start[e + 1];
   const int rows = min(AT_ROWS, s1 - s0);
   const int p_first = b.ent_pos0[e] + t * AT_ROWS, p_last = p_first + rows - 1;
-  const int Ck = G * dk, Cv = ex.v_ld > 0 ? ex.v_ld : G * dv;
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  load_tile64<LQ>(Qs, q + ((size_t)s0 * H + h) * dk, (size_t)H * dk, dk, rows);
+  const int Ck = G * dk, Cv = ex.v_ld > 0 ? ex.v_ld : G / MAPS * dv;
+#pragma unroll
+  for (int i = 0; i < MAPS; i++) load_tile64<LQ>(Q0 + i * AT_ROWS * LQ, q + ((size_t)s0 * H + h + i) * dk, (size_t)H * dk, dk, rows);
   __syncthreads();
   // this thread's two rows of its warp's 16
   const int r0 = warp * 16 + (lane >> 2), r1w = r0 + 8;
@@ -1519,10 +1632,12 @@ __global__ void __launch_bounds__(128) k_attn_tiles(Batch b, const bf16* __restr
   // pooled blocks behind the window come first, 64 to a tile, in ascending block order; then the pages of the tokens
   const int nb0 = p0 >= 0 ? attn_pooled(p0, chunk, ex) : 0, nb1 = p1 >= 0 ? attn_pooled(p1, chunk, ex) : 0;
   const int nb_last = attn_pooled(p_last, chunk, ex), pool_tiles = (nb_last + AT_ROWS - 1) / AT_ROWS;
-  const int tok0 = (lo_tile / PAGE) * PAGE, tok_tiles = p_last >= tok0 ? (p_last - tok0) / PAGE + 1 : 0;
-  for (int it = 0; it < pool_tiles + tok_tiles; it++) {
+  // (kept first tokens: their pages come before the window's)
+  const int kept_tiles = (attn_kept(lo_tile, ex) + PAGE - 1) / PAGE;
+  const int tok0 = max(lo_tile / PAGE, kept_tiles) * PAGE, tok_tiles = p_last >= tok0 ? (p_last - tok0) / PAGE + 1 : 0;
+  for (int it = 0; it < pool_tiles + kept_tiles + tok_tiles; it++) {
     const bool pooled = it < pool_tiles;
-    const int j0 = pooled ? it * AT_ROWS : tok0 + (it - pool_tiles) * PAGE;
+    const int j0 = pooled || it < pool_tiles + kept_tiles ? (pooled ? it : it - pool_tiles) * AT_ROWS : tok0 + (it - pool_tiles - kept_tiles) * PAGE;
     __syncthreads();
     if (pooled) {
       load_tile64_rows<LQ>(Ks, (const bf16*)ex.pk + (size_t)g * dk, (size_t)Ck, dk, min(AT_ROWS, nb_last - j0), bt, j0, ex.pool);
@@ -1530,9 +1645,10 @@ __global__ void __launch_bounds__(128) k_attn_tiles(Batch b, const bf16* __restr
     } else {
       const size_t prow = (size_t)bt[j0 / PAGE] * PAGE;
       const int kvalid = min(PAGE, p_last - j0 + 1);      // rows of the page beyond the last query's position are not read
-      load_tile64<LQ>(Ks, kpool + prow * Ck + (size_t)g * dk, (size_t)Ck, dk, kvalid);
-      if (!vk) load_tile64<LV>(Vs, vpool + prow * Cv + (size_t)g * dv, (size_t)Cv, dv, kvalid);
-      if (SIG || ex.r1) tb[threadIdx.x] = r1 * log1pf(r2 * (float)max(0, p_first - j0 - (AT_ROWS - 1) + (int)threadIdx.x)) - soff;
+#pragma unroll
+      for (int i = 0; i < MAPS; i++) load_tile64<LQ>(K0 + i * AT_ROWS * LQ, kpool + prow * Ck + (size_t)(g + i) * dk, (size_t)Ck, dk, kvalid);
+      if (!vk) load_tile64<LV>(Vs, vpool + prow * Cv + (size_t)gv * dv, (size_t)Cv, dv, kvalid);
+      if ((SIG || ex.r1) && threadIdx.x < 2 * AT_ROWS) tb[threadIdx.x] = r1 * log1pf(r2 * (float)max(0, p_first - j0 - (AT_ROWS - 1) + (int)threadIdx.x)) - soff;
     }
     __syncthreads();
     if (!warp_live) continue;
@@ -1562,7 +1678,7 @@ __global__ void __launch_bounds__(128) k_attn_tiles(Batch b, const bf16* __restr
           float a = sc[j][i] * scale;
           if (ex.softcap > 0.f) a = ex.softcap * tanhf(a / ex.softcap);
           const float z = (tb[(i < 2 ? r0 : r1w) + (AT_ROWS - 1) - kc] - a) * LOG2E_;
-          const bool see = i < 2 ? (key <= p0 && key >= lo0) : (key <= p1 && key >= lo1);
+          const bool see = i < 2 ? (key <= p0 && (key >= lo0 || key < ex.keep)) : (key <= p1 && (key >= lo1 || key < ex.keep));
           sc[j][i] = see ? __fdividef(1.f, 1.f + exp2f(z)) : 0.f;
         }
       }
@@ -1577,8 +1693,8 @@ __global__ void __launch_bounds__(128) k_attn_tiles(Batch b, const bf16* __restr
         float a0 = sc[j][i] * scale, a1 = sc[j][2 + i] * scale;
         if (ex.softcap > 0.f) { a0 = ex.softcap * tanhf(a0 / ex.softcap); a1 = ex.softcap * tanhf(a1 / ex.softcap); }
         if (biased) { a0 -= tb[r0 + (AT_ROWS - 1) - (key - j0)]; a1 -= tb[r1w + (AT_ROWS - 1) - (key - j0)]; }
-        sc[j][i] = (pooled ? key < nb0 : (key <= p0 && key >= lo0)) ? a0 : -INFINITY;
-        sc[j][2 + i] = (pooled ? key < nb1 : (key <= p1 && key >= lo1)) ? a1 : -INFINITY;
+        sc[j][i] = (pooled ? key < nb0 : (key <= p0 && (key >= lo0 || key < ex.keep))) ? a0 : -INFINITY;
+        sc[j][2 + i] = (pooled ? key < nb1 : (key <= p1 && (key >= lo1 || key < ex.keep))) ? a1 : -INFINITY;
         mx0 = fmaxf(mx0, sc[j][i]);
         mx1 = fmaxf(mx1, sc[j][2 + i]);
       }
@@ -1627,6 +1743,46 @@ __global__ void __launch_bounds__(128) k_attn_tiles(Batch b, const bf16* __restr
         mma_bf16(o[2 * jj + 1], pl, vf[2], vf[3]);
       }
     }
+  }
+  if (MAPS == 2) {
+    const float i0 = p0 >= 0 ? 1.f / l0 : 0.f, i1 = p1 >= 0 ? 1.f / l1 : 0.f;
+    float* ex2 = reinterpret_cast<float*>(smraw);      // [64][DVP + 4]: the second map's rows (the tiles have been read out)
+    constexpr int LE = DVP + 4;
+    __syncthreads();
+    if (map == 1 && warp_live) {
+#pragma unroll
+      for (int j = 0; j < DVP / 8; j++) {
+        const int d = j * 8 + (lane & 3) * 2;
+        *reinterpret_cast<float2*>(ex2 + r0 * LE + d) = make_float2(o[j][0] * i0, o[j][1] * i0);
+        *reinterpret_cast<float2*>(ex2 + r1w * LE + d) = make_float2(o[j][2] * i1, o[j][3] * i1);
+      }
+    }
+    __syncthreads();
+    if (map == 1 || !warp_live) return;
+    const float lm = *ex.lam;
+    float s0q = 0.f, s1q = 0.f;
+#pragma unroll
+    for (int j = 0; j < DVP / 8; j++) {      // (columns from dv on are zero in both maps)
+      const int d = j * 8 + (lane & 3) * 2;
+      const float2 a = *reinterpret_cast<const float2*>(ex2 + r0 * LE + d), c = *reinterpret_cast<const float2*>(ex2 + r1w * LE + d);
+      o[j][0] = o[j][0] * i0 - lm * a.x; o[j][1] = o[j][1] * i0 - lm * a.y;
+      o[j][2] = o[j][2] * i1 - lm * c.x; o[j][3] = o[j][3] * i1 - lm * c.y;
+      s0q += o[j][0] * o[j][0]; s0q += o[j][1] * o[j][1];
+      s1q += o[j][2] * o[j][2]; s1q += o[j][3] * o[j][3];
+    }
+    s0q += __shfl_xor_sync(0xffffffffu, s0q, 1); s0q += __shfl_xor_sync(0xffffffffu, s0q, 2);
+    s1q += __shfl_xor_sync(0xffffffffu, s1q, 1); s1q += __shfl_xor_sync(0xffffffffu, s1q, 2);
+    const float f0 = ex.post / sqrtf(s0q / (float)dv + ex.eps), f1 = ex.post / sqrtf(s1q / (float)dv + ex.eps);
+    const int Ho = H / 2, ho = h / 2;
+#pragma unroll
+    for (int j = 0; j < DVP / 8; j++) {
+      const int d = j * 8 + (lane & 3) * 2;
+      if (d < dv) {
+        if (p0 >= 0) *reinterpret_cast<uint32_t*>(out + ((size_t)(s0 + r0) * Ho + ho) * dv + d) = pack_bf16(o[j][0] * f0, o[j][1] * f0);
+        if (p1 >= 0) *reinterpret_cast<uint32_t*>(out + ((size_t)(s0 + r1w) * Ho + ho) * dv + d) = pack_bf16(o[j][2] * f1, o[j][3] * f1);
+      }
+    }
+    return;
   }
   if (!warp_live) return;
   if (ex.sink) {       // one more term of the denominator, with no value: fold it in as a last key

@@ -14,6 +14,7 @@
 // serves prompt portions and decode steps, whatever the cut.
 //
 // Rotary pairs are (2i, 2i + 1) or (i, i + rot / 2), on the first `rot` numbers of the rotated part; angles are fp32.
+// A sink adds exp(sink_h) to the softmax denominator of head h; a layer may read the rows that an earlier layer cached.
 #pragma once
 #include "dn_seq_kernels.cuh"
 #include "dn_seq_moe.cuh"      // warp_dot
@@ -25,6 +26,8 @@ struct LatentPrep {
   int rot, half;           // rotated numbers of the rotated part; 1: pairs half apart
   float eps;
   const float* inv_freq;   // [rot / 2]
+  float mscale;            // cos and sin are multiplied by this
+  int own;                 // 0: the cached rows are another layer's (only the queries are prepared)
 };
 
 // pair i of a rotated part: its two indices
@@ -42,16 +45,19 @@ __global__ void k_latent_prep(LatentPrep a, Batch b, const T* __restrict__ Uq, c
   const int n = blockIdx.x, slot = b.slot[n], p = b.pos[n];
   const int Ck = a.R + a.dr, dq = a.dn + a.dr;
   const T* kv = Ukv + (size_t)n * Ck;
-  float ss = 0.f;
-  for (int c = threadIdx.x; c < a.R; c += blockDim.x) { const float v = ldf(kv + c); ss += v * v; }
-  ss = block_sum(ss, red);
-  const float rinv = 1.f / sqrtf(ss / (float)a.R + a.eps);
-  const int page = b.bt[(size_t)slot * b.max_pages + p / PAGE], prow = p % PAGE;
-  T* row = kpool + ((size_t)page * PAGE + prow) * Ck;
-  for (int c = threadIdx.x; c < a.R; c += blockDim.x) stf(row + c, ldf(kv + c) * rinv * ldf(cnorm + c));
+  T* row = nullptr;
+  if (a.own) {
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < a.R; c += blockDim.x) { const float v = ldf(kv + c); ss += v * v; }
+    ss = block_sum(ss, red);
+    const float rinv = 1.f / sqrtf(ss / (float)a.R + a.eps);
+    const int page = b.bt[(size_t)slot * b.max_pages + p / PAGE], prow = p % PAGE;
+    row = kpool + ((size_t)page * PAGE + prow) * Ck;
+    for (int c = threadIdx.x; c < a.R; c += blockDim.x) stf(row + c, ldf(kv + c) * rinv * ldf(cnorm + c));
+  }
   // rotated parts: source 0 is the shared key part, sources 1..H the heads' query parts
   const int np = a.rot / 2, per = np + (a.dr - a.rot);      // work items a source: the pairs, then the numbers that do not turn
-  for (int e = threadIdx.x; e < (a.H + 1) * per; e += blockDim.x) {
+  for (int e = threadIdx.x + (a.own ? 0 : per); e < (a.H + 1) * per; e += blockDim.x) {
     const int src = e / per, i = e % per;
     const T* in = src == 0 ? kv + a.R : Uq + (size_t)n * a.H * dq + (size_t)(src - 1) * dq + a.dn;
     T* out = src == 0 ? row + a.R : qout + ((size_t)n * a.H + (src - 1)) * Ck + a.R;
@@ -61,6 +67,7 @@ __global__ void k_latent_prep(LatentPrep a, Batch b, const T* __restrict__ Uq, c
       const float u = ldf(in + ia), v = ldf(in + ib);
       float sn, cs;
       sincosf((float)p * a.inv_freq[i], &sn, &cs);
+      sn *= a.mscale; cs *= a.mscale;
       stf(out + ia, u * cs - v * sn);
       stf(out + ib, v * cs + u * sn);
     } else {
@@ -391,7 +398,14 @@ __global__ void __launch_bounds__(256, 1) k_latent_tiles(Batch b, const bf16* __
     }
     return;
   }
-  float i0 = p0 >= 0 ? 1.f / l0 : 0.f, i1 = p1 >= 0 ? 1.f / l1 : 0.f;
+  float f0 = 1.f, f1 = 1.f;
+  if (ex.sink) {       // one more term of the denominator, with no value
+    const float snk = __bfloat162float(((const bf16*)ex.sink)[h]);
+    const float n0 = fmaxf(m0, snk), n1 = fmaxf(m1, snk);
+    f0 = expf(m0 - n0); f1 = expf(m1 - n1);
+    l0 = l0 * f0 + expf(snk - n0); l1 = l1 * f1 + expf(snk - n1);
+  }
+  float i0 = p0 >= 0 ? f0 / l0 : 0.f, i1 = p1 >= 0 ? f1 / l1 : 0.f;
   if (ex.gate) {
     if (p0 >= 0) i0 *= sigmoid_f(ex.gate[(size_t)(s0 + r0) * H + h]);
     if (p1 >= 0) i1 *= sigmoid_f(ex.gate[(size_t)(s0 + r1) * H + h]);
@@ -419,9 +433,10 @@ __global__ void k_latent_merge(Batch b, int H, int R, int chunk, int zmax, AttnE
   if (threadIdx.x < 32) {
     const int z = threadIdx.x;
     const float m = z < nz ? pg[(size_t)z * part_ld] : -INFINITY;
-    const float M = warp_max(m);
+    const float snk = ex.sink ? __bfloat162float(((const bf16*)ex.sink)[h]) : -INFINITY;
+    const float M = fmaxf(warp_max(m), snk);
     const float fz = z < nz ? expf(m - M) : 0.f;
-    const float L = warp_sum(z < nz ? pg[(size_t)z * part_ld + 1] * fz : 0.f);
+    const float L = warp_sum(z < nz ? pg[(size_t)z * part_ld + 1] * fz : 0.f) + (ex.sink ? expf(snk - M) : 0.f);
     f[z] = fz;
     if (z == 0) scale = (ex.gate ? sigmoid_f(ex.gate[(size_t)n * H + h]) : 1.f) / L;
   }

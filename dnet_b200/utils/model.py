@@ -29,7 +29,7 @@ NORM_RE = re.compile(r"^model\.norm\.(.+)$")
 # checkpoints of the layer-list families (core/models/seqmix.py): l<i>.<tensor>, embed, final.norm, head
 SEQ_LAYER_RE = re.compile(r"^l(\d+)\.(.+)$")
 SEQ_API = {"embed": "embed_tokens", "final.norm": "norm", "head": "lm_head"}
-SEQ_EMBED_EXTRA = ("bigram", "pos")      # further tables the embedding reads
+SEQ_EMBED_EXTRA = ("bigram", "pos", "side.embed")      # further tables the embedding reads
 SEQ_MODEL_RE = re.compile(r"^(embed|final|head|loop)\.(.+)$")
 
 

@@ -6,7 +6,8 @@
  * key channel, decayed outer-product recurrences, or attention beside one of those) plus an optional dense, gated or
  * routed feed-forward, tied together by S residual streams; a span of layers may run several times on the same weights;
  * every sublayer's input may pass a short causal convolution first, and the embedding may add a hashed bigram row or a
- * learned position row; a layer's mixer and feed-forward run one after the other or side by side on one normed input.
+ * learned position row; a layer's mixer and feed-forward run one after the other or side by side on one normed input; a
+ * sublayer's output may be scaled per channel, and a layer may end with a gated row of a token table of its own.
  *
  * Same conventions as dnet_b200.h: plain C, opaque handles, 0 or a negative DN_E* code, dn_seq_last_error() for
  * the text, caller-owned streams and buffers, weights BORROWED by pointer.  One handle serves one compute thread.
@@ -59,6 +60,7 @@ extern "C" {
 
 #define DN_FF_GEGLU 0       /* dense feed-forward: gelu_tanh(W_gate h) * (W_up h) */
 #define DN_FF_RELU2 1       /* dense feed-forward: relu(W_up h + b)^2, no gate; up and down may carry biases (unbound: none) */
+#define DN_FF_SWIGLU 2      /* dense feed-forward: silu(W_gate h) * (W_up h) */
 
 #define DN_ROUTER_TOPK 0    /* the `top` largest logits choose; softmax over the chosen logits weighs */
 #define DN_ROUTER_SCORED 1  /* every expert gets a score (DN_SCORE_*); a correction, if bound, is added for the choice only; experts form
@@ -84,7 +86,7 @@ typedef struct dn_seq_layer_cfg {
   int32_t rot_dims;    /* attention: rotated dims per head (0: none) */
   float rot_base;
   float scale;         /* attention: score scale */
-  int32_t kv_from;     /* attention: layer whose pages hold this layer's keys and values (-1: its own) */
+  int32_t kv_from;     /* attention, latent attention: layer whose pages hold this layer's keys and values (-1: its own) */
   int32_t ff;          /* feed-forward width, of one expert for DN_MLP_MOE (0: the layer has no feed-forward) */
   /* attention (also the attention half of DN_MIX_PARALLEL) */
   int32_t qk_norm;     /* DN_QKNORM_*: RMS norm of q and k with learned weights, before rotation */
@@ -132,6 +134,15 @@ typedef struct dn_seq_layer_cfg {
   int32_t attn_weight; /* DN_ATTN_*: what turns a score into a key's weight */
   int32_t dist_bias;   /* 1: r1_h ln(1 + r2_h (i - j)) is taken off the score of the key at j for the query at i */
   int32_t score_kind;  /* DN_SCORE_*: DN_ROUTER_SCORED */
+  /* rotary frequencies scaled by wavelength l = 2 pi / f: f where l < original / high, f / factor where l > original / low, between
+   * them (1 - s) f / factor + s f with s = (original / l - low) / (high - low).  band_factor 0: no */
+  float band_factor, band_low, band_high, band_original;
+  int32_t keep_first;  /* DN_MASK_WINDOW: the sequence's first keep_first positions stay visible behind the window */
+  /* DN_MIX_ATTENTION.  2: differential attention -- a head has two queries and two keys of `dim` (laid out head by head, map by map)
+   * over one value; with a1, a2 the two softmax outputs and one number a layer
+   * lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff, the head's output is (1 - diff) rms(a1 - lambda a2), no weight.  0, 1: plain */
+  int32_t maps;
+  float diff;
 } dn_seq_layer_cfg;
 
 typedef struct dn_seq_cfg {
@@ -162,6 +173,10 @@ typedef struct dn_seq_cfg {
   int32_t parallel_ff;
   float residual_mult;       /* sublayer outputs are multiplied by this as they join the residual (0: by 1) */
   int32_t max_positions;     /* rows of DN_SQ_POS: row p is added to the embedding of the token at position p (0: none); no sequence grows longer */
+  int32_t layer_scale;       /* 1: a sublayer's output is multiplied by DN_SQ_LS1 / DN_SQ_LS2 [W] as it joins the residual */
+  /* after a layer's last sublayer x <- x + rms(W_p (gelu_tanh(W_g x) * e)) w, with e the columns [i side_dim, (i + 1) side_dim) of the
+   * token's row of DN_SQ_SIDE_EMBED [vocab, n_layers side_dim] for layer i, and a plain RMS norm (0: none) */
+  int32_t side_dim;
 } dn_seq_cfg;
 
 /* tensors of a layer (dn_seq_bind: layer >= 0) and of the model (layer = -1) */
@@ -195,9 +210,12 @@ enum {
   DN_SQ_CANON1, DN_SQ_CANON2, DN_SQ_L_OUT, DN_SQ_R_OUT, DN_SQ_R_A, DN_SQ_R_AB,
   /* dist_bias: r1, r2 [H]; DN_ATTN_SIGMOID: the offset of the scores [H] */
   DN_SQ_DIST1, DN_SQ_DIST2, DN_SQ_ATTN_OFF,
+  /* layer_scale [W] each; maps = 2: lambda's vectors [dim] each; side_dim: gate [side_dim, W], projection [W, side_dim], norm [W] */
+  DN_SQ_LS1, DN_SQ_LS2, DN_SQ_LQ1, DN_SQ_LK1, DN_SQ_LQ2, DN_SQ_LK2, DN_SQ_SIDE_GATE, DN_SQ_SIDE_PROJ, DN_SQ_SIDE_NORM,
   DN_SQ_COUNT,
   DN_SQ_EMBED = 100, DN_SQ_FINAL_NORM, DN_SQ_HEAD, DN_SQ_FINAL_NORM_B, DN_SQ_FINAL_NORM_ALPHA,
-  DN_SQ_EMBED_NORM, DN_SQ_EMBED_NORM_B, DN_SQ_EMBED_NORM_ALPHA, DN_SQ_LOOP_IN, DN_SQ_BIGRAM, DN_SQ_POS
+  DN_SQ_EMBED_NORM, DN_SQ_EMBED_NORM_B, DN_SQ_EMBED_NORM_ALPHA, DN_SQ_LOOP_IN, DN_SQ_BIGRAM, DN_SQ_POS,
+  DN_SQ_SIDE_EMBED
 };
 /* matrices of a routed expert (dn_seq_bind_expert) */
 enum { DN_SQ_E_GATE = 0, DN_SQ_E_UP, DN_SQ_E_DOWN };
@@ -242,6 +260,7 @@ enum {
   DN_SEQ_PH_LATENT_IN,    /* latent attention: the cached row, rotary, queries absorbed into the latent space */
   DN_SEQ_PH_LATENT_OUT,   /* latent attention: the heads' outputs taken out of the latent space */
   DN_SEQ_PH_CANON,        /* the sublayers' input convolutions and their carried rows */
+  DN_SEQ_PH_SIDE,         /* the token input after a layer's sublayers */
   DN_SEQ_PH_COUNT
 };
 int dn_seq_profile(dn_seq_model* m, int on);
