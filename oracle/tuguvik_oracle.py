@@ -1,8 +1,8 @@
 """Float64 oracle of the Tuguvik family: one plain function per mechanism, whole sequences only, no cache.
 
 It shares nothing with the product path (dnet_b200/core/models/seqmix.py, libdnet_b200_seq): keys and values are formed
-per head from the latent of every position, the two maps of a differential attention are two separate softmaxes over an
-explicit list of visible positions per query, and nothing is absorbed, permuted or paged.
+per head from the latent of every position, the two maps of a differential attention are two separate softmaxes over a dense
+[T, T] table whose visible places are listed query by query, and nothing is absorbed, permuted or paged.
 
 Notation: T tokens, W width, H query heads on G key / value heads; dyt(x) = tanh(alpha x) w + b; rms(x) = x / sqrt(mean(x^2) + eps).
 
@@ -111,11 +111,22 @@ def visible(i: int, mask: Optional[dict]) -> List[int]:
     return [j for j in range(i + 1) if size <= 0 or i - j < size or j < keep]
 
 
-def weights_with_sink(s: torch.Tensor, sink: Optional[torch.Tensor]) -> torch.Tensor:
-    """softmax over the scores s [n]; the sink adds exp(sink) to the denominator"""
-    m = s.max() if sink is None else torch.maximum(s.max(), sink)
+def visible_table(T: int, mask: Optional[dict]) -> torch.Tensor:
+    """[T, T] bool, row i true at visible(i)"""
+    out = torch.zeros(T, T, dtype=torch.bool)
+    for i in range(T):
+        out[i, visible(i, mask)] = True
+    return out
+
+
+def weights_with_sink(s: torch.Tensor, vis: torch.Tensor, sink: Optional[torch.Tensor]) -> torch.Tensor:
+    """softmax over the visible scores of every row of s [T, T]; the sink adds exp(sink) to every denominator"""
+    s = s.masked_fill(~vis, -math.inf)
+    m = s.max(-1, keepdim=True).values
+    if sink is not None:
+        m = torch.maximum(m, sink)
     e = torch.exp(s - m)
-    return e / (e.sum() + (torch.exp(sink - m) if sink is not None else 0.0))
+    return e / (e.sum(-1, keepdim=True) + (torch.exp(sink - m) if sink is not None else 0.0))
 
 
 # -- mixers ------------------------------------------------------------------------------------------------------------------
@@ -138,12 +149,11 @@ def latent_attention(w, p: str, mx: dict, h: torch.Tensor, eps: float, rows: Tup
     k_un = (lat @ w[p + "mix.uk"].T).reshape(T, H, dn)
     val = (lat @ w[p + "mix.uv"].T).reshape(T, H, dv)
     gate = torch.sigmoid(h @ w[p + "mix.g"].T)
+    vis = visible_table(T, mx.get("mask"))
     out = torch.zeros(T, H, dv, dtype=F64)
-    for i in range(T):
-        js = torch.tensor(visible(i, mx.get("mask")))
-        for hh in range(H):
-            s = (k_un[js, hh] @ q[i, hh, :dn] + k_rot[js] @ q_rot[i, hh]) * float(mx["scale"])
-            out[i, hh] = weights_with_sink(s, w[p + "mix.sink"][hh]) @ val[js, hh] * gate[i, hh]
+    for hh in range(H):
+        s = (q[:, hh, :dn] @ k_un[:, hh].T + q_rot[:, hh] @ k_rot.T) * float(mx["scale"])
+        out[:, hh] = weights_with_sink(s, vis, w[p + "mix.sink"][hh]) @ val[:, hh] * gate[:, hh, None]
     return out.reshape(T, H * dv) @ w[p + "mix.o"].T
 
 
@@ -159,13 +169,12 @@ def diff_attention(w, p: str, mx: dict, h: torch.Tensor, eps: float) -> torch.Te
     k = turn((h @ w[p + "mix.k"].T).reshape(T, G, 2, dk), freqs, mult, "half")
     v = (h @ w[p + "mix.v"].T).reshape(T, G, dv)
     lam = diff_lambda(w, p, diff)
+    vis = visible_table(T, mx.get("mask"))
     out = torch.zeros(T, H, dv, dtype=F64)
-    for i in range(T):
-        js = torch.tensor(visible(i, mx.get("mask")))
-        for hh in range(H):
-            g = hh // (H // G)
-            a = [weights_with_sink(k[js, g, m] @ q[i, hh, m] * float(mx["scale"]), None) @ v[js, g] for m in range(2)]
-            out[i, hh] = unit_rms(a[0] - lam * a[1], eps) * (1.0 - diff)
+    for hh in range(H):
+        g = hh // (H // G)
+        a = [weights_with_sink(q[:, hh, m] @ k[:, g, m].T * float(mx["scale"]), vis, None) @ v[:, g] for m in range(2)]
+        out[:, hh] = unit_rms(a[0] - lam * a[1], eps) * (1.0 - diff)
     return out.reshape(T, H * dv) @ w[p + "mix.o"].T
 
 
