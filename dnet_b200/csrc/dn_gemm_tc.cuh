@@ -213,46 +213,62 @@ k_gemm_tc(const __grid_constant__ CUtensorMap mapW, const __grid_constant__ CUte
       const int n = nt * TC_BM + ew * 32 + lane;      // output feature owned by this thread
       const uint32_t ab = (NACC == 2) ? (it & 1u) : 0u;
       const uint32_t acc_phase = ((NACC == 2) ? (it >> 1) : it) & 1u;
+      // what a joining epilogue reads is asked for 32 tokens ahead, the first of them before the products are done
+      constexpr bool OPS = EPI == EPI_JOIN || EPI == EPI_GELU_TAB;
+      float jls = 0.f, jw = 0.f, jb = 0.f, ja = 0.f, jx[OPS ? 32 : 1];
+      auto ahead = [&](int c) {
+#pragma unroll
+        for (int j = 0; j < 32; ++j) {
+          const int t = tt * BN + c + j;
+          if (t < p.T) jx[OPS ? j : 0] = EPI == EPI_JOIN ? p.x[(size_t)t * p.ldy + n] : __bfloat162float(p.tab[(size_t)p.row[t] * p.tab_ld + n]);
+        }
+      };
+      if (OPS && n < p.N) {
+        ahead(0);
+        if (EPI == EPI_JOIN) {
+          jls = p.ls ? p.mul * __bfloat162float(p.ls[n]) : p.mul;
+          if (p.nalpha) { ja = 2.885390081777927f * __bfloat162float(*p.nalpha); jw = __bfloat162float(p.nw[n]); jb = __bfloat162float(p.nb[n]); }      // 2 log2(e) alpha
+        }
+      }
       mbar_wait(&tmem_full[ab], acc_phase, p.err);
       tc_fence_after();
       const uint32_t trow = tmem_base + ab * ACC_COLS + ((uint32_t)(ew * 32) << 16);
       float bias = 0.f;
       if ((EPI == EPI_STORE || EPI == EPI_STORE_F32 || EPI == EPI_RELU2) && p.bias != nullptr && n < p.N) bias = __bfloat162float(p.bias[n]);
-      float jls = 0.f, jw = 0.f, jb = 0.f, ja = 0.f;
-      if (EPI == EPI_JOIN && n < p.N) {
-        jls = p.ls ? p.mul * __bfloat162float(p.ls[n]) : p.mul;
-        if (p.nalpha) { ja = __bfloat162float(*p.nalpha); jw = __bfloat162float(p.nw[n]); jb = __bfloat162float(p.nb[n]); }
-      }
       const int t_base = GROUPED ? p.g_tile_r0[tt] : tt * BN;
       const int t_end = GROUPED ? t_base + p.g_tile_rows[tt] : p.T;
+      if constexpr (OPS) {
+#pragma unroll 1
+        for (int c = 0; c < BN; c += 32) {
+          float v[32];
+          tc_ld16(trow + c, *reinterpret_cast<float(*)[16]>(v));
+          tc_ld16(trow + c + 16, *reinterpret_cast<float(*)[16]>(v + 16));
+          if (n >= p.N) continue;
+          float op[32];
+#pragma unroll
+          for (int j = 0; j < 32; ++j) op[j] = jx[j];
+          if (c + 32 < BN) ahead(c + 32);
+#pragma unroll
+          for (int j = 0; j < 32; ++j) {
+            const int t = tt * BN + c + j;
+            if (t >= p.T) continue;
+            if (EPI == EPI_JOIN) {
+              const float xn = op[j] + v[j] * jls;
+              p.x[(size_t)t * p.ldy + n] = xn;
+              // tanh(z) = 1 - 2 / (1 + e^2z): an absolute error of a few 1e-7, far below the rounding of the result
+              if (p.nh) p.nh[(size_t)t * p.ldy + n] = __float2bfloat16_rn(p.nalpha ? fmaf(1.f - __fdividef(2.f, 1.f + exp2f(fminf(ja * xn, 80.f))), jw, jb) : xn);
+            } else {
+              const float g = v[j];
+              p.Y[(size_t)t * p.ldy + p.col0 + n] = __float2bfloat16_rn(0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * op[j]);
+            }
+          }
+        }
+      } else {
 #pragma unroll 1
       for (int c = 0; c < BN; c += 16) {
         float v[16], v2[16];
         tc_ld16(trow + c, v);
         if (NA == 2) tc_ld16(trow + BN + c, v2);
-        if (EPI == EPI_JOIN || EPI == EPI_GELU_TAB) {      // all of the chunk's loads first
-          if (n < p.N) {
-#pragma unroll
-            for (int j = 0; j < 16; ++j) {
-              const int t = t_base + c + j;
-              if (t < t_end) v2[j] = EPI == EPI_JOIN ? p.x[(size_t)t * p.ldy + n] : __bfloat162float(p.tab[(size_t)p.row[t] * p.tab_ld + n]);
-            }
-#pragma unroll
-            for (int j = 0; j < 16; ++j) {
-              const int t = t_base + c + j;
-              if (t >= t_end) continue;
-              if (EPI == EPI_JOIN) {
-                const float xn = v2[j] + v[j] * jls;
-                p.x[(size_t)t * p.ldy + n] = xn;
-                if (p.nh) p.nh[(size_t)t * p.ldy + n] = __float2bfloat16_rn(p.nalpha ? tanhf(ja * xn) * jw + jb : xn);
-              } else {
-                const float g = v[j];
-                p.Y[(size_t)t * p.ldy + p.col0 + n] = __float2bfloat16_rn(0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * v2[j]);
-              }
-            }
-          }
-          continue;
-        }
         if (n < p.N) {
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
@@ -289,6 +305,7 @@ k_gemm_tc(const __grid_constant__ CUtensorMap mapW, const __grid_constant__ CUte
             }
           }
         }
+      }
       }
       tc_fence_before();
       __syncwarp();

@@ -776,6 +776,7 @@ static cudaError_t gemm_tc(const CUtensorMap& w, const CUtensorMap& w2, const XM
 // One product Y[N, O] = X[N, K] W[O, K]^T (act: an ACT_* epilogue, the two-operand ones on X W^T and X W2^T).  bf16 batches of 16 tokens and more run on
 // the tcgen05 GEMM when the operands have TMA descriptors; a few rows (decode) on the weight-streaming row kernel;
 // everything else, and all of fp32, on the CUDA-core tiles.
+constexpr int ROWS_SPLIT = 512;      // output features below which a warp's row leaves most SMs idle
 constexpr int ROWS_PAIR = 2048;      // output features from which a warp of the row kernels takes two (fewer leave too few warps)
 struct LinMaps { const CUtensorMap* w; const CUtensorMap* w2; const XMaps* x; };
 template <class T>
@@ -805,13 +806,20 @@ static cudaError_t linear(dn_seq_model* m, cudaStream_t s, const T* X, const voi
     if (out32) return gemm_tc<dn::EPI_STORE_F32>(*tm.w, *tm.w, *tm.x, p, s);
     return gemm_tc<dn::EPI_STORE>(*tm.w, *tm.w, *tm.x, p, s);
   }
+  if (N <= 8 && O < ROWS_SPLIT && !act_two(act)) {      // few features: the warps of a block split the reduction
+#define LS(NT) launch(k_linear_rows_split<T, NT>, dim3((O + 1) / 2), dim3(256), 0, s, X, (const T*)W, Y, out32 ? 1 : 0, N, O, K, act, alim, (const T*)bias, epi)
+    return N == 1 ? LS(1) : N == 2 ? LS(2) : N <= 4 ? LS(4) : LS(8);
+#undef LS
+  }
   if (N <= 8) {
     const bool two = act_two(act), pair = !two && O >= ROWS_PAIR;
     const int per = pair ? 2 : 1;
     dim3 grid((O + 8 * per - 1) / (8 * per));
-#define LR(NT) (two || pair ? launch(k_linear_rows<T, NT, true>, grid, dim3(256), 0, s, X, (const T*)W, (const T*)W2, Y, out32 ? 1 : 0, N, O, K, act, per, alim, (const T*)bias, epi) \
-                            : launch(k_linear_rows<T, NT, false>, grid, dim3(256), 0, s, X, (const T*)W, (const T*)W2, Y, out32 ? 1 : 0, N, O, K, act, per, alim, (const T*)bias, epi))
+    const bool own = act == ACT_JOIN || act == ACT_GELU_TAB;      // an epilogue with operands of its own
+#define LRK(NT, TW, EPv) launch(k_linear_rows<T, NT, TW, EPv>, grid, dim3(256), 0, s, X, (const T*)W, (const T*)W2, Y, out32 ? 1 : 0, N, O, K, act, per, alim, (const T*)bias, epi)
+#define LR(NT) (two || pair ? (own ? LRK(NT, true, true) : LRK(NT, true, false)) : (own ? LRK(NT, false, true) : LRK(NT, false, false)))
     return N == 1 ? LR(1) : N == 2 ? LR(2) : N <= 4 ? LR(4) : LR(8);
+#undef LRK
 #undef LR
   }
   dim3 grid((O + 63) / 64, (N + 63) / 64);
@@ -886,7 +894,7 @@ static int attn_rows_stages(const dn_seq_layer_cfg& lc, int N) {      // 0: not 
   if (N > AT_SPLIT_ROWS || lc.pool > 0 || lc.dim > 128 || lc.vdim > 128 || (lc.dim * esz) % 16 || (lc.vdim * esz) % 16) return 0;
   const bool one = lc.chunk > 0 && lc.chunk + lc.keep_first <= AT_MAX_SPLITS * AR_KEYS;
   for (int st = one ? 1 : 2; st > 0; st--)
-    if (ar_smem_bytes(lc.dim * n_maps(lc), lc.vdim, esz, lc.v_is_k != 0, st, 4, n_maps(lc)) + 1024 <= g_max_smem) return st;
+    if (ar_smem_bytes(lc.dim * n_maps(lc), lc.vdim, esz, lc.v_is_k != 0, st, 4, n_maps(lc)) + 2048 <= g_max_smem) return st;
   return 0;
 }
 template <class T, bool SIG, int HB, int MAPS>

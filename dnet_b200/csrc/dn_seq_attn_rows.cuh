@@ -37,6 +37,7 @@ __global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* _
   extern __shared__ __align__(16) unsigned char smb[];
   __shared__ uint32_t rows_s[AR_WARPS][32];
   __shared__ bool last_s;
+  __shared__ float fz[HB * MAPS][AT_MAX_SPLITS];
   constexpr int V = Vec16<T>::n, ESZ = (int)sizeof(T), NV = HB * MAPS;      // NV: score rows of the block (head i, map m: i MAPS + m)
   H /= MAPS; G /= MAPS;                                      // heads and key heads with all their maps
   const int dk1 = dk;
@@ -183,17 +184,17 @@ __global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* _
   }
   __syncthreads();
   const bool split = nz > 1;
-  // row i's (head's) output from `cnt` partials at stride `st` floats (shared memory, or scratch written by other blocks: read past L1)
+  // row i's (head's) output from the warps' partials at stride `st` floats
   float* os = reinterpret_cast<float*>(tiles);      // MAPS = 2: [NV][dv], the maps' outputs (the tiles have been read out)
-  auto finish = [&](int i, int d, const float* pr, size_t st, int cnt, bool global) {
-    auto rd = [&](const float* a) { return global ? __ldcg(a) : *a; };
+  auto finish = [&](int i, int d, const float* pr, size_t st) {
+    constexpr int cnt = AR_WARPS;
     if (MAPS == 2) {
       float M = -INFINITY, L = 0.f, a = 0.f;
-      for (int w = 0; w < cnt; w++) M = fmaxf(M, rd(pr + w * st));
+      for (int w = 0; w < cnt; w++) M = fmaxf(M, pr[w * st]);
       for (int w = 0; w < cnt; w++) {
-        const float f = expf(rd(pr + w * st) - M);
-        L += rd(pr + w * st + 1) * f;
-        a += rd(pr + w * st + 2 + d) * f;
+        const float f = expf(pr[w * st] - M);
+        L += pr[w * st + 1] * f;
+        a += pr[w * st + 2 + d] * f;
       }
       os[i * dv + d] = a / L;
       return;
@@ -202,18 +203,18 @@ __global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* _
     const float og = ex.gate ? sigmoid_f(ex.gate[(size_t)n * H + h]) : 1.f;
     float a = 0.f;
     if (SIG) {
-      for (int w = 0; w < cnt; w++) a += rd(pr + w * st + 2 + d);
+      for (int w = 0; w < cnt; w++) a += pr[w * st + 2 + d];
       stf(out + ((size_t)n * H + h) * dv + d, a * og);
       return;
     }
     const float snk = ex.sink ? ldf((const T*)ex.sink + h) : -INFINITY;
     float M = snk;
-    for (int w = 0; w < cnt; w++) M = fmaxf(M, rd(pr + w * st));
+    for (int w = 0; w < cnt; w++) M = fmaxf(M, pr[w * st]);
     float L = ex.sink ? expf(snk - M) : 0.f;
     for (int w = 0; w < cnt; w++) {
-      const float f = expf(rd(pr + w * st) - M);      // a warp without a tile has maximum -inf and weight 0
-      L += rd(pr + w * st + 1) * f;
-      a += rd(pr + w * st + 2 + d) * f;
+      const float f = expf(pr[w * st] - M);      // a warp without a tile has maximum -inf and weight 0
+      L += pr[w * st + 1] * f;
+      a += pr[w * st + 2 + d] * f;
     }
     stf(out + ((size_t)n * H + h) * dv + d, a / L * og);
   };
@@ -231,7 +232,7 @@ __global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* _
   };
   const int nrows = nh * MAPS;
   if (!split) {
-    for (int e = threadIdx.x; e < nrows * dv; e += blockDim.x) finish(e / dv, e % dv, part + (size_t)(e / dv) * PL, (size_t)NV * PL, AR_WARPS, false);
+    for (int e = threadIdx.x; e < nrows * dv; e += blockDim.x) finish(e / dv, e % dv, part + (size_t)(e / dv) * PL, (size_t)NV * PL);
     if (MAPS == 2) diff_out();
     return;
   }
@@ -258,8 +259,34 @@ __global__ void __launch_bounds__(AR_WARPS * 32) k_attn_rows(Batch b, const T* _
   if (!last_s) return;
   __threadfence();
   if (threadIdx.x == 0) count[(size_t)n * gridDim.y + blockIdx.y] = 0;      // ready for the next launch
-  for (int e = threadIdx.x; e < nrows * dv; e += blockDim.x)
-    finish(e / dv, e % dv, part_g + ((size_t)n * H * MAPS + h0 * MAPS + e / dv) * zmax * PL, (size_t)PL, nz, true);
+  // a warp a row turns the splits' maxima and sums into one factor a split (a lane each), then every thread adds its numbers over the
+  // splits, all loads in flight at once
+  const float* rows_g = part_g + ((size_t)n * H + h0) * MAPS * zmax * PL;
+  for (int i = warp; i < nrows; i += AR_WARPS) {
+    const float* pr = rows_g + (size_t)i * zmax * PL;
+    float f = lane < nz ? 1.f : 0.f;
+    if (!SIG) {
+      const float snk = MAPS == 1 && ex.sink ? ldf((const T*)ex.sink + h0 + i) : -INFINITY;
+      const float mz = lane < nz ? __ldcg(pr + (size_t)lane * PL) : -INFINITY, lz = lane < nz ? __ldcg(pr + (size_t)lane * PL + 1) : 0.f;
+      const float M = fmaxf(warp_max(mz), snk);
+      f = lane < nz ? expf(mz - M) : 0.f;
+      f /= warp_sum(lz * f) + (MAPS == 1 && ex.sink ? expf(snk - M) : 0.f);
+    }
+    if (MAPS == 1 && ex.gate) f *= sigmoid_f(ex.gate[(size_t)n * H + h0 + i]);
+    if (lane < AT_MAX_SPLITS) fz[i][lane] = f;
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < nrows * dv; e += blockDim.x) {
+    const int i = e / dv, d = e - i * dv;
+    const float* pr = rows_g + (size_t)i * zmax * PL + 2 + d;
+    float v[AT_MAX_SPLITS], a = 0.f;
+#pragma unroll
+    for (int z1 = 0; z1 < AT_MAX_SPLITS; z1++) v[z1] = z1 < nz ? __ldcg(pr + (size_t)z1 * PL) : 0.f;
+#pragma unroll
+    for (int z1 = 0; z1 < AT_MAX_SPLITS; z1++) a = fmaf(v[z1], fz[i][z1], a);
+    if (MAPS == 2) os[i * dv + d] = a;
+    else stf(out + ((size_t)n * H + h0 + i) * dv + d, a);
+  }
   if (MAPS == 2) diff_out();
 }
 

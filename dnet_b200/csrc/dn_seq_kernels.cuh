@@ -611,7 +611,7 @@ __device__ __forceinline__ void lin_join(const LinEpi<T>& ep, size_t at, int o, 
 template <class T, bool OUT32>
 __global__ void __launch_bounds__(256) k_linear(const T* __restrict__ X, const T* __restrict__ Wt, const T* __restrict__ W2,
                                                 void* __restrict__ Y, int N, int O, int K, int act, float alim,
-                                                const T* __restrict__ bias, LinEpi<T> ep) {
+                                                const T* __restrict__ bias, const __grid_constant__ LinEpi<T> ep) {
   const bool two = act_two(act);
   constexpr int BM = 64, BN = 64, BK = 16;
   __shared__ float Xs[BK][BM + 4], Ws[BK][BN + 4], Vs[BK][BN + 4];
@@ -745,14 +745,14 @@ __device__ __forceinline__ void linear_row(const T* __restrict__ X, const T* __r
 // output feature), or the next output feature (PAIR).  Every output's sum runs in the order of linear_row.
 template <class T, int NT, bool TWO>
 __device__ __forceinline__ void dot_rows(const T* __restrict__ X, const T* __restrict__ wa, const T* __restrict__ wb, int N, int K, bool vec,
-                                         float (&a)[NT], float (&b)[NT]) {
+                                         float (&a)[NT], float (&b)[NT], int ldx = 0) {
   constexpr int V = Vec16<T>::n;
   const int lane = threadIdx.x & 31;
 #pragma unroll
   for (int i = 0; i < NT; i++) a[i] = b[i] = 0.f;
   size_t xo[NT];
 #pragma unroll
-  for (int i = 0; i < NT; i++) xo[i] = (size_t)min(i, N - 1) * K;
+  for (int i = 0; i < NT; i++) xo[i] = (size_t)min(i, N - 1) * (ldx > 0 ? ldx : K);
   if (vec) {
 #pragma unroll (NT <= 2 ? 4 : 2)
     for (int k = lane * V; k < K; k += 32 * V) {
@@ -787,11 +787,35 @@ __device__ __forceinline__ void dot_rows(const T* __restrict__ X, const T* __res
     if (TWO) b[i] = warp_sum(b[i]);
   }
 }
+// what an epilogue with operands of its own (LinEpi) reads for one output, kept as loaded until the product is there
+template <class T>
+struct EpiArgs {
+  float x; T t, w, b, al;
+  __device__ __forceinline__ void load(const LinEpi<T>& ep, int act, int n, int o, int O) {
+    if (act == ACT_JOIN) {
+      x = ep.x[(size_t)n * O + o];
+      if (ep.ls) t = ep.ls[o];
+      if (ep.nx.alpha) { al = *ep.nx.alpha; w = ep.nx.w[o]; b = ep.nx.b[o]; }
+    } else if (act == ACT_GELU_TAB) t = ep.tab[(size_t)ep.row[n] * ep.ld + o];
+  }
+  __device__ __forceinline__ void finish(const LinEpi<T>& ep, int act, float v, int n, int o, int O, void* Y, bool out32, float alim) const {
+    const size_t at = (size_t)n * O + o;
+    if (act == ACT_JOIN) {
+      const float xn = x + v * (ep.ls ? ep.mul * ldf(&t) : ep.mul);
+      ep.x[at] = xn;
+      if (ep.nx.h) stf(ep.nx.h + at, ep.nx.alpha ? tanhf(ldf(&al) * xn) * ldf(&w) + ldf(&b) : xn);
+      return;
+    }
+    v = act_apply(act, v, act == ACT_GELU_TAB ? ldf(&t) : 0.f, alim);
+    if (out32) ((float*)Y)[at] = v;
+    else stf((T*)Y + at, v);
+  }
+};
 // output feature o (and o + 1 where `pair`) of one product
-template <class T, int NT, bool TWO>
+template <class T, int NT, bool TWO, bool EP>
 __device__ __forceinline__ void linear_rows_at(const T* __restrict__ X, const T* __restrict__ Wt, const T* __restrict__ W2, void* __restrict__ Y, bool out32,
                                                int N, int O, int K, int actc, int o, float alim, const T* __restrict__ bias,
-                                               const LinEpi<T>* ep = nullptr) {
+                                               const LinEpi<T>& ep) {
   constexpr int V = Vec16<T>::n;
   const bool two = act_two(actc);
   const bool pair = TWO && !two && o + 1 < O;
@@ -799,33 +823,20 @@ __device__ __forceinline__ void linear_rows_at(const T* __restrict__ X, const T*
   const T* wb = two ? W2 + (size_t)o * K : pair ? wa + K : wa;
   const bool vec = (K % V == 0) && ((((uintptr_t)Wt | (uintptr_t)X | (uintptr_t)(two ? W2 : Wt)) & 15) == 0);
   float a[NT], b[NT];
-  if (ep) {
+  if (EP) {
     // an epilogue with operands of its own: lane i takes row i (lane NT + i the second output feature's), and what the epilogue reads
     // is asked for before the product
     const int lane = threadIdx.x & 31, i = lane % NT, oo = o + lane / NT;
     const bool live = i < N && (lane < NT || (pair && lane < 2 * NT));
-    const size_t at = (size_t)i * O + oo;
-    float x = 0.f, s = 1.f, nw = 0.f, nb = 0.f, na = 0.f;
-    if (live && actc == ACT_JOIN) {
-      x = ep->x[at];
-      s = ep->ls ? ep->mul * ldf(ep->ls + oo) : ep->mul;
-      if (ep->nx.alpha) { na = ldf(ep->nx.alpha); nw = ldf(ep->nx.w + oo); nb = ldf(ep->nx.b + oo); }
-    } else if (live && actc == ACT_GELU_TAB) x = ldf(ep->tab + (size_t)ep->row[i] * ep->ld + oo);
+    EpiArgs<T> ea;
+    if (live) ea.load(ep, actc, i, oo, O);
     dot_rows<T, NT, TWO>(X, wa, wb, N, K, vec, a, b);
     if (!live) return;
     float v = 0.f;
 #pragma unroll
     for (int k = 0; k < NT; k++) if (k == i) v = lane < NT ? a[k] : b[k];
     if (bias) v += ldf(bias + oo);
-    if (actc == ACT_JOIN) {
-      const float xn = x + v * s;
-      ep->x[at] = xn;
-      if (ep->nx.h) stf(ep->nx.h + at, ep->nx.alpha ? tanhf(na * xn) * nw + nb : xn);
-      return;
-    }
-    v = act_apply(actc, v, x, alim);
-    if (out32) ((float*)Y)[at] = v;
-    else stf((T*)Y + at, v);
+    ea.finish(ep, actc, v, i, oo, O, Y, out32, alim);
     return;
   }
   dot_rows<T, NT, TWO>(X, wa, wb, N, K, vec, a, b);
@@ -842,13 +853,40 @@ __device__ __forceinline__ void linear_rows_at(const T* __restrict__ X, const T*
   }
 }
 // TWO: two-operand products one output feature a warp, others two (`per` = 1 or 2 output features a warp)
-template <class T, int NT, bool TWO>
-__global__ void __launch_bounds__(256) k_linear_rows(const T* __restrict__ X, const T* __restrict__ Wt, const T* __restrict__ W2,
+template <class T, int NT, bool TWO, bool EP>
+__global__ void __launch_bounds__(256, NT == 1 ? 6 : NT == 2 ? 5 : NT == 4 ? 4 : 2) k_linear_rows(const T* __restrict__ X, const T* __restrict__ Wt, const T* __restrict__ W2,
                                                      void* __restrict__ Y, int out32, int N, int O, int K, int act, int per, float alim,
-                                                     const T* __restrict__ bias, LinEpi<T> ep) {
+                                                     const T* __restrict__ bias, const __grid_constant__ LinEpi<T> ep) {
   const int o = (blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5)) * per;
   if (o >= O) return;
-  linear_rows_at<T, NT, TWO>(X, Wt, W2, Y, out32 != 0, N, O, K, act, o, alim, bias, act == ACT_JOIN || act == ACT_GELU_TAB ? &ep : nullptr);
+  linear_rows_at<T, NT, TWO, EP>(X, Wt, W2, Y, out32 != 0, N, O, K, act, o, alim, bias, ep);
+}
+// The same for products of few output features: four warps of a block take a quarter of the reduction each (two features a block), and
+// their sums are added in warp order.
+template <class T, int NT>
+__global__ void __launch_bounds__(256) k_linear_rows_split(const T* __restrict__ X, const T* __restrict__ Wt, void* __restrict__ Y, int out32, int N, int O, int K, int act,
+                                                           float alim, const T* __restrict__ bias, const __grid_constant__ LinEpi<T> ep) {
+  constexpr int V = Vec16<T>::n;
+  __shared__ float part[8][NT];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, o = blockIdx.x * 2 + (warp >> 2), q = warp & 3;
+  const bool vec = (K % V == 0) && ((((uintptr_t)Wt | (uintptr_t)X) & 15) == 0);
+  const int per = ((K + 3) / 4 + V - 1) / V * V, k0 = min(K, q * per), k1 = min(K, k0 + per);
+  const bool fin = q == 0 && lane < NT && lane < N && o < O;
+  EpiArgs<T> ea;
+  if (fin) ea.load(ep, act, lane, o, O);
+  float a[NT], unused[NT];
+  if (o < O) dot_rows<T, NT, false>(X + k0, Wt + (size_t)o * K + k0, nullptr, N, k1 - k0, vec, a, unused, K);
+  else {
+#pragma unroll
+    for (int i = 0; i < NT; i++) a[i] = 0.f;
+  }
+#pragma unroll
+  for (int i = 0; i < NT; i++) if (lane == i) part[warp][i] = a[i];
+  __syncthreads();
+  if (!fin) return;
+  float v = ((part[warp][lane] + part[warp + 1][lane]) + part[warp + 2][lane]) + part[warp + 3][lane];
+  if (bias) v += ldf(bias + o);
+  ea.finish(ep, act, v, lane, o, O, Y, out32 != 0, alim);
 }
 // several products of the same few rows in one launch (the projections of a mixer in a decode step): blocks are
 // dealt to the products in order, 8 output features each (16 where a warp takes two)
@@ -875,8 +913,8 @@ __global__ void __launch_bounds__(256) k_linear_rows_multi(const T* __restrict__
   if (i >= sg.n) return;
   const int o = (blk * 8 + (threadIdx.x >> 5)) * PER;
   if (o >= sg.O[i]) return;
-  linear_rows_at<T, NT, TWO>(sg.X[i] ? (const T*)sg.X[i] : X, (const T*)sg.W[i], (const T*)nullptr, sg.Y[i], sg.out32[i] != 0, N, sg.O[i],
-                             sg.K[i] > 0 ? sg.K[i] : K, sg.act[i], o, 0.f, (const T*)nullptr);
+  linear_rows_at<T, NT, TWO, false>(sg.X[i] ? (const T*)sg.X[i] : X, (const T*)sg.W[i], (const T*)nullptr, sg.Y[i], sg.out32[i] != 0, N, sg.O[i],
+                             sg.K[i] > 0 ? sg.K[i] : K, sg.act[i], o, 0.f, (const T*)nullptr, LinEpi<T>{});
 }
 
 // ---------------------------------------------------------------------------------------------------------------
