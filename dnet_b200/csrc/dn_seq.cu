@@ -9,6 +9,7 @@
 #include "dn_seq_gdelta.cuh"
 #include "dn_gemm_tc.cuh"      // the tcgen05 / TMA GEMM the llama-family prefill runs on (namespace dn)
 #include "dn_seq_attn_tc.cuh"
+#include "dn_seq_attn_diff.cuh"
 #include "../../include/dnet_b200_seq.h"
 
 #include <algorithm>
@@ -213,6 +214,11 @@ static void make_xmaps(XMaps* x, const void* base, int rows, int cols) {
 }
 
 static int n_maps(const dn_seq_layer_cfg& c) { return c.maps == 2 ? 2 : 1; }
+// layers whose prompt portions take k_diff_attn_tc
+static bool diff_tc_sizes(const dn_seq_cfg& cfg, const dn_seq_layer_cfg& c) {
+  return cfg.dtype == DN_SEQ_BF16 && c.mixer == DN_MIX_ATTENTION && n_maps(c) == 2 && c.softcap <= 0.f && c.scale > 0.f && (c.dim == 64 || c.dim == 128) &&
+         (c.vdim == 64 || c.vdim == 128);
+}
 // rotary frequencies base^(-2j/dims), j = 0 .. dims/2 - 1, optionally scaled.  By a ramp over the pairs (yarn_*): pairs that turn fast
 // within the original context keep theirs, slow ones are divided by the factor, a line between.  By wavelength (band_*): short ones keep
 // theirs, long ones are divided, a blend between.
@@ -522,7 +528,7 @@ extern "C" int dn_seq_model_create(const dn_seq_cfg* cfg, const dn_seq_layer_cfg
           memset(&vm, 0, sizeof(vm));
           const int prows = cfg->pool_pages * PAGE;
           const void* vp = c.v_is_k ? m->kpool.back() : m->vpool.back();
-          const bool ok = sig_tc_sizes(*cfg, c) && make_tmap(&km, m->kpool.back(), prows, l.Ck, PAGE) && make_tmap(&vm, vp, prows, c.v_is_k ? l.Ck : l.Cv, PAGE);
+          const bool ok = (sig_tc_sizes(*cfg, c) || diff_tc_sizes(*cfg, c)) && make_tmap(&km, m->kpool.back(), prows, l.Ck, PAGE) && make_tmap(&vm, vp, prows, c.v_is_k ? l.Ck : l.Cv, PAGE);
           m->kmap.push_back(km);
           m->vmap.push_back(vm);
           m->map_ok.push_back(ok ? 1 : 0);
@@ -884,6 +890,29 @@ static cudaError_t sig_attn(dn_seq_model* m, cudaStream_t s, const Batch& b, int
   const SigParams p{q, out, m->dist_tab, ex.gate, lc.heads, lc.kv_heads, lc.chunk, ex.window, D, std::min(lc.heads / lc.kv_heads, SG_HEADS), lc.scale, m->tc_err};
   if (lc.dim == 64) return lc.vdim == 64 ? sig_attn_launch<64, 64>(m, s, b, kv, p) : sig_attn_launch<64, 128>(m, s, b, kv, p);
   return lc.vdim == 64 ? sig_attn_launch<128, 64>(m, s, b, kv, p) : sig_attn_launch<128, 128>(m, s, b, kv, p);
+}
+
+// differential attention, prompt portions: a CTA per (block of tokens, key head, up to DA_HEADS of its query heads)
+template <int DK, int DV>
+static cudaError_t diff_attn_launch(dn_seq_model* m, cudaStream_t s, const Batch& b, int kv, const DiffParams& p) {
+  constexpr size_t smem = da_smem(DK, DV);
+  static bool attr = false;
+  if (!attr) {
+    cudaError_t e = cudaFuncSetAttribute(k_diff_attn_tc<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return e;
+    attr = true;
+  }
+  const int TB = 128 / p.hpc, R = p.H / p.G;
+  int blocks = 0;
+  for (int n : m->ent_len) blocks += (n + TB - 1) / TB;
+  g_launches++;
+  k_diff_attn_tc<DK, DV><<<dim3(blocks, p.G * ((R + p.hpc - 1) / p.hpc)), DA_THREADS, smem, s>>>(m->kmap[kv], m->vmap[kv], b, p);
+  return cudaGetLastError();
+}
+static cudaError_t diff_attn(dn_seq_model* m, cudaStream_t s, const Batch& b, int kv, const bf16* q, const dn_seq_layer_cfg& lc, const AttnExtra& ex, bf16* out) {
+  const DiffParams p{q, out, ex.lam, lc.heads, lc.kv_heads, lc.chunk, ex.window, ex.keep, std::min(lc.heads / lc.kv_heads, DA_HEADS), lc.scale, ex.post, ex.eps, m->tc_err};
+  if (lc.dim == 64) return lc.vdim == 64 ? diff_attn_launch<64, 64>(m, s, b, kv, p) : diff_attn_launch<64, 128>(m, s, b, kv, p);
+  return lc.vdim == 64 ? diff_attn_launch<128, 64>(m, s, b, kv, p) : diff_attn_launch<128, 128>(m, s, b, kv, p);
 }
 
 // few rows: the latency form (k_attn_rows) where the head sizes fit it.  Two stages a warp where a row's keys can exceed what the
@@ -1297,7 +1326,9 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
         CK(launch(k_pool_rows<T>, dim3(N), dim3(128), 0, s, b, lc.pool, Ckk, lc.v_is_k ? 0 : lc.kv_heads * lc.vdim, (const T*)m->kpool[run.kv_index], (const T*)vpl,
                   (T*)pkp, (T*)pvp));
       PH(DN_SEQ_PH_ATTN);
-      if (b.max_len >= 16 && m->map_ok[run.kv_index] && sig_tc_sizes(c, lc))
+      if (b.max_len >= 16 && m->map_ok[run.kv_index] && diff_tc_sizes(c, lc))
+        CK(diff_attn(m, s, b, run.kv_index, (const bf16*)m->qb, lc, ex, (bf16*)m->mo));
+      else if (b.max_len >= 16 && m->map_ok[run.kv_index] && sig_tc_sizes(c, lc))
         CK(sig_attn(m, s, b, run.kv_index, (const bf16*)m->qb, lc, ex, (bf16*)m->mo));
       else if (attn_tiles_ok<T>(lc, b))
         CK(attn_tiles(s, b, (const bf16*)m->qb, (const bf16*)m->kpool[run.kv_index], (const bf16*)vpl, lc, ex, (bf16*)m->mo));
