@@ -1318,6 +1318,10 @@ static int step_T(dn_seq_model* m, const Batch& b, int n_want, const int32_t* wa
         CK(launch(kern, dim3((N + tok - 1) / tok, (units + PREP_WARPS - 1) / PREP_WARPS), dim3(32 * PREP_WARPS), 0, s, a, b, tok, (const T*)m->uq, (const T*)m->uk,
                   (const T*)m->uv, w(DN_SQ_Q_CONV), w(DN_SQ_K_CONV), w(DN_SQ_V_CONV), w(DN_SQ_Q_NORM), w(DN_SQ_K_NORM), cst, m->conv_stride, (T*)m->qb,
                   (T*)m->kpool[run.kv_index], (T*)m->vpool[run.kv_index]));
+      } else if (lc.conv == 0 && lc.qk_norm != DN_QKNORM_WHOLE && lc.rot_dims <= 2 * ROT_MAX_PAIRS) {
+        const int units = Hm + (l.Ck ? Gm + (lc.v_is_k ? 0 : lc.kv_heads) : 0), per = N > 64 ? 8 : 1;      // (many tokens: eight heads share their cosines and sines)
+        CK(launch(k_attn_prep_rot<T>, dim3(N, (units + per * PREP_WARPS - 1) / (per * PREP_WARPS)), dim3(32 * PREP_WARPS), 0, s, a, b, per, (const T*)m->uq, (const T*)m->uk,
+                  (const T*)m->uv, w(DN_SQ_Q_NORM), w(DN_SQ_K_NORM), (T*)m->qb, (T*)m->kpool[run.kv_index], (T*)m->vpool[run.kv_index]));
       } else
         CK(launch(k_attn_prep<T>, dim3(N), dim3(256), sm, s, a, b, (const T*)m->uq, (const T*)m->uk, (const T*)m->uv, w(DN_SQ_Q_CONV),
                   w(DN_SQ_K_CONV), w(DN_SQ_V_CONV), w(DN_SQ_Q_NORM), w(DN_SQ_K_NORM), cst, m->conv_stride, (T*)m->qb,

@@ -1245,6 +1245,66 @@ __global__ void __launch_bounds__(32 * PREP_WARPS) k_attn_prep_heads(AttnPrep a,
   }
 }
 
+// The same for heads without convolutions that rotate (and are normed alone or not at all): a warp takes `per` heads of one token, in the
+// order q, k, v, and forms the token's cosines and sines once for them.  A head's sum of squares runs over a lane's dims in ascending order,
+// then pairwise over the lanes, so a head's result depends on its own row only.
+constexpr int ROT_MAX_PAIRS = 128;
+template <class T>
+__global__ void __launch_bounds__(32 * PREP_WARPS) k_attn_prep_rot(AttnPrep a, Batch b, int per, const T* __restrict__ Uq, const T* __restrict__ Uk, const T* __restrict__ Uv,
+                                                                   const T* __restrict__ nq, const T* __restrict__ nk, T* __restrict__ qout, T* __restrict__ kpool,
+                                                                   T* __restrict__ vpool) {
+  const int n = blockIdx.x, lane = threadIdx.x & 31, units = a.H + (a.own_kv ? a.G + (a.own_v ? a.gv : 0) : 0);
+  int u = (blockIdx.y * PREP_WARPS + (threadIdx.x >> 5)) * per;
+  const int u1 = min(units, u + per);
+  if (u >= units) return;
+  const int p = b.pos[n], hr = a.rot / 2;
+  float cs[ROT_MAX_PAIRS / 32], sn[ROT_MAX_PAIRS / 32];
+#pragma unroll
+  for (int x = 0; x < ROT_MAX_PAIRS / 32; x++) {
+    const int i = x * 32 + lane;
+    if (i < hr && u < a.H + a.G) {
+      sincosf((float)p * a.inv_freq[i], &sn[x], &cs[x]);
+      cs[x] *= a.mscale;
+      sn[x] *= a.mscale;
+    }
+  }
+  const float qt = a.qt_every > 0 ? 1.f + a.qt_coef * logf((float)((p + 1) / a.qt_every + 1)) : 1.f;
+  const size_t row = (size_t)b.bt[(size_t)b.slot[n] * b.max_pages + p / PAGE] * PAGE + p % PAGE;
+  for (; u < u1; u++) {
+    if (u >= a.H + a.G) {      // a value head
+      const size_t c = (size_t)(u - a.H - a.G) * a.dv;
+      const T* in = Uv + (size_t)n * a.gv * a.dv + c;
+      T* out = vpool + row * a.gv * a.dv + c;
+      for (int d = lane; d < a.dv; d += 32) out[d] = in[d];
+      continue;
+    }
+    const bool isq = u < a.H;
+    const int h = isq ? u : u - a.H, heads = isq ? a.H : a.G;
+    const T* in = (isq ? Uq : Uk) + ((size_t)n * heads + h) * a.dk;
+    T* out = isq ? qout + ((size_t)n * heads + h) * a.dk : kpool + (row * heads + h) * a.dk;
+    const T* nw = isq ? nq : nk;
+    float f = 1.f;
+    if (a.norm == 2) {
+      float ss = 0.f;
+      for (int d = lane; d < a.dk; d += 32) { const float x = ldf(in + d); ss += x * x; }
+      f = 1.f / sqrtf(warp_sum(ss) / (float)a.dk + a.eps);
+    }
+    const float s = isq ? qt : 1.f;
+    auto val = [&](int d) { return a.norm == 2 ? ldf(in + d) * f * ldf(nw + d) : ldf(in + d); };
+#pragma unroll
+    for (int x = 0; x < ROT_MAX_PAIRS / 32; x++) {
+      const int i = x * 32 + lane;
+      if (i < hr) {
+        const int ia = a.half ? i : 2 * i, ib = a.half ? i + hr : 2 * i + 1;
+        const float y0 = val(ia), y1 = val(ib);
+        stf(out + ia, (y0 * cs[x] - y1 * sn[x]) * s);
+        stf(out + ib, (y1 * cs[x] + y0 * sn[x]) * s);
+      }
+    }
+    for (int d = a.rot + lane; d < a.dk; d += 32) stf(out + d, val(d) * s);
+  }
+}
+
 // Mean-pooled blocks behind a sliding window.  Block j of a sequence holds the positions j P .. j P + P - 1; its pooled
 // key (value) is the mean of the P keys (values) as the pages hold them.  A pooled row lives with the page of the
 // block's last position e = j P + P - 1: row j - floor(64 (e / 64) / P) of that page's POOL_ROWS(P) = ceil(64 / P) rows
