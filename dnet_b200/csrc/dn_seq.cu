@@ -790,7 +790,7 @@ static cudaError_t linear(dn_seq_model* m, cudaStream_t s, const T* X, const voi
                           int act, LinMaps tm = LinMaps{nullptr, nullptr, nullptr}, float alim = 0.f, const void* bias = nullptr, const LinEpi<T>* ep = nullptr) {
   const LinEpi<T> epi = ep ? *ep : LinEpi<T>{nullptr, nullptr, 0, nullptr, nullptr, 1.f, {nullptr, nullptr, nullptr, nullptr}};
   // (a weight of fewer than 128 rows fills part of a tile: still far ahead of the CUDA-core tiles once K is in the thousands)
-  if (std::is_same<T, bf16>::value && N >= 16 && O >= 16 && tm.w && tm.x && tm.x->ok && (!bias || act == ACT_RELU2 || (act == ACT_NONE && out32)) &&
+  if (std::is_same<T, bf16>::value && N >= 16 && tm.w && tm.x && tm.x->ok && (!bias || act == ACT_RELU2 || (act == ACT_NONE && out32)) &&
       (act == ACT_NONE || act == ACT_TANH || act == ACT_RELU2 || act == ACT_GELU_TAB || act == ACT_JOIN || (act_two(act) && tm.w2))) {
     dn::TcParams p;
     memset(&p, 0, sizeof(p));
