@@ -65,7 +65,8 @@ def test_header_and_binding_agree():
              "HEAD_GATE": "head_gate", "SINK": "sink", "BONUS": "bonus", "DECAY1": "decay1", "DECAY2": "decay2", "DECAY_B": "decay.b",
              "ROUTER": "router", "ROUTER_B": "router.b", "SH_GATE": "shared.gate", "SH_UP": "shared.up", "SH_DOWN": "shared.down",
              "UP_B": "mlp.up.b", "DOWN_B": "mlp.down.b", "ROUTER_CORR": "router.corr", "SH_SG": "shared.sg",
-             "CANON1": "canon1", "CANON2": "canon2", "L_OUT": "l.out", "DIST1": "mix.r1", "DIST2": "mix.r2", "ATTN_OFF": "mix.pb"}
+             "CANON1": "canon1", "CANON2": "canon2", "L_OUT": "l.out", "DIST1": "mix.r1", "DIST2": "mix.r2", "ATTN_OFF": "mix.pb",
+             "LS1": "ls1", "LS2": "ls2", "SIDE_GATE": "side.gate", "SIDE_PROJ": "side.proj", "SIDE_NORM": "side.norm"}
     for i, name in enumerate(order):
         n = name[len("DN_SQ_"):]
         if n in spell:
@@ -77,7 +78,7 @@ def test_header_and_binding_agree():
         assert _seqabi.LAYER_SLOT[want] == i, (name, want)
     model = [n.strip().split("=")[0].strip() for n in txt.split("DN_SQ_COUNT,", 1)[1].split("}", 1)[0].replace("\n", " ").split(",") if n.strip()]
     assert [_seqabi.MODEL_SLOT[k] for k in ("embed", "final.norm", "head", "final.norm.b", "final.norm.alpha", "embed.norm", "embed.norm.b",
-                                           "embed.norm.alpha", "loop.in", "bigram", "pos")] == list(range(100, 100 + len(model)))
+                                           "embed.norm.alpha", "loop.in", "bigram", "pos", "side.embed")] == list(range(100, 100 + len(model)))
 
 
 def _filinex_cfg():
@@ -562,3 +563,73 @@ def test_generate_refuses_requests_beyond_the_position_table():
     assert not eng.live
     with pytest.raises(ValueError, match="empty"):
         eng.generate([GenRequest("none", [])])
+
+
+def _tuguvik_cfg():
+    lat = {"heads": 3, "dim": 10, "rot_dim": 6, "vdim": 7, "kv_rank": 12, "q_rank": 9, "scale": 0.3, "mask": {"size": 19},
+           "rot": {"base": 700.0, "dims": 6, "scaling": {"factor": 3.0, "original": 40, "fast": 8.0, "slow": 0.5}}}
+    dif = {"heads": 4, "kv_heads": 2, "dim": 8, "vdim": 5, "scale": 0.35, "diff": 0.25, "mask": {"size": 23, "keep_first": 6},
+           "rot": {"base": 90.0, "dims": 4, "scaling": {"factor": 5.0, "low": 1.5, "high": 3.0, "original": 60}}}
+    dense = {"kind": "dense", "ff": 24}
+    return {"architecture": "Tuguvik", "vocab": 50, "width": 36, "norm": {"eps": 1e-5}, "token_side": {"dim": 11},
+            "layers": [{"type": "latent_attention", "mixer": lat, "mlp": dense}, {"type": "attention", "mixer": dif, "mlp": None},
+                       {"type": "latent_attention", "mixer": {**lat, "kv_from": 0, "heads": 2}, "mlp": None}]}
+
+
+def test_tuguvik_config_and_checkpoint_names():
+    """every constant of the config lands in the structs, what the design fixes comes from the family, and every tensor the
+    oracle writes finds its place through the aliases with its shape"""
+    from dnet_b200 import _seqabi
+    from dnet_b200.core.models import ring_model_class
+    from dnet_b200.core.models.seqmix import _LAYER_KEY, parse_layer_list
+    from oracle import tuguvik_oracle as to
+
+    cfg = _tuguvik_cfg()
+    cls = ring_model_class("tuguvik")
+    sc, layers = parse_layer_list(cfg, cls.family, to.tensor_shapes(cfg))
+    assert (sc.norm_kind, sc.layer_scale, sc.side_dim, sc.post_norm, sc.no_pre_norm, sc.parallel_ff) == (_seqabi.DN_NORM_DYT, 1, 11, 0, 0, 0)
+    a, b, c = layers
+    assert (a.mixer, a.q_rank, a.kv_rank, a.rot_part, a.out_gate, a.sink, a.kv_from, a.maps) == (_seqabi.DN_MIX_LATENT, 9, 12, 6, 1, 1, -1, 0)
+    assert (a.rot_layout, a.yarn_factor, a.yarn_original, a.yarn_fast, a.yarn_slow, a.band_factor) == (_seqabi.DN_ROT_INTERLEAVED, 3.0, 40.0, 8.0, 0.5, 0.0)
+    assert (a.ff_act, a.ff, a.chunk, a.mask_kind) == (_seqabi.DN_FF_SWIGLU, 24, 19, _seqabi.DN_MASK_WINDOW)
+    assert (b.mixer, b.maps, b.diff, b.keep_first, b.chunk, b.sink, b.out_gate) == (_seqabi.DN_MIX_ATTENTION, 2, 0.25, 6, 23, 0, 0)
+    assert (b.rot_layout, b.rot_dims, b.yarn_factor) == (_seqabi.DN_ROT_HALF, 4, 0.0)
+    assert (b.band_factor, b.band_low, b.band_high, b.band_original) == (5.0, 1.5, 3.0, 60.0)
+    assert (c.kv_from, c.heads, c.ff) == (0, 2, 0)
+    m = cls.__new__(cls)
+    m.config, m._cfg_struct, m._layer_structs, m.hidden_size, m.vocab_size = cfg, sc, layers, sc.width, sc.vocab
+    want, got = m.expected_tensors(), {}
+    for key, sh in to.tensor_shapes(cfg).items():
+        if _LAYER_KEY.match(key):
+            lname, suffix = key.split(".", 1)
+            kind = cfg["layers"][int(lname[1:])]["type"]
+            key = f"{lname}.{cls.tensor_alias.get(kind, {}).get(suffix, suffix)}"
+        got[key] = tuple(sh)
+    assert got == {k: tuple(v) for k, v in want.items()}
+    assert want["side.embed"] == (50, 33) and "l2.mix.dkv" not in want and "l1.ls2" not in want
+    for k in want:
+        if _LAYER_KEY.match(k):
+            assert k.split(".", 1)[1] in _seqabi.LAYER_SLOT, k
+        else:
+            assert k in _seqabi.MODEL_SLOT, k
+
+
+def test_tuguvik_oracle_by_hand():
+    """the oracle's pieces on numbers small enough to follow"""
+    from oracle import tuguvik_oracle as to
+
+    D = torch.float64
+    # position 9 with a window of 3 that keeps 2 tokens
+    assert to.visible(9, {"size": 3, "keep_first": 2}) == [0, 1, 7, 8, 9] and to.visible(3, {"size": 3, "keep_first": 2}) == [0, 1, 2, 3]
+    assert to.visible(2, None) == [0, 1, 2] and to.visible(4, {"size": 1}) == [4]
+    # two equal scores and a sink of the same size: a third each; without it a half
+    s, vis = torch.zeros(2, 2, dtype=D), torch.ones(2, 2, dtype=torch.bool)
+    assert torch.allclose(to.weights_with_sink(s, vis, torch.tensor(0.0, dtype=D)), torch.full((2, 2), 1 / 3, dtype=D))
+    assert torch.allclose(to.weights_with_sink(s, vis, None), torch.full((2, 2), 0.5, dtype=D))
+    # wavelengths: f = 1 (2 pi) below original / high keeps its frequency, a long one is divided
+    f = to.banded_frequencies(4, 1e6, {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 100})
+    assert f[0] == 1.0 and abs(f[1] - 1e-3 / 8) < 1e-15
+    f, mult = to.ramped_frequencies(4, 1e6, {"factor": 8.0, "original": 100, "fast": 4.0, "slow": 1.0})
+    assert f[0] == 1.0 and abs(f[1] - 1e-3 / 8) < 1e-15 and abs(mult - (0.1 * math.log(8.0) + 1.0)) < 1e-12
+    w = {"mix.lq1": torch.tensor([1.0, 2.0], dtype=D), "mix.lk1": torch.tensor([0.5, 0.25], dtype=D), "mix.lq2": torch.zeros(2, dtype=D), "mix.lk2": torch.ones(2, dtype=D)}
+    assert abs(float(to.diff_lambda(w, "", 0.3)) - (math.e - 1.0 + 0.3)) < 1e-12
